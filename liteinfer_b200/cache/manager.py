@@ -6,7 +6,7 @@ What the model must remember between steps is declared by its parts
 page allocator, and one block table per request (logical block -> page, -1 once
 given back).  A group that keeps every key never frees a page before the
 request ends; a group with a window frees the pages that the window has passed
-after each step.  Beside the groups, every request holds one slot of
+after each step, a group read in chunks those of the chunks that are over.  Beside the groups, every request holds one slot of
 fixed-size state for the mixers that declare a `StateNeed` (the slot exists
 even when no layer uses it, so the step function always passes one).  A layer
 may declare several needs of either kind (two mixers in one block, a mixer with
@@ -57,24 +57,21 @@ class KVGroup:
     @property
     def kept_blocks(self) -> int:
         """Leading blocks that a window never passes: those of the first tokens that stay visible."""
-        return _cdiv(self.need.keep_first, self.page_size) if self.need.window is not None else 0
+        return 0 if self.need.keeps_all else _cdiv(self.need.keep_first, self.page_size)
 
     def pages_at(self, total: int, largest_step: int) -> int:
         """The most pages a request holds here at any time on its way to `total` tokens, when no step brings it
         more than `largest_step` of them: every block for a group that keeps all keys; for a group with a
-        window, the blocks that the window still reaches at a step's start plus those the step writes."""
+        window or chunks, the blocks that are still read at a step's start plus those the step writes."""
         every = _cdiv(total, self.page_size)
-        if self.need.window is None:
+        if self.need.keeps_all:
             return every
-        span = self.need.window - 1 + max(1, min(largest_step, total))
+        span = self.need.span - 1 + max(1, min(largest_step, total))
         return min(every, _cdiv(span, self.page_size) + 1 + self.kept_blocks)
 
     def first_needed_block(self, total: int) -> int:
         """First logical block a request holding `total` tokens can still read."""
-        if self.need.window is None:
-            return 0
-        # The next query sits at position >= total and sees keys > position - window.
-        return max(0, total - self.need.window + 1) // self.page_size
+        return self.need.first_needed(total) // self.page_size
 
     def missing_blocks(self, request_id: str, old_total: int, new_total: int) -> list[int]:
         """Logical blocks that positions [old_total, new_total) touch and that hold no page yet."""
@@ -263,10 +260,10 @@ class CacheManager:
                     table[block] = page
 
     def commit(self, request_id: str, new_total: int) -> None:
-        """The step that wrote up to `new_total` succeeded: count it, and give back what a window has passed."""
+        """The step that wrote up to `new_total` succeeded: count it, and give back what no later token reads."""
         self._length[request_id] = new_total
         for group in self.groups:
-            if group.need.window is None:
+            if group.need.keeps_all:
                 continue
             table = group.tables[request_id]
             passed = min(group.first_needed_block(new_total), len(table))

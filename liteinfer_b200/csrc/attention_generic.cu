@@ -26,10 +26,11 @@
 
 namespace li {
 
-constexpr int kMaxHeadDim = 256;
+constexpr int kMaxKeyDim = 1024;
 constexpr int kQueriesPerBlock = 8;
 
-template <typename T>
+// kDimsPerLane: a lane keeps this many of a value's dimensions, so values have at most 32 times as many.
+template <typename T, int kDimsPerLane>
 __global__ void __launch_bounds__(256)
 paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, T* __restrict__ out, int out_row_stride,
                                const T* __restrict__ k_pool, const T* __restrict__ v_pool,
@@ -50,8 +51,6 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, T* __r
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nwarps = blockDim.x >> 5;
   float* qs = q_smem + warp * head_dim;
   const int* table = block_table + (size_t)seq * table_stride;
-  constexpr int kDimsPerLane = kMaxHeadDim / 32;
-
   for (int row = warp; row < rows; row += nwarps) {
     const int qi = tile_start + row / groups;          // query index within the sequence's queries
     const int head = kvh * groups + row % groups;
@@ -61,8 +60,7 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, T* __r
     for (int d = lane; d < head_dim; d += 32) qs[d] = to_float(qrow[d]);
     __syncwarp();
 
-    int first = 0;
-    if (window > 0 && qpos - window + 1 > 0) first = qpos - window + 1;
+    const int first = first_visible(qpos, window);
     float m = -INFINITY, l = 0.f;
     float acc[kDimsPerLane];
 #pragma unroll
@@ -131,13 +129,26 @@ paged_attention_generic_kernel(const T* __restrict__ q, int q_row_stride, T* __r
   }
 }
 
+template <typename T, int kDimsPerLane>
+int launch_generic(dim3 grid, int threads, size_t smem, cudaStream_t stream, const void* q, int q_row_stride, void* out,
+                   int out_row_stride, const void* k_pool, const void* v_pool, const int* block_table, int table_stride,
+                   const int* query_start_loc, const int* context_lens, int heads, int kv_heads, int head_dim, int v_dim,
+                   int page_size, int num_pages, float scale, int window, int keep_first, float softcap,
+                   const float* sink) {
+  paged_attention_generic_kernel<T, kDimsPerLane><<<grid, threads, smem, stream>>>(
+      (const T*)q, q_row_stride, (T*)out, out_row_stride, (const T*)k_pool, (const T*)v_pool, block_table, table_stride,
+      query_start_loc, context_lens, heads, kv_heads, head_dim, v_dim, page_size, num_pages, scale, window, keep_first,
+      softcap, sink);
+  LI_LAUNCH_CHECK();
+}
+
 }  // namespace li
 
 using namespace li;
 
 // q: [tokens, q_row_stride] with head h of a token at columns [h*head_dim, (h+1)*head_dim).
 // out: [tokens, out_row_stride] with head h at columns [h*v_dim, (h+1)*v_dim).  k_pool: [num_pages, kv_heads,
-// page_size, head_dim]; v_pool likewise with v_dim.  window <= 0: every earlier key is visible.  sink: null or [heads].
+// page_size, head_dim]; v_pool likewise with v_dim.  window: see first_visible (common.cuh).  sink: null or [heads].
 LI_EXPORT int li_paged_attention_generic(int dtype, const void* q, int q_row_stride, void* out, int out_row_stride,
                                          const void* k_pool, const void* v_pool, const int* block_table,
                                          int table_stride, const int* query_start_loc, const int* context_lens,
@@ -146,21 +157,21 @@ LI_EXPORT int li_paged_attention_generic(int dtype, const void* q, int q_row_str
                                          int keep_first, float softcap, const float* sink,
                                          cudaStream_t stream) {
   if (num_seqs == 0 || max_q_len == 0) return 0;
-  if (head_dim < 1 || head_dim > kMaxHeadDim || kv_heads < 1 || heads % kv_heads) return LI_ERR_UNSUPPORTED;
-  if (v_dim < 1 || v_dim > kMaxHeadDim) return LI_ERR_UNSUPPORTED;
+  if (head_dim < 1 || head_dim > kMaxKeyDim || kv_heads < 1 || heads % kv_heads) return LI_ERR_UNSUPPORTED;
+  if (v_dim < 1 || v_dim > 32 * 32) return LI_ERR_UNSUPPORTED;
   if (kv_heads > 65535 || num_seqs > 65535) return LI_ERR_UNSUPPORTED;
   const int threads = 256;
   const dim3 grid((max_q_len + kQueriesPerBlock - 1) / kQueriesPerBlock, kv_heads, num_seqs);
   const size_t smem = (size_t)(threads / 32) * head_dim * sizeof(float);
-  if (dtype == kFloat32)
-    paged_attention_generic_kernel<float><<<grid, threads, smem, stream>>>(
-        (const float*)q, q_row_stride, (float*)out, out_row_stride, (const float*)k_pool, (const float*)v_pool,
-        block_table, table_stride, query_start_loc, context_lens, heads, kv_heads, head_dim, v_dim, page_size,
-        num_pages, scale, window, keep_first, softcap, sink);
-  else
-    paged_attention_generic_kernel<bf16><<<grid, threads, smem, stream>>>(
-        (const bf16*)q, q_row_stride, (bf16*)out, out_row_stride, (const bf16*)k_pool, (const bf16*)v_pool,
-        block_table, table_stride, query_start_loc, context_lens, heads, kv_heads, head_dim, v_dim, page_size,
-        num_pages, scale, window, keep_first, softcap, sink);
-  LI_LAUNCH_CHECK();
+#define LI_GENERIC(T, N)                                                                                              \
+  return launch_generic<T, N>(grid, threads, smem, stream, q, q_row_stride, out, out_row_stride, k_pool, v_pool,       \
+                              block_table, table_stride, query_start_loc, context_lens, heads, kv_heads, head_dim,    \
+                              v_dim, page_size, num_pages, scale, window, keep_first, softcap, sink)
+  if (dtype == kFloat32) {
+    if (v_dim <= 256) LI_GENERIC(float, 8);
+    LI_GENERIC(float, 32);
+  }
+  if (v_dim <= 256) LI_GENERIC(bf16, 8);
+  LI_GENERIC(bf16, 32);
+#undef LI_GENERIC
 }

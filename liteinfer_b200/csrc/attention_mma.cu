@@ -36,7 +36,7 @@ namespace li {
 // is a few instructions per copy; a page size that is a power of two is divided by shifting.
 template <int D>
 __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const AttnParams& p, const int* table, int kvh,
-                                             int tile_start, int lo, int hi, int kept_end = 0) {
+                                             int part, int tile_start, int lo, int hi, int kept_end = 0) {
   constexpr int kChunks = D / 8;
   constexpr int kKeysPerPass = kWarps * 32 / kChunks;
   const int chunk = threadIdx.x % kChunks, key0 = threadIdx.x / kChunks;
@@ -45,16 +45,20 @@ __device__ __forceinline__ void load_kv_tile(bf16* ks, bf16* vs, const AttnParam
     const int key = key0 + pass * kKeysPerPass;
     const int kpos = tile_start + key;
     bool valid = (kpos >= lo || kpos < kept_end) && kpos < hi;
-    size_t off = 0;
+    size_t off = 0, v_off = 0;
     if (valid) {
       const int block = p.page_shift >= 0 ? kpos >> p.page_shift : kpos / p.page_size;
       const int slot = p.page_shift >= 0 ? kpos & (p.page_size - 1) : kpos - block * p.page_size;
       const int page = table[block];
       valid = page >= 0 && page < p.num_pages;
-      if (valid) off = (((size_t)page * p.kv_heads + kvh) * p.page_size + slot) * D + chunk * 8;
+      if (valid) {
+        const size_t row = ((size_t)page * p.kv_heads + kvh) * p.page_size + slot;
+        off = row * D + chunk * 8;
+        v_off = (row * p.v_parts + part) * D + chunk * 8;
+      }
     }
     cp_async16(tile_ptr<D>(ks, key, chunk), p.k_pool + off, valid);
-    cp_async16(tile_ptr<D>(vs, key, chunk), p.v_pool + off, valid);
+    cp_async16(tile_ptr<D>(vs, key, chunk), p.v_pool + v_off, valid);
   }
 }
 
@@ -74,7 +78,7 @@ attention_mma_kernel(const AttnParams p) {
   // Tables and lengths are inputs of the step; what an earlier kernel wrote is read after the wait below.
   const int seq = p.seq_index ? p.seq_index[blockIdx.z] : blockIdx.z;
   if (seq < 0) return;        // a place of padding in the list of sequences
-  const int kvh = blockIdx.y;
+  const int kvh = (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts;
   // The last query tiles see the most keys: they are handed out first.
   const int split = blockIdx.x % p.num_splits, qtile = (int)(gridDim.x / p.num_splits) - 1 - (int)(blockIdx.x / p.num_splits);
   const int q_begin = p.query_start_loc[seq], q_len = p.query_start_loc[seq + 1] - q_begin;
@@ -95,7 +99,7 @@ attention_mma_kernel(const AttnParams p) {
   // Visible keys of this tile: [lo, hi).
   const int first_qpos = ctx - q_len + q0, last_qpos = first_qpos + tile_q - 1;
   const int hi = last_qpos + 1;
-  const int lo = (p.window > 0 && first_qpos - p.window + 1 > 0) ? first_qpos - p.window + 1 : 0;
+  const int lo = first_visible(first_qpos, p.window);
   const int tile_lo = lo / kBlockN, tile_hi = (hi + kBlockN - 1) / kBlockN;   // key tiles [tile_lo, tile_hi)
   // The first keys that stay visible behind the window, [0, kept_end), are walked first: the tiles that hold
   // them and lie before the window's first tile get the places [place_lo, tile_lo) in front of the window's
@@ -123,7 +127,7 @@ attention_mma_kernel(const AttnParams p) {
 #pragma unroll
     for (int st = 0; st < kStages - 1; ++st) {
       if (my_lo + st < my_hi)
-        load_kv_tile<D>(kbuf + st * kBlockN * D, vbuf + st * kBlockN * D, p, table, kvh,
+        load_kv_tile<D>(kbuf + st * kBlockN * D, vbuf + st * kBlockN * D, p, table, kvh, part,
                         LI_TILE_AT(my_lo + st) * kBlockN, lo, hi, kept_end);
       cp_async_commit();
     }
@@ -167,9 +171,9 @@ attention_mma_kernel(const AttnParams p) {
           }
         } else {
           const int j = (w - kItems) * 8;
-          const Vec16<bf16> v = load16(p.v_new + token + (size_t)kvh * D + j);
+          const Vec16<bf16> v = load16(p.v_new + token + ((size_t)kvh * p.v_parts + part) * D + j);
           store16(newest + D + j, v);
-          if (store) store16(v_pool + dst + j, v);
+          if (store) store16(v_pool + dst * p.v_parts + (size_t)part * D + j, v);
         }
       }
     }
@@ -189,7 +193,7 @@ attention_mma_kernel(const AttnParams p) {
 #pragma unroll
     for (int st = 0; st < kStages - 1; ++st) {
       if (my_lo + st < my_hi)
-        load_kv_tile<D>(kbuf + st * kBlockN * D, vbuf + st * kBlockN * D, p, table, kvh,
+        load_kv_tile<D>(kbuf + st * kBlockN * D, vbuf + st * kBlockN * D, p, table, kvh, part,
                         LI_TILE_AT(my_lo + st) * kBlockN, lo, hi, kept_end);
       cp_async_commit();
     }
@@ -204,12 +208,14 @@ attention_mma_kernel(const AttnParams p) {
                 tile_ptr<D>(qs, row_base + (lane & 15), kk * 2 + (lane >> 4)));
 
   // Rows of this thread: row_base + g and + 8.
-  int qpos[2];
+  int qpos[2], row_lo[2];
 #pragma unroll
   for (int h = 0; h < 2; ++h) {
     const int row = row_base + g + 8 * h;
     qpos[h] = row < rows_used ? first_qpos + row / groups : -1;   // -1: a padding row sees nothing
+    row_lo[h] = first_visible(qpos[h], p.window);
   }
+  const int last_lo = first_visible(last_qpos, p.window);
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
   float o[D / 8][4];
 #pragma unroll
@@ -226,7 +232,7 @@ attention_mma_kernel(const AttnParams p) {
     {
       const int ahead = place + kStages - 1, abuf = (ahead - my_lo) % kStages;
       if (ahead < my_hi)
-        load_kv_tile<D>(kbuf + abuf * kBlockN * D, vbuf + abuf * kBlockN * D, p, table, kvh,
+        load_kv_tile<D>(kbuf + abuf * kBlockN * D, vbuf + abuf * kBlockN * D, p, table, kvh, part,
                         LI_TILE_AT(ahead) * kBlockN, lo, hi, kept_end);
     }
     cp_async_commit();
@@ -268,7 +274,7 @@ attention_mma_kernel(const AttnParams p) {
     // A tile needs the mask only where it meets the diagonal or the window's start.  (Rows of padding hold
     // zero queries: their scores are finite, and they are never stored.)
     const bool all_visible = (tile + 1) * kBlockN - 1 <= first_qpos &&
-                             (p.window <= 0 || tile * kBlockN > last_qpos - p.window);
+                             (p.window == 0 || tile * kBlockN >= last_lo);
     if (capped) {
 #pragma unroll
       for (int i = 0; i < kGroupsPerWarp * 2; ++i)
@@ -290,7 +296,7 @@ attention_mma_kernel(const AttnParams p) {
         for (int j = 0; j < 4; ++j) {
           const int kpos = key0 + i * 8 + 2 * t + (j & 1);
           const int qp = qpos[j >> 1];
-          const bool visible = kpos <= qp && (p.window <= 0 || kpos > qp - p.window || kpos < p.keep_first);
+          const bool visible = kpos <= qp && (kpos >= row_lo[j >> 1] || kpos < p.keep_first);
           s[i][j] = visible ? s[i][j] * p.scale_log2 : -INFINITY;
           tile_max[j >> 1] = fmaxf(tile_max[j >> 1], s[i][j]);
         }
@@ -373,7 +379,7 @@ attention_mma_kernel(const AttnParams p) {
       }
     }
     __syncthreads();
-    combine_warps<D>(p, os, ms, ls, rows_used, groups, q_begin, q0, kvh, split);
+    combine_warps<D>(p, os, ms, ls, rows_used, groups, q_begin, q0, kvh, part, split);
   } else {
 #pragma unroll
     for (int h = 0; h < 2; ++h) {
@@ -383,12 +389,12 @@ attention_mma_kernel(const AttnParams p) {
       if (p.num_splits == 1 && p.sink != nullptr) l[h] += exp2f(p.sink[head] * kLog2e - m[h]);
       const float inv = l[h] > 0.f ? 1.f / l[h] : 0.f;
       if (p.num_splits == 1) {
-        bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (size_t)head * D;
+        bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (size_t)out_head(p, head, part) * D;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
           *reinterpret_cast<unsigned*>(dst + i * 8 + 2 * t) = pack_bf16(o[i][2 * h] * inv, o[i][2 * h + 1] * inv);
       } else {
-        const size_t slot = ((size_t)(q_begin + qi) * p.heads + head) * p.num_splits + split;
+        const size_t slot = ((size_t)(q_begin + qi) * p.heads * p.v_parts + out_head(p, head, part)) * p.num_splits + split;
         float* dst = p.partial_out + slot * D;
 #pragma unroll
         for (int i = 0; i < D / 8; ++i)
@@ -400,7 +406,7 @@ attention_mma_kernel(const AttnParams p) {
   }
   if (p.num_splits == 1) return;
 
-  merge_splits<D>(p, smem_raw, &is_last, rows_used, groups, q_begin, q0, kvh, qtile);
+  merge_splits<D>(p, smem_raw, &is_last, rows_used, groups, q_begin, q0, kvh, part, qtile);
 }
 
 template <int D, bool kDecode, int kStages>
@@ -415,7 +421,7 @@ int launch_attention(const AttnParams& p, int num_seqs, int max_q_len, cudaStrea
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const dim3 grid(((max_q_len + tq - 1) / tq) * p.num_splits, p.kv_heads, num_seqs);
+  const dim3 grid(((max_q_len + tq - 1) / tq) * p.num_splits, p.kv_heads * p.v_parts, num_seqs);
   return (int)launch_pdl((long)num_seqs * max_q_len, attention_mma_kernel<D, kDecode, kStages>, grid, dim3(kWarps * 32), smem, stream, p);
 }
 
@@ -442,7 +448,8 @@ int decode_capacity() {
 
 using namespace li;
 
-// Counters the launch needs when num_splits > 1 (unsigned, all zero before the first launch).
+// Counters the launch needs when num_splits > 1 (unsigned, all zero before the first launch), for each part of D
+// dimensions that a value has.
 LI_EXPORT int li_paged_attention_mma_counters(int num_seqs, int max_q_len, int heads, int kv_heads) {
   const int groups = heads / kv_heads;
   const bool decode = max_q_len == 1 && groups <= 16;
@@ -459,11 +466,12 @@ LI_EXPORT int li_paged_attention_mma_decode_capacity(int head_dim) {
 // Tensor-core paged attention (bfloat16; head_dim 64 or 128; groups of at most 64 heads).
 // keep_first (with a window): the first keys of a sequence stay visible behind the window.  softcap > 0: a scaled
 // score s becomes softcap * tanh(s / softcap).  Neither goes with rope_inv_freq.  sink (optional, [heads] float32):
-// exp(sink[h]) is one more term of head h's denominator.
+// exp(sink[h]) is one more term of head h's denominator.  window: see first_visible (common.cuh).  v_dim: the size of
+// a value, a multiple of head_dim (out and v_new then have v_dim columns a head).
 // seq_index (optional, [num_seqs]): the batch rows to run, so that a mixed step can send its
 // single-token sequences through a split launch and the others through an unsplit one.
 // num_splits > 1 needs scratch: partial_out [tokens*heads*splits, head_dim] and partial_lse
-// [tokens*heads*splits] (float32, tokens = rows of q), and `counters`
+// [tokens*heads*splits] (float32, tokens = rows of q; heads times v_dim / head_dim), and `counters`
 // (li_paged_attention_mma_counters(...) unsigned values, zero; the kernel leaves them zero).
 // rope_inv_freq (optional, [head_dim / 2] float32; only with max_q_len 1 and groups of at most 16): the rotary
 // encoding and the cache write are done here instead of by li_rope_kv_write.  q, k_new and v_new then point at
@@ -478,14 +486,16 @@ LI_EXPORT int li_paged_attention_mma(const void* q, int q_row_stride, void* out,
                                      int head_dim, int page_size, int num_pages, float scale, int window,
                                      int num_splits, float* partial_out, float* partial_lse, unsigned* counters,
                                      const float* rope_inv_freq, const void* k_new, const void* v_new, int store_new,
-                                     int keep_first, float softcap, const float* sink, cudaStream_t stream) {
+                                     int keep_first, float softcap, const float* sink, int v_dim, cudaStream_t stream) {
   if (num_seqs == 0 || max_q_len == 0) return 0;
   if (rope_inv_freq && (keep_first > 0 || softcap > 0.f)) return LI_ERR_UNSUPPORTED;
   if (scale == 0.f) return LI_ERR_UNSUPPORTED;
   if (kv_heads < 1 || heads % kv_heads) return LI_ERR_UNSUPPORTED;
   const int groups = heads / kv_heads;
   if (groups > kBlockM || (head_dim != 64 && head_dim != 128)) return LI_ERR_UNSUPPORTED;
-  if (kv_heads > 65535 || num_seqs > 65535 || num_splits < 1 || num_splits > 32) return LI_ERR_UNSUPPORTED;
+  if (v_dim < head_dim || v_dim % head_dim) return LI_ERR_UNSUPPORTED;
+  const int v_parts = v_dim / head_dim;
+  if ((long)kv_heads * v_parts > 65535 || num_seqs > 65535 || num_splits < 1 || num_splits > 32) return LI_ERR_UNSUPPORTED;
   if (num_splits > 1 && (out_row_stride % 4)) return LI_ERR_ALIGNMENT;
   if (num_splits > 1 && (!partial_out || !partial_lse || !counters)) return LI_ERR_UNSUPPORTED;
   if ((q_row_stride % 8) || (out_row_stride % 2) || !aligned16(q) || !aligned16(k_pool) || !aligned16(v_pool))
@@ -501,6 +511,7 @@ LI_EXPORT int li_paged_attention_mma(const void* q, int q_row_stride, void* out,
   p.cap_in = softcap > 0.f ? scale / softcap : 0.f;
   p.cap_out = softcap > 0.f ? softcap / scale : 0.f;
   p.sink = sink;
+  p.v_parts = v_parts;
   const bool decode = max_q_len == 1 && groups <= 16;
   if (rope_inv_freq && (!decode || !k_new || !v_new || !aligned16(k_new) || !aligned16(v_new))) return LI_ERR_UNSUPPORTED;
   if (!decode)
@@ -513,7 +524,7 @@ LI_EXPORT int li_paged_attention_mma(const void* q, int q_row_stride, void* out,
     const char* e = getenv("LITEINFER_DECODE_STAGES");
     stages_override = e ? atoi(e) : 0;
   }
-  const long blocks = (long)num_seqs * kv_heads * num_splits;
+  const long blocks = (long)num_seqs * kv_heads * v_parts * num_splits;
   if (head_dim == 64) {
     int stages = blocks <= decode_capacity<64, 4>() ? 4 : (blocks <= decode_capacity<64, 3>() ? 3 : 2);
     if (stages_override) stages = stages_override;

@@ -25,7 +25,7 @@ struct AttnParams {
   int heads, kv_heads, page_size, num_pages;
   int page_shift;         // log2(page_size) when it is a power of two, else -1
   float scale_log2;       // scale * log2(e)
-  int window;
+  int window;             // see first_visible (common.cuh)
   int num_splits;
   float* partial_out;     // [tokens * heads * splits, D] when num_splits > 1
   float* partial_lse;     // [tokens * heads * splits]
@@ -47,7 +47,13 @@ struct AttnParams {
   // [heads] float or null: exp(sink[h]) is one more term of head h's denominator, with no key and no value.  It is
   // added where a row's final result is made (the unsplit epilogues, or the merge of the splits), exactly once.
   const float* sink;
+  // Values wider than keys: v_parts blocks side by side share a (sequence, KV head, split), each computing the scores
+  // and D of the v_parts * D dimensions of the output (blockIdx.y = KV head * v_parts + part).
+  int v_parts;
 };
+
+// Where a head's part of the output (and of the split partials) lies, in units of D.
+__device__ __forceinline__ int out_head(const AttnParams& p, int head, int part) { return head * p.v_parts + part; }
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem, bool valid) {
   const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
@@ -100,7 +106,8 @@ template <int D> __device__ __forceinline__ bf16* tile_ptr(bf16* base, int row, 
 // or with several splits this split's partial result and its log-sum-exp.
 template <int D>
 __device__ __forceinline__ void combine_warps(const AttnParams& p, const float* os, const float* ms, const float* ls,
-                                              int rows_used, int groups, int q_begin, int q0, int kvh, int split) {
+                                              int rows_used, int groups, int q_begin, int q0, int kvh, int part,
+                                              int split) {
   for (int e = threadIdx.x; e < rows_used * D; e += kWarps * 32) {
     const int row = e / D, d = e % D;
     float mx = -INFINITY;
@@ -118,9 +125,9 @@ __device__ __forceinline__ void combine_warps(const AttnParams& p, const float* 
     if (p.num_splits == 1 && p.sink != nullptr) denom += exp2f(p.sink[head] * kLog2e - mx);
     const float value = denom > 0.f ? acc / denom : 0.f;
     if (p.num_splits == 1) {
-      p.out[(size_t)(q_begin + qi) * p.out_row_stride + (size_t)head * D + d] = __float2bfloat16_rn(value);
+      p.out[(size_t)(q_begin + qi) * p.out_row_stride + (size_t)out_head(p, head, part) * D + d] = __float2bfloat16_rn(value);
     } else {
-      const size_t slot = ((size_t)(q_begin + qi) * p.heads + head) * p.num_splits + split;
+      const size_t slot = ((size_t)(q_begin + qi) * p.heads * p.v_parts + out_head(p, head, part)) * p.num_splits + split;
       p.partial_out[slot * D + d] = value;
       if (d == 0) p.partial_lse[slot] = denom > 0.f ? mx + log2f(denom) : -INFINITY;
     }
@@ -132,7 +139,8 @@ __device__ __forceinline__ void combine_warps(const AttnParams& p, const float* 
 // of every block of a split launch, after the block's partial result is written (`smem_raw` is not used any more).
 template <int D>
 __device__ __forceinline__ void merge_splits(const AttnParams& p, unsigned char* smem_raw, bool* is_last_flag,
-                                             int rows_used, int groups, int q_begin, int q0, int kvh, int qtile) {
+                                             int rows_used, int groups, int q_begin, int q0, int kvh, int v_part,
+                                             int qtile) {
   // ---- the block that arrives last merges the splits of this (sequence, KV head, query tile).
   __threadfence();
   __syncthreads();
@@ -158,7 +166,7 @@ __device__ __forceinline__ void merge_splits(const AttnParams& p, unsigned char*
     const int item = live ? e / P : 0, part = e % P;
     const int row = item / (D / 4), d4 = item % (D / 4);
     const int qi = q0 + row / groups, head = kvh * groups + row % groups;
-    const size_t first = ((size_t)(q_begin + qi) * p.heads + head) * S;
+    const size_t first = ((size_t)(q_begin + qi) * p.heads * p.v_parts + out_head(p, head, v_part)) * S;
     const float* lse = p.partial_lse + first;
     const float4* src = reinterpret_cast<const float4*>(p.partial_out + first * D) + d4;
     float mx = -INFINITY, denom = 0.f;
@@ -204,7 +212,7 @@ __device__ __forceinline__ void merge_splits(const AttnParams& p, unsigned char*
     if (live && part == 0) {
       if (p.sink != nullptr) denom += exp2f(p.sink[head] * kLog2e - mx);
       const float inv = denom > 0.f ? 1.f / denom : 0.f;
-      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (size_t)head * D + d4 * 4;
+      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (size_t)out_head(p, head, v_part) * D + d4 * 4;
       *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x * inv, acc.y * inv), pack_bf16(acc.z * inv, acc.w * inv));
     }
   }

@@ -68,7 +68,7 @@ __device__ __forceinline__ unsigned piece_addr(unsigned half_base, int row, int 
 // A function of its own, so that its registers are not the loop's.
 template <int D>
 __device__ __noinline__ void merge_in_cluster(const AttnParams& p, const float* os, const float* ms, float* ls, int groups,
-                                              int q_begin, int kvh, int split) {
+                                              int q_begin, int kvh, int v_part, int split) {
   // ---- the splits are one cluster (rank = split).  This block's result: mine [groups][D], normalised, and its
   // log-sum-exp per row, behind the warps' states in this block's own shared memory.
   float* mine = ls + kWarps * 16;                        // [16][D]
@@ -134,7 +134,7 @@ __device__ __noinline__ void merge_in_cluster(const AttnParams& p, const float* 
         if (s < S) {
           acc.x += w[s] * v[s].x; acc.y += w[s] * v[s].y; acc.z += w[s] * v[s].z; acc.w += w[s] * v[s].w;
         }
-      bf16* dst = p.out + (size_t)q_begin * p.out_row_stride + (size_t)(kvh * groups + row) * D + d4 * 4;
+      bf16* dst = p.out + (size_t)q_begin * p.out_row_stride + (size_t)out_head(p, kvh * groups + row, v_part) * D + d4 * 4;
       *reinterpret_cast<uint2*>(dst) = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
     }
   }
@@ -160,14 +160,14 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 
   const int seq = p.seq_index ? p.seq_index[blockIdx.z] : blockIdx.z;
   if (seq < 0) return;        // a place of padding in the list of sequences
-  const int kvh = blockIdx.y, split = blockIdx.x;
+  const int kvh = (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts, split = blockIdx.x;
   const int q_begin = p.query_start_loc[seq];
   const int groups = p.heads / p.kv_heads;
   const int ctx = p.context_lens[seq];
   const int* table = p.block_table + (size_t)seq * p.table_stride;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
   const int qpos = ctx - 1, hi = ctx;
-  const int lo = (p.window > 0 && qpos - p.window + 1 > 0) ? qpos - p.window + 1 : 0;
+  const int lo = first_visible(qpos, p.window);
   const int tile_lo = lo / kBlockN, tile_hi = (hi + kBlockN - 1) / kBlockN;
   const int per_split = (tile_hi - tile_lo + p.num_splits - 1) / p.num_splits;
   const int my_lo = tile_lo + split * per_split, my_hi = min(tile_hi, my_lo + per_split);
@@ -214,7 +214,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 #pragma unroll
     for (int b = 0; b < kBoxes; ++b) {
       tma_load_2d(slot + b * 2048, &map_k, bar, b * 64, (int)row);
-      tma_load_2d(slot + kHalfBytes + b * 2048, &map_v, bar, b * 64, (int)row);
+      tma_load_2d(slot + kHalfBytes + b * 2048, &map_v, bar, part * D + b * 64, (int)row);
     }
   };
   // The pages hold nothing that the kernel before this one wrote when the cache write is fused in here; otherwise
@@ -259,9 +259,9 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
       } else {
         const int j = (w - D / 16) * 8;
-        const Vec16<bf16> v = load16(p.v_new + token + (size_t)kvh * D + j);
+        const Vec16<bf16> v = load16(p.v_new + token + ((size_t)kvh * p.v_parts + part) * D + j);
         store16(newest + D + j, v);
-        if (store) store16(v_pool + dst + j, v);
+        if (store) store16(v_pool + dst * p.v_parts + (size_t)part * D + j, v);
       }
     }
     __syncthreads();
@@ -456,12 +456,12 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
   }
   __syncthreads();
   if (!kCluster) {
-    combine_warps<D>(p, os, ms, ls, groups, groups, q_begin, 0, kvh, split);
+    combine_warps<D>(p, os, ms, ls, groups, groups, q_begin, 0, kvh, part, split);
     if (p.num_splits == 1) return;
-    merge_splits<D>(p, generic_base, &is_last, groups, groups, q_begin, 0, kvh, 0);
+    merge_splits<D>(p, generic_base, &is_last, groups, groups, q_begin, 0, kvh, part, 0);
     return;
   }
-  merge_in_cluster<D>(p, os, ms, ls, groups, q_begin, kvh, split);
+  merge_in_cluster<D>(p, os, ms, ls, groups, q_begin, kvh, part, split);
 }
 
 // The rings, which at the end hold the warps' states ([4][16][D] floats and two of [4][16]) and, with a cluster's
@@ -472,7 +472,8 @@ template <int D, int kRing> constexpr size_t stream_smem() {
   return (rings > states ? rings : states) + 1024;
 }
 
-// The pool [pages, kv_heads, page_size, D] as a 2-D map of rows of D with boxes of 16 rows x 64 dimensions.
+// The pool [pages, kv_heads, page_size, row] as a 2-D map of rows (D of a key, v_parts * D of a value) with boxes of
+// 16 rows x 64 dimensions.
 static bool make_group_map(CUtensorMap* map, const void* pool, long rows, int head_dim) {
   static std::map<std::tuple<const void*, long, int>, CUtensorMap> cache;
   static std::mutex guard;                 // several host threads may launch (an asyncio engine beside its caller)
@@ -510,7 +511,7 @@ int launch_stream(const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  const dim3 grid(p.num_splits, p.kv_heads, num_seqs);
+  const dim3 grid(p.num_splits, p.kv_heads * p.v_parts, num_seqs);
   if (!p.cluster_merge)
     return (int)launch_pdl(num_seqs, attention_stream_kernel<D, kRing, false>, grid, dim3(kWarps * 32), stream_smem<D, kRing>(), stream, mk, mv, p);
   cudaLaunchConfig_t config = {};
@@ -605,7 +606,8 @@ LI_EXPORT int li_paged_attention_stream_capacity(int head_dim) {
 // Every launched sequence brings exactly one token.  Arguments as li_paged_attention_mma (its counters export
 // says how many counters a split launch needs); sizes as li_paged_attention_stream_supports allows.
 // error_flag (device int, zero; may be null): set to 21 if a wait for a group of keys ever gave up.
-// sink (optional, [heads] float32): exp(sink[h]) is one more term of head h's denominator.
+// sink (optional, [heads] float32): exp(sink[h]) is one more term of head h's denominator.  v_dim: the size of a value,
+// a multiple of head_dim.
 LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* out, int out_row_stride,
                                         const void* k_pool, const void* v_pool, const int* block_table,
                                         int table_stride, const int* query_start_loc, const int* context_lens,
@@ -613,10 +615,13 @@ LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* o
                                         int page_size, int num_pages, float scale, int window, int num_splits,
                                         float* partial_out, float* partial_lse, unsigned* counters,
                                         const float* rope_inv_freq, const void* k_new, const void* v_new,
-                                        int store_new, int* error_flag, const float* sink, cudaStream_t stream) {
+                                        int store_new, int* error_flag, const float* sink, int v_dim,
+                                        cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   if (!li_paged_attention_stream_supports(heads, kv_heads, head_dim, page_size)) return LI_ERR_UNSUPPORTED;
-  if (kv_heads > 65535 || num_seqs > 65535 || num_splits < 1 || num_splits > 32) return LI_ERR_UNSUPPORTED;
+  if (v_dim < head_dim || v_dim % head_dim) return LI_ERR_UNSUPPORTED;
+  const int v_parts = v_dim / head_dim;
+  if ((long)kv_heads * v_parts > 65535 || num_seqs > 65535 || num_splits < 1 || num_splits > 32) return LI_ERR_UNSUPPORTED;
   if (num_splits > 1 && (out_row_stride % 4)) return LI_ERR_ALIGNMENT;
   if (num_splits > 1 && (!partial_out || !partial_lse || !counters)) return LI_ERR_UNSUPPORTED;
   if ((q_row_stride % 8) || (out_row_stride % 2) || !aligned16(q) || !aligned16(k_pool) || !aligned16(v_pool))
@@ -625,7 +630,7 @@ LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* o
   const long rows = (long)num_pages * kv_heads * page_size;
   if (rows > 0x7fffffffL) return LI_ERR_UNSUPPORTED;
   CUtensorMap mk, mv;
-  if (!make_group_map(&mk, k_pool, rows, head_dim) || !make_group_map(&mv, v_pool, rows, head_dim))
+  if (!make_group_map(&mk, k_pool, rows, head_dim) || !make_group_map(&mv, v_pool, rows, v_dim))
     return LI_ERR_UNSUPPORTED;
   AttnParams p{(const bf16*)q, q_row_stride, (bf16*)out, out_row_stride, (const bf16*)k_pool, (const bf16*)v_pool,
                block_table, table_stride, query_start_loc, context_lens, seq_index, heads, kv_heads, page_size,
@@ -637,9 +642,10 @@ LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* o
   // while the one before it drains (programmatic dependent launch), a launch of clusters starts later than a
   // launch of single blocks does, and the step loses more than the merge gains (1.065 against 0.948 ms).
   const char* cluster_env = getenv("LITEINFER_ATTN_CLUSTER_MERGE");
+  p.v_parts = v_parts;
   p.sink = sink;      // added by the merges of attention_mma.cuh; the merge inside a cluster does not know it
   if (cluster_env && atoi(cluster_env) == 1 && sink == nullptr && num_splits >= 2 && num_splits <= 16 &&
-      li_paged_attention_stream_cluster_capacity(head_dim, num_splits) >= kv_heads * num_seqs)
+      li_paged_attention_stream_cluster_capacity(head_dim, num_splits) >= kv_heads * v_parts * num_seqs)
     p.cluster_merge = 1;
   if ((page_size & (page_size - 1)) == 0)
     for (int s = 0; s < 31; ++s)

@@ -162,7 +162,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int seq = p.seq_index ? p.seq_index[blockIdx.y] : blockIdx.y;
   if (seq < 0) return;        // a place of padding in the list of sequences
-  const int kvh = blockIdx.x;
+  // Values wider than keys: the blocks of a KV head's parts lie side by side, each with all scores and D of a value's
+  // dimensions.
+  const int parts = (int)gridDim.x / p.kv_heads, kvh = (int)blockIdx.x / parts, part = (int)blockIdx.x - kvh * parts;
   const int q_begin = p.query_start_loc[seq], q_len = p.query_start_loc[seq + 1] - q_begin;
   const int groups = p.heads / p.kv_heads;
   const int tq = kRows / groups;
@@ -174,7 +176,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   const int block_q = min(X * tq, q_len - block_q0);         // query tokens of the block: its tiles walk the same keys
   const int* table = p.block_table + (size_t)seq * p.table_stride;
   const int hi = ctx - q_len + block_q0 + block_q;
-  const int lo = (p.window > 0 && ctx - q_len + block_q0 - p.window + 1 > 0) ? ctx - q_len + block_q0 - p.window + 1 : 0;
+  const int lo = first_visible(ctx - q_len + block_q0, p.window);
   // The warp's own tile (issuer x is warp 1 + x, its softmax warps are 1 + X + 4 x ...): its queries and positions.
   const int x = X == 1 ? 0 : (warp <= X ? max(warp - 1, 0) : (warp - 1 - X) >> 2);
   const int q0 = block_q0 + x * tq;
@@ -248,7 +250,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
       for (int sub = 0; sub < kSub; ++sub) {
         tma_load_2d(k_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_k, kv_full(stage), sub * 64, row);
-        tma_load_2d(v_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_v, kv_full(stage), sub * 64, row);
+        tma_load_2d(v_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_v, kv_full(stage), part * D + sub * 64, row);
       }
     }
     return true;
@@ -350,6 +352,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     const int row = quarter * 32 + lane;
     const unsigned lane_field = (unsigned)(quarter * 32) << 16;
     const int qpos = row < rows_used ? first_qpos + row / groups : -1;
+    const int row_lo = first_visible(qpos, p.window), last_lo = first_visible(last_qpos, p.window);
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int t = 0; ok && t < ntiles; ++t) {
@@ -370,7 +373,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           sb[j] = __float_as_uint(p.cap_out * tanh_fast(__uint_as_float(sb[j]) * p.cap_in));
         }
       }
-      const bool all_visible = key0 + kKeys - 1 <= first_qpos && (p.window <= 0 || key0 > last_qpos - p.window);
+      const bool all_visible = key0 + kKeys - 1 <= first_qpos && key0 >= last_lo;
       float mx = m;
       if (all_visible && qpos >= 0) {
         float part[4] = {m, m, m, m};      // four chains, so that the maxima do not wait for one another
@@ -381,8 +384,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           const int ka = key0 + j, kb = key0 + 32 + j;
-          const bool va = ka <= qpos && (p.window <= 0 || ka > qpos - p.window || (kOptions && ka < p.keep_first));
-          const bool vb = kb <= qpos && (p.window <= 0 || kb > qpos - p.window || (kOptions && kb < p.keep_first));
+          const bool va = ka <= qpos && (ka >= row_lo || (kOptions && ka < p.keep_first));
+          const bool vb = kb <= qpos && (kb >= row_lo || (kOptions && kb < p.keep_first));
           if (!va) sa[j] = __float_as_uint(-INFINITY);
           if (!vb) sb[j] = __float_as_uint(-INFINITY);
           mx = fmaxf(mx, fmaxf(__uint_as_float(sa[j]), __uint_as_float(sb[j])));
@@ -458,7 +461,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
       // (Compiled into the kernel's form with options only, so that the plain form is what it was.)
       if (kOptions && p.sink != nullptr && row < rows_used) l += exp2f(p.sink[head] * kLog2eF - m * p.scale_log2);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (size_t)head * D;
+      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + ((size_t)head * parts + part) * D;
 #pragma unroll
       for (int half = 0; half < D / 32; ++half) {
         unsigned o[32];
@@ -490,8 +493,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   }
 }
 
-// The pool [pages, kv_heads, page_size, head_dim] as a 2-D map of rows of head_dim; a box is 64 dimensions of one
-// page of one head.
+// The pool [pages, kv_heads, page_size, row] as a 2-D map of rows (of `head_dim` numbers: a key's or a value's); a box is
+// 64 dimensions of one page of one head.
 static bool make_pool_map(CUtensorMap* map, const void* pool, long rows, int page_size, int head_dim) {
   static std::map<std::tuple<const void*, long, int, int>, CUtensorMap> cache;
   static std::mutex guard;                 // several host threads may launch (an asyncio engine beside its caller)
@@ -557,24 +560,27 @@ LI_EXPORT int li_paged_attention_tcgen05_supports(int heads, int kv_heads, int h
 }
 
 // bfloat16; head_dim 64 or 128; page_size 16, 32 or 64; groups of at most 128 heads.  Sequences may bring any number of queries
-// (the kernel is meant for those that bring many).  error_flag (device int, zero): set if a wait inside gave up.
+// (the kernel is meant for those that bring many).  window: see first_visible (common.cuh).  v_dim: the size of a value, a
+// multiple of head_dim.  error_flag (device int, zero): set if a wait inside gave up.
 LI_EXPORT int li_paged_attention_tcgen05(const void* q, int q_row_stride, void* out, int out_row_stride,
                                          const void* k_pool, const void* v_pool, const int* block_table,
                                          int table_stride, const int* query_start_loc, const int* context_lens,
                                          const int* seq_index, int num_seqs, int max_q_len, int heads, int kv_heads,
                                          int head_dim, int page_size, int num_pages, float scale, int window,
                                          int* error_flag, int keep_first, float softcap, const float* sink,
-                                         cudaStream_t stream) {
+                                         int v_dim, cudaStream_t stream) {
   if (num_seqs == 0 || max_q_len == 0) return 0;
   if (softcap > 0.f && scale == 0.f) return LI_ERR_UNSUPPORTED;
   if (!li_paged_attention_tcgen05_supports(heads, kv_heads, head_dim, page_size)) return LI_ERR_UNSUPPORTED;
+  if (v_dim < head_dim || v_dim % head_dim) return LI_ERR_UNSUPPORTED;
+  const int v_parts = v_dim / head_dim;
   if (num_seqs > 65535 || (max_q_len + 0L) * heads / kv_heads / kRows >= 65535) return LI_ERR_UNSUPPORTED;
   if ((q_row_stride % 8) || (out_row_stride % 8) || !aligned16(q) || !aligned16(out) || !aligned16(k_pool) ||
       !aligned16(v_pool))
     return LI_ERR_ALIGNMENT;
   CUtensorMap mk, mv;
   const long rows = (long)num_pages * kv_heads * page_size;
-  if (!make_pool_map(&mk, k_pool, rows, page_size, head_dim) || !make_pool_map(&mv, v_pool, rows, page_size, head_dim))
+  if (!make_pool_map(&mk, k_pool, rows, page_size, head_dim) || !make_pool_map(&mv, v_pool, rows, page_size, v_dim))
     return LI_ERR_UNSUPPORTED;
   int shift = 0;
   while ((1 << shift) < page_size) ++shift;
@@ -588,8 +594,8 @@ LI_EXPORT int li_paged_attention_tcgen05(const void* q, int q_row_stride, void* 
   // (LITEINFER_TCGEN05_ATTN_TILES=1 keeps one).
   static const bool one_tile = [] { const char* e = getenv("LITEINFER_TCGEN05_ATTN_TILES"); return e && atoi(e) == 1; }();
   if (head_dim == 128 && max_q_len > tq && !one_tile)
-    return launch_tc_attention<128, 2>(mk, mv, p, dim3(kv_heads, num_seqs, (max_q_len + 2 * tq - 1) / (2 * tq)), stream);
-  const dim3 grid(kv_heads, num_seqs, (max_q_len + tq - 1) / tq);
+    return launch_tc_attention<128, 2>(mk, mv, p, dim3(kv_heads * v_parts, num_seqs, (max_q_len + 2 * tq - 1) / (2 * tq)), stream);
+  const dim3 grid(kv_heads * v_parts, num_seqs, (max_q_len + tq - 1) / tq);
   return head_dim == 64 ? launch_tc_attention<64, 1>(mk, mv, p, grid, stream)
                         : launch_tc_attention<128, 1>(mk, mv, p, grid, stream);
 }

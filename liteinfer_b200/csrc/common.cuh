@@ -190,6 +190,15 @@ inline cudaError_t launch_pdl(long rows, void (*kernel)(KernelArgs...), dim3 gri
   return cudaLaunchKernelEx(&config, kernel, KernelArgs(args)...);
 }
 
+// ---- which keys a query sees ------------------------------------------------------------------------
+// The first key that the query at `pos` may read (it reads no later key than itself).  span > 0: a sliding window,
+// the newest `span` keys; span < 0: chunks of -span positions counted from the sequence's start, the keys of its own
+// chunk; 0: every key.  It never falls as pos grows, so a run of queries starts at its first query's.
+__device__ __forceinline__ int first_visible(int pos, int span) {
+  if (span > 0) return pos - span + 1 > 0 ? pos - span + 1 : 0;
+  return span < 0 && pos > 0 ? pos - pos % -span : 0;
+}
+
 __host__ __device__ inline bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
 
 }  // namespace li

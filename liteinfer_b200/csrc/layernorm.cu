@@ -9,8 +9,8 @@
 //   li_projection_rmsnorm  x = w * x / sqrt(mean(x^2) + eps) in place over whole rows of one or two neighbouring
 //                          column slices (q and k of a fused projection, each normalised across all its heads)
 //   li_gated_rmsnorm       out = w * x / sqrt(mean(x^2) + eps) * act(gate) per head; one warp a (token, head);
-//                          act = silu or sigmoid; w shared by the heads or one per head; x optionally divided by
-//                          a number per (token, head) first
+//                          act = silu or sigmoid, or no gate at all; w shared by the heads or one per head; x
+//                          optionally divided by a number per (token, head) first; out may be a column slice
 //
 // x of li_layernorm may be float while value, weights and out are bfloat16: the stream stays 32-bit, what the
 // products read is rounded once.  Means, variances, the sum into the stream and every product before the final
@@ -222,12 +222,12 @@ projection_rmsnorm_kernel(T* __restrict__ x, size_t stride, int width_a, const T
   for (int c = threadIdx.x; c < width; c += blockDim.x) p[c] = from_float<T>(to_float(p[c]) * inv * to_float(w[c]));
 }
 
-// weight_stride: 0 = one weight vector for every head, `size` = one per head.  act: 0 silu, 1 sigmoid.  den (may
-// be null): x[t, h] is divided by den[t * heads + h] before anything else.
+// weight_stride: 0 = one weight vector for every head, `size` = one per head.  act: 0 silu, 1 sigmoid, 2 no gate (gate
+// is null).  den (may be null): x[t, h] is divided by den[t * heads + h] before anything else.
 template <typename T>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __restrict__ gate, size_t gate_stride,
-                                     const float* __restrict__ weight, T* __restrict__ out, int tokens, int heads,
-                                     int size, float eps, int weight_stride, int act, const float* __restrict__ den) {
+                                     const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int tokens,
+                                     int heads, int size, float eps, int weight_stride, int act, const float* __restrict__ den) {
   grid_dependency_wait();
   const int lane = threadIdx.x & 31;
   const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);   // (token, head)
@@ -244,12 +244,16 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __res
   const float inv = 1.0f / sqrtf(warp_sum(q) / (float)size + eps);
   const T* g = gate + t * gate_stride + (size_t)h * size;
   const float* w = weight + (size_t)h * weight_stride;
-  T* o = out + (t * heads + h) * size;
+  T* o = out + t * out_stride + (size_t)h * size;
   for (int c = lane; c < size; c += 32) {
-    const float z = to_float(g[c]);
-    const float s = 1.0f / (1.0f + expf(-z));
     const float v = den != nullptr ? xr[c] / under : xr[c];
-    o[c] = from_float<T>(v * inv * w[c] * (act == 1 ? s : z * s));
+    float by = 1.0f;
+    if (act != 2) {
+      const float z = to_float(g[c]);
+      const float s = 1.0f / (1.0f + expf(-z));
+      by = act == 1 ? s : z * s;
+    }
+    o[c] = from_float<T>(v * inv * w[c] * by);
   }
 }
 
@@ -258,8 +262,8 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __res
 // bfloat16) aligned.
 template <typename T, int NV>
 __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* __restrict__ gate, size_t gate_stride,
-                                         const float* __restrict__ weight, T* __restrict__ out, int tokens, int heads,
-                                         int size, float eps, int weight_stride, int act,
+                                         const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int tokens,
+                                         int heads, int size, float eps, int weight_stride, int act,
                                          const float* __restrict__ den) {
   const int lane = threadIdx.x & 31;
   const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);   // (token, head)
@@ -282,7 +286,7 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
     v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (lane + 32 * j < quads) {
       v[j] = *reinterpret_cast<const float4*>(xr + 4 * (lane + 32 * j));
-      load4(g + 4 * (lane + 32 * j), z[j]);
+      if (act != 2) load4(g + 4 * (lane + 32 * j), z[j]);
     }
   }
   if (den != nullptr) {
@@ -294,7 +298,7 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
 #pragma unroll
   for (int j = 0; j < NV; ++j) q += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
   const float inv = 1.0f / sqrtf(warp_sum(q) / (float)size + eps);
-  T* o = out + (t * heads + h) * size;
+  T* o = out + t * out_stride + (size_t)h * size;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     if (lane + 32 * j >= quads) continue;
@@ -302,8 +306,12 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
     float r[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const float s = 1.0f / (1.0f + expf(-z[j][e]));
-      r[e] = xs[e] * inv * ws[e] * (act == 1 ? s : z[j][e] * s);
+      float by = 1.0f;
+      if (act != 2) {
+        const float s = 1.0f / (1.0f + expf(-z[j][e]));
+        by = act == 1 ? s : z[j][e] * s;
+      }
+      r[e] = xs[e] * inv * ws[e] * by;
     }
     store4(o + 4 * (lane + 32 * j), r);
   }
@@ -404,10 +412,11 @@ LI_EXPORT int li_projection_rmsnorm(int dtype, void* x, size_t stride, int rows,
 }
 
 LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size_t gate_stride, const float* weight,
-                               void* out, int tokens, int heads, int size, float eps, int weight_per_head, int act,
+                               void* out, size_t out_stride, int tokens, int heads, int size, float eps,
+                               int weight_per_head, int act,
                                const float* den, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (heads < 1 || size < 1 || act < 0 || act > 1) return LI_ERR_UNSUPPORTED;
+  if (heads < 1 || size < 1 || act < 0 || act > 2 || (act == 2) != (gate == nullptr)) return LI_ERR_UNSUPPORTED;
   const size_t items = (size_t)tokens * heads;
   const int warps = 8;
   const int weight_stride = weight_per_head ? size : 0;
@@ -415,12 +424,12 @@ LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size
   // Heads of up to 512 whose rows 16-byte accesses can walk keep their row in registers.
   const size_t gate_unit = dtype == kFloat32 ? 4 : 2;
   const bool wide = size % 4 == 0 && size <= 512 && aligned16(x) && aligned16(weight) && aligned16(out) &&
-                    ((uintptr_t)gate * 1) % (4 * gate_unit) == 0 && gate_stride % 4 == 0;
+                    (uintptr_t)gate % (4 * gate_unit) == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0;
   if (wide) {
     const int nv = size <= 128 ? 1 : size <= 256 ? 2 : 4;
 #define LI_GATED(T, NV)                                                                                                \
   return (int)launch_pdl(tokens, gated_rmsnorm_vec_kernel<T, NV>, grid, dim3(warps * 32), 0, stream, x,               \
-                         (const T*)gate, gate_stride, weight, (T*)out, tokens, heads, size, eps, weight_stride, act,   \
+                         (const T*)gate, gate_stride, weight, (T*)out, out_stride, tokens, heads, size, eps, weight_stride, act, \
                          den)
     if (dtype == kFloat32) {
       if (nv == 1) LI_GATED(float, 1);
@@ -434,7 +443,7 @@ LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size
   }
   if (dtype == kFloat32)
     return (int)launch_pdl(tokens, gated_rmsnorm_kernel<float>, grid, dim3(warps * 32), 0, stream, x, (const float*)gate,
-                           gate_stride, weight, (float*)out, tokens, heads, size, eps, weight_stride, act, den);
+                           gate_stride, weight, (float*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den);
   return (int)launch_pdl(tokens, gated_rmsnorm_kernel<bf16>, grid, dim3(warps * 32), 0, stream, x, (const bf16*)gate,
-                         gate_stride, weight, (bf16*)out, tokens, heads, size, eps, weight_stride, act, den);
+                         gate_stride, weight, (bf16*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den);
 }

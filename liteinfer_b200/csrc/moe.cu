@@ -1,9 +1,11 @@
 // A mixture of experts: routing, and the experts' products grouped by expert.
 //
-//   li_moe_route     per token: scores = softmax over all experts of the router's logits (32-bit); where the experts
-//                    form `groups` equal groups of neighbours, a group's score is its largest score and only experts
-//                    of the best `keep` groups can be chosen; the `top` largest scores among those are chosen (ties
-//                    go to the lower index); the weights are the chosen scores, or those divided by their sum.
+//   li_moe_route     per token: scores = softmax over all experts of the router's logits (32-bit), or the sigmoid of each;
+//                    the choice scores are those plus a correction per expert, if there is one; where the experts form
+//                    `groups` equal groups of neighbours, a group's score is its largest choice score (or the sum of
+//                    its two largest) and only experts of the best `keep` groups can be chosen; the `top` largest choice
+//                    scores among those are chosen (ties go to the lower index); the weights are the chosen experts'
+//                    scores (without the correction), or those divided by their sum.
 //   li_moe_sort      the (token, slot) pairs ordered by expert, each expert's run cut into tiles of `tile_rows` rows:
 //                    order[], offsets[experts + 1], and per tile its expert and first row (-1: no such tile).
 //   li_moe_grouped   out[pair] = f(W_e x[row of the pair]) for every pair of expert e, tile by tile, so that an
@@ -34,10 +36,10 @@ __device__ __forceinline__ float expert_activation(float g, float u, int act, fl
 }
 
 // ------------------------------------------------------------------------------------------ route
-// The index of the largest of v[0..n) (ties: the lowest index); every lane gets it.  Entries are scores >= 0 or marks
-// of -1 and -2; whatever they hold, the result is an index below n (a row of padding may bring anything).
+// The index of the largest of v[0..n) (ties: the lowest index); every lane gets it.  A mark of -inf is never larger than
+// anything; whatever the entries hold, the result is an index below n (a row of padding may bring anything).
 __device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
-  float best = -3.0f;
+  float best = -INFINITY;
   int at = 0x7fffffff;
   for (int i = lane; i < n; i += 32)
     if (v[i] > best) { best = v[i]; at = i; }
@@ -52,87 +54,121 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
 
 constexpr int kRouteWarps = 4;
 
-// One warp routes one token: z [experts] its logits; sc [experts] and gb [groups] scratch in shared memory (sc may be z).
-__device__ __forceinline__ void route_token(const float* z, float* sc, float* gb, int lane, int t, int experts, int top,
-                                            int groups, int keep, int renormalise, int* __restrict__ ids,
-                                            float* __restrict__ weights) {
-  float mx = -INFINITY;
-  for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < experts; e += 32) {
-    const float v = expf(z[e] - mx);
-    sc[e] = v;
-    sum += v;
+// How a router turns its logits into chosen experts and weights.
+struct RouteRule {
+  int experts, top, groups, keep, renormalise;
+  int sigmoid;                // scores: 0 softmax over all experts, 1 the sigmoid of each logit
+  int pair_rank;              // a group's score: 0 its largest choice score, 1 the sum of its two largest
+  int slots;                  // entries of ids and weights a token has (>= top; the first `top` are the chosen experts)
+  float floor;                // added to the sum the weights are divided by
+  const float* correction;    // [experts] or null
+};
+
+__host__ __device__ __forceinline__ int route_floats(int experts, int groups) { return 2 * experts + 2 * groups; }
+
+// One warp routes one token: z [experts] its logits; scratch of `route_floats` floats in shared memory, whose first
+// `experts` places may be z itself.
+__device__ __forceinline__ void route_token(const float* z, float* scratch, int lane, int t, const RouteRule& rule,
+                                            int* __restrict__ ids, float* __restrict__ weights) {
+  const int experts = rule.experts, groups = rule.groups;
+  float* sc = scratch;                  // scores
+  float* choice = sc + experts;         // what the choice goes by; -inf: cannot be chosen (any more)
+  float* gb = choice + experts;         // the groups' scores
+  float* kept = gb + groups;            // 1: the group is kept
+  if (rule.sigmoid) {
+    for (int e = lane; e < experts; e += 32) sc[e] = 1.0f / (1.0f + expf(-z[e]));
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < experts; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < experts; e += 32) {
+      const float v = expf(z[e] - mx);
+      sc[e] = v;
+      sum += v;
+    }
+    const float inv = 1.0f / warp_sum(sum);
+    for (int e = lane; e < experts; e += 32) sc[e] = sc[e] * inv;
   }
-  const float inv = 1.0f / warp_sum(sum);
   for (int e = lane; e < experts; e += 32) {
-    const float score = sc[e] * inv;
-    sc[e] = score >= 0.f ? score : 0.f;       // a row of padding may hold anything, NaN too: its choice stays an expert
+    const float score = sc[e] >= 0.f ? sc[e] : 0.f;   // a row of padding may hold anything, NaN too: its choice stays an expert
+    sc[e] = score;
+    choice[e] = rule.correction != nullptr ? score + rule.correction[e] : score;
   }
   __syncwarp();
   if (groups > 1) {
     const int per = experts / groups;
     for (int g = lane; g < groups; g += 32) {
-      float best = 0.f;
-      for (int j = 0; j < per; ++j) best = fmaxf(best, sc[g * per + j]);
-      gb[g] = best;
+      float best = -INFINITY, second = -INFINITY;
+      for (int j = 0; j < per; ++j) {
+        const float v = choice[g * per + j];
+        second = fmaxf(second, fminf(best, v));
+        best = fmaxf(best, v);
+      }
+      gb[g] = rule.pair_rank && per > 1 ? best + second : best;
+      kept[g] = 0.f;
     }
     __syncwarp();
-    for (int r = 0; r < keep; ++r) {          // a kept group is marked by -2 (scores are never negative)
+    for (int r = 0; r < rule.keep; ++r) {
       const int g = warp_argmax(gb, groups, lane);
       __syncwarp();
-      if (lane == 0) gb[g] = -2.0f;
+      if (lane == 0) { gb[g] = -INFINITY; kept[g] = 1.f; }
       __syncwarp();
     }
     for (int e = lane; e < experts; e += 32)
-      if (gb[e / per] != -2.0f) sc[e] = -1.0f;
+      if (kept[e / per] == 0.f) choice[e] = -INFINITY;
     __syncwarp();
   }
   float total = 0.f;
-  for (int r = 0; r < top; ++r) {
-    const int e = warp_argmax(sc, experts, lane);
+  for (int r = 0; r < rule.top; ++r) {
+    const int e = warp_argmax(choice, experts, lane);
     const float w = sc[e];
     total += w;
     __syncwarp();
     if (lane == 0) {
-      ids[(size_t)t * top + r] = e;
-      weights[(size_t)t * top + r] = w;
-      sc[e] = -1.0f;
+      ids[(size_t)t * rule.slots + r] = e;
+      weights[(size_t)t * rule.slots + r] = w;
+      choice[e] = -INFINITY;
     }
     __syncwarp();
   }
-  if (renormalise && lane < top) weights[(size_t)t * top + lane] /= total;     // (top <= 32 where this is asked for)
+  if (rule.renormalise && lane < rule.top)     // (top <= 32 where this is asked for)
+    weights[(size_t)t * rule.slots + lane] /= total + rule.floor;
 }
 
 __global__ void __launch_bounds__(kRouteWarps * 32)
-moe_route_kernel(const float* __restrict__ logits, int tokens, int experts, int top, int groups, int keep,
-                 int renormalise, int* __restrict__ ids, float* __restrict__ weights) {
-  extern __shared__ float route_smem[];       // per warp: scores[experts], group scores[groups]
+moe_route_kernel(const float* __restrict__ logits, int tokens, const RouteRule rule, int* __restrict__ ids,
+                 float* __restrict__ weights) {
+  extern __shared__ float route_smem[];       // per warp: `route_floats`
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * kRouteWarps + warp;
   grid_dependency_wait();
   if (t >= tokens) return;
-  float* sc = route_smem + warp * (experts + groups);
-  route_token(logits + (size_t)t * experts, sc, sc + experts, lane, t, experts, top, groups, keep, renormalise, ids,
-              weights);
+  route_token(logits + (size_t)t * rule.experts, route_smem + warp * route_floats(rule.experts, rule.groups), lane, t, rule,
+              ids, weights);
 }
 
 // The router's product and the routing in one launch: logits[e] = sum_k x[k] * w[e][k] in 32-bit (lane l adds up
 // k = l, l + 32, ..., then the lanes' sums meet in a fixed tree: the same bits whatever else is in the step), then
 // `route_token`.  A block takes TOK tokens; its warps take the experts in turn: eight warps for eight tokens of a wide
 // step, thirty-two for the one token of a narrow step, where a warp's chain of loads is what the launch waits for.
+//
+// `gated`: w has one more row, whose logit's sigmoid is a number per token for an expert that every token runs.  It goes
+// to gate[token] (where given) and is the weight of the slots behind the chosen experts, which hold the experts
+// `experts`, `experts` + 1, ...
 template <typename T, int TOK, int kRouterWarps>
 __global__ void __launch_bounds__(kRouterWarps * 32)
-moe_router_kernel(const T* __restrict__ x, size_t x_stride, const float* __restrict__ w, int tokens, int K, int experts,
-                  int top, int groups, int keep, int renormalise, int* __restrict__ ids, float* __restrict__ weights) {
-  extern __shared__ float route_smem[];       // TOK x (logits[experts], group scores[groups])
+moe_router_kernel(const T* __restrict__ x, size_t x_stride, const float* __restrict__ w, int tokens, int K,
+                  const RouteRule rule, int gated, int* __restrict__ ids, float* __restrict__ weights,
+                  float* __restrict__ gate) {
+  extern __shared__ float route_smem[];       // TOK x (`route_floats`, of which the first are the logits, and the gate's)
+  const int per_token = route_floats(rule.experts, rule.groups) + 1, experts = rule.experts;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t0 = blockIdx.x * TOK;
   grid_dependency_wait();
   // Four k a lane and round where the rows allow 16-byte reads (several rounds' loads are in flight at once), else one.
   const bool wide = (K % 4) == 0 && (x_stride % 4) == 0 && aligned16(w) && (reinterpret_cast<uintptr_t>(x) % (4 * sizeof(T))) == 0;
-  for (int e = warp; e < experts; e += kRouterWarps) {
+  for (int e = warp; e < experts + gated; e += kRouterWarps) {
     const float* we = w + (size_t)e * K;
     float acc[TOK];
 #pragma unroll
@@ -168,13 +204,22 @@ moe_router_kernel(const T* __restrict__ x, size_t x_stride, const float* __restr
 #pragma unroll
     for (int t = 0; t < TOK; ++t) {
       const float sum = warp_sum(acc[t]);
-      if (lane == 0) route_smem[t * (experts + groups) + e] = sum;
+      if (lane == 0) route_smem[t * per_token + (e < experts ? e : per_token - 1)] = sum;
     }
   }
   __syncthreads();
   if (warp < TOK && t0 + warp < tokens) {
-    float* sc = route_smem + warp * (experts + groups);
-    route_token(sc, sc, sc + experts, lane, t0 + warp, experts, top, groups, keep, renormalise, ids, weights);
+    float* sc = route_smem + warp * per_token;
+    const int t = t0 + warp;
+    route_token(sc, sc, lane, t, rule, ids, weights);
+    if (gated) {
+      const float g = 1.0f / (1.0f + expf(-sc[per_token - 1]));
+      if (lane == 0 && gate != nullptr) gate[t] = g;
+      for (int r = rule.top + lane; r < rule.slots; r += 32) {
+        ids[(size_t)t * rule.slots + r] = experts + r - rule.top;
+        weights[(size_t)t * rule.slots + r] = g;
+      }
+    }
   }
 }
 
@@ -486,17 +531,23 @@ static int launch_mma(const void* a, size_t a_stride, const void* w, void* out, 
 
 using namespace li;
 
-// logits [tokens, experts] float; ids [tokens, top] int; weights [tokens, top] float.
+static bool bad_rule(const RouteRule& r) {
+  return r.experts < 1 || r.top < 1 || r.top > r.experts || r.groups < 1 || r.experts % r.groups || r.keep < 1 ||
+         r.keep > r.groups || r.keep * (r.experts / r.groups) < r.top || (r.renormalise && r.top > 32) || r.slots < r.top;
+}
+
+// logits [tokens, experts] float; ids [tokens, top] int; weights [tokens, top] float.  sigmoid, pair_rank, floor,
+// correction: see RouteRule.
 LI_EXPORT int li_moe_route(const float* logits, int tokens, int experts, int top, int groups, int keep,
-                           int renormalise, int* ids, float* weights, cudaStream_t stream) {
+                           int renormalise, int sigmoid, int pair_rank, float floor, const float* correction, int* ids,
+                           float* weights, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  if (experts < 1 || top < 1 || top > experts || groups < 1 || experts % groups || keep < 1 || keep > groups)
-    return LI_ERR_UNSUPPORTED;
-  if (keep * (experts / groups) < top || (renormalise && top > 32)) return LI_ERR_UNSUPPORTED;
-  const size_t smem = (size_t)kRouteWarps * (experts + groups) * sizeof(float);
+  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top, floor, correction};
+  if (bad_rule(rule)) return LI_ERR_UNSUPPORTED;
+  const size_t smem = (size_t)kRouteWarps * route_floats(experts, groups) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
   return (int)launch_pdl(tokens, moe_route_kernel, dim3((tokens + kRouteWarps - 1) / kRouteWarps), dim3(kRouteWarps * 32),
-                         smem, stream, logits, tokens, experts, top, groups, keep, renormalise, ids, weights);
+                         smem, stream, logits, tokens, rule, ids, weights);
 }
 
 // Rows of a tile of the grouped product that li_moe_grouped will run for this dtype and these sizes.
@@ -518,21 +569,21 @@ LI_EXPORT int li_moe_sort(const int* ids, int pairs, int experts, int tile_rows,
 }
 
 // x [tokens, K] (rows x_stride apart) in the engine's dtype, w [experts, K] float: the router's product and the routing
-// of li_moe_route in one launch.
+// of li_moe_route in one launch.  gated: w has a row more (see moe_router_kernel); ids and weights are [tokens, top +
+// extra], gate [tokens] float or null.
 LI_EXPORT int li_moe_router(int dtype, const void* x, size_t x_stride, const float* w, int tokens, int K, int experts,
-                            int top, int groups, int keep, int renormalise, int* ids, float* weights,
+                            int top, int groups, int keep, int renormalise, int sigmoid, int pair_rank, float floor,
+                            const float* correction, int gated, int extra, int* ids, float* weights, float* gate,
                             cudaStream_t stream) {
   if (tokens == 0) return 0;
-  if (experts < 1 || top < 1 || top > experts || groups < 1 || experts % groups || keep < 1 || keep > groups || K < 1)
-    return LI_ERR_UNSUPPORTED;
-  if (keep * (experts / groups) < top || (renormalise && top > 32)) return LI_ERR_UNSUPPORTED;
+  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top + extra, floor, correction};
+  if (K < 1 || extra < 0 || (extra > 0 && !gated) || bad_rule(rule)) return LI_ERR_UNSUPPORTED;
   const bool wide = tokens > 128;
-  const size_t smem = (size_t)(wide ? 8 : 1) * (experts + groups) * sizeof(float);
+  const size_t smem = (size_t)(wide ? 8 : 1) * (route_floats(experts, groups) + 1) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
 #define LI_ROUTER(T, TOK, WARPS)                                                                                      \
   return (int)launch_pdl(tokens, moe_router_kernel<T, TOK, WARPS>, dim3((tokens + TOK - 1) / TOK), dim3(WARPS * 32),   \
-                         smem, stream, (const T*)x, x_stride, w, tokens, K, experts, top, groups, keep, renormalise,  \
-                         ids, weights)
+                         smem, stream, (const T*)x, x_stride, w, tokens, K, rule, gated ? 1 : 0, ids, weights, gate)
   if (dtype == kFloat32) { if (wide) LI_ROUTER(float, 8, 8); LI_ROUTER(float, 1, 32); }
   if (wide) LI_ROUTER(bf16, 8, 8);
   LI_ROUTER(bf16, 1, 32);

@@ -53,12 +53,21 @@ _SIGNATURES = {
                                                   c_size_t, c_void_p, c_int, c_float, c_void_p]),
     "li_sigmoid_gate": ("rope_cache", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_void_p]),
     "li_softcap": ("elementwise", [c_int, c_void_p, c_size_t, c_float, c_void_p]),
-    "li_moe_route": ("moe", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p]),
+    "li_moe_route": ("moe", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
+                             c_void_p, c_void_p]),
     "li_moe_tile_rows": ("moe", [c_int, c_int, c_int]),
     "li_moe_sort": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
                             c_void_p]),
     "li_moe_router": ("moe", [c_int, c_void_p, c_size_t, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                              c_void_p, c_void_p, c_void_p]),
+                              c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
+    "li_hgrn2_steps": ("hgrn2", [c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "li_hgrn2_token": ("hgrn2", [c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_int, c_void_p, c_float, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p]),
+    "li_hgrn2_record_floats": ("hgrn2", [c_int, c_int]),
+    "li_sum_norms": ("sum_norms", [c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
+                                   c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                                   c_float, c_int, c_void_p]),
     "li_moe_gather": ("moe", [c_int, c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]),
     "li_gemm_tcgen05_grouped": ("gemm_tcgen05", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                                  c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
@@ -79,7 +88,7 @@ _SIGNATURES = {
                                    c_int, c_int, c_float, c_float, c_int, c_int, c_void_p]),
     "li_projection_rmsnorm": ("layernorm", [c_int, c_void_p, c_size_t, c_int, c_int, c_void_p, c_int, c_void_p,
                                             c_float, c_void_p]),
-    "li_gated_rmsnorm": ("layernorm", [c_int, c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_int, c_int, c_int,
+    "li_gated_rmsnorm": ("layernorm", [c_int, c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_size_t, c_int, c_int, c_int,
                                        c_float, c_int, c_int, c_void_p, c_void_p]),
     "li_short_conv": ("delta_rule", [c_int, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                      c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
@@ -91,11 +100,11 @@ _SIGNATURES = {
     "li_paged_attention_mma": ("attention_mma", [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_void_p]),
+        c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p]),
     "li_paged_attention_stream": ("attention_stream", [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p]),
+        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p]),
     "li_paged_attention_stream_supports": ("attention_stream", [c_int, c_int, c_int, c_int]),
     "li_paged_attention_stream_capacity": ("attention_stream", [c_int]),
     "li_paged_attention_stream_cluster_capacity": ("attention_stream", [c_int, c_int]),
@@ -103,7 +112,8 @@ _SIGNATURES = {
     "li_paged_attention_mma_decode_capacity": ("attention_mma", [c_int]),
     "li_paged_attention_tcgen05": ("attention_tcgen05", [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p]),
+        c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_void_p, c_int,
+        c_void_p]),
     "li_paged_attention_tcgen05_supports": ("attention_tcgen05", [c_int, c_int, c_int, c_int]),
     "li_gemm_skinny": ("gemm_skinny", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                        c_void_p, c_size_t, c_void_p, c_int, c_void_p]),
@@ -829,9 +839,11 @@ def cluster_capacity(head_dim: int, splits: int) -> int:
 def paged_attention_generic(q, q_row_stride, out, k_pool, v_pool, block_table, query_start_loc, context_lens,
                             num_seqs, max_q_len, heads, kv_heads, head_dim, scale, window=0, keep_first=0,
                             softcap=0.0, sink=None) -> torch.Tensor:
-    """The plain SIMT kernel: any dtype, key and value sizes up to 256 (they may differ), any grouping, a window
-    that may keep the first `keep_first` keys visible, scores capped by softcap * tanh(score / softcap), a sink."""
-    _on_gpu(q, out, k_pool, v_pool, block_table, query_start_loc, context_lens, sink)
+    """The plain SIMT kernel: any dtype, key and value sizes up to 1,024 (they may differ), any grouping, a window
+    that may keep the first `keep_first` keys visible (`window` < 0: chunks of -window positions instead), scores
+    capped by softcap * tanh(score / softcap), a sink."""
+    _rows2d(q, "q"); _rows2d(out, "out")
+    _on_gpu(k_pool, v_pool, block_table, query_start_loc, context_lens, sink)
     pages, kvh, page_size, hd = k_pool.shape
     _check(_fn("li_paged_attention_generic")(
         _code(q), q.data_ptr(), q_row_stride, out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(),
@@ -852,15 +864,19 @@ def paged_attention_mma(q, q_row_stride, out, k_pool, v_pool, block_table, query
     rotates q and the key and stores key and value itself.  `streaming` (single-token sequences, sizes that
     `stream_attention_supports` allows): the kernel that passes K and V through registers only.  `keep_first`
     (with a window) and `softcap`: as in `paged_attention`; not with `newest` or `streaming`.  `sink`: as in
-    `paged_attention`; every form takes it."""
-    _on_gpu(q, out, k_pool, v_pool, block_table, query_start_loc, context_lens, seq_index, sink)
+    `paged_attention`; every form takes it.  `window` < 0: chunks of -window positions.  Values may be a multiple of
+    the head size wide."""
+    _rows2d(q, "q"); _rows2d(out, "out")
+    _on_gpu(k_pool, v_pool, block_table, query_start_loc, context_lens, seq_index, sink)
     pages, kvh, page_size, hd = k_pool.shape
+    v_dim = v_pool.shape[3]
+    parts = v_dim // head_dim
     partial_out = partial_lse = counters = None
     if num_splits > 1:
-        total = q.shape[0] * heads * num_splits
+        total = q.shape[0] * heads * parts * num_splits
         partial_out = torch.empty((total, head_dim), dtype=torch.float32, device=q.device)
         partial_lse = torch.empty((total,), dtype=torch.float32, device=q.device)
-        need = int(_fn("li_paged_attention_mma_counters")(num_seqs, max_q_len, heads, kv_heads))
+        need = int(_fn("li_paged_attention_mma_counters")(num_seqs, max_q_len, heads, kv_heads)) * parts
         counters = scratch_for(q.device).attention_counters
         if need > counters.numel():
             counters = torch.zeros(need, dtype=torch.int32, device=q.device)
@@ -873,14 +889,14 @@ def paged_attention_mma(q, q_row_stride, out, k_pool, v_pool, block_table, query
             block_table.data_ptr(), block_table.stride(0), query_start_loc.data_ptr(), context_lens.data_ptr(),
             _ptr(seq_index), num_seqs, heads, kv_heads, head_dim, page_size, pages, float(scale), int(window),
             int(num_splits), _ptr(partial_out), _ptr(partial_lse), _ptr(counters), *tail,
-            scratch_for(q.device).gemm_error.data_ptr(), _ptr(sink), _stream()), "paged_attention_stream")
+            scratch_for(q.device).gemm_error.data_ptr(), _ptr(sink), v_dim, _stream()), "paged_attention_stream")
         return out
     _check(_fn("li_paged_attention_mma")(
         q.data_ptr(), q_row_stride, out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(),
         block_table.data_ptr(), block_table.stride(0), query_start_loc.data_ptr(), context_lens.data_ptr(),
         _ptr(seq_index), num_seqs, max_q_len, heads, kv_heads, head_dim, page_size, pages, float(scale),
         int(window), int(num_splits), _ptr(partial_out), _ptr(partial_lse), _ptr(counters), *tail, int(keep_first),
-        float(softcap), _ptr(sink), _stream()),
+        float(softcap), _ptr(sink), v_dim, _stream()),
         "paged_attention_mma")
     return out
 
@@ -906,16 +922,18 @@ def paged_attention_tcgen05(q, q_row_stride, out, k_pool, v_pool, block_table, q
                             seq_index, num_seqs, max_q_len, heads, kv_heads, head_dim, scale, window=0, keep_first=0,
                             softcap=0.0, sink=None) -> torch.Tensor:
     """The tcgen05 / TMA / tensor-memory attention kernel for prompts and portions (bfloat16, head size 64 or 128,
-    pages of 16, 32 or 64 tokens, groups of at most 128 heads; `keep_first` and `softcap` as in `paged_attention`).
+    pages of 16, 32 or 64 tokens, groups of at most 128 heads; `keep_first` and `softcap` as in `paged_attention`;
+    `window` < 0: chunks of -window positions; values may be a multiple of the head size wide).
     `gemm_error_flag(device)` tells afterwards whether a wait inside the kernel ever gave up."""
-    _on_gpu(q, out, k_pool, v_pool, block_table, query_start_loc, context_lens, seq_index, sink)
+    _rows2d(q, "q"); _rows2d(out, "out")
+    _on_gpu(k_pool, v_pool, block_table, query_start_loc, context_lens, seq_index, sink)
     pages, kvh, page_size, hd = k_pool.shape
     _check(_fn("li_paged_attention_tcgen05")(
         q.data_ptr(), q_row_stride, out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(),
         block_table.data_ptr(), block_table.stride(0), query_start_loc.data_ptr(), context_lens.data_ptr(),
         _ptr(seq_index), num_seqs, max_q_len, heads, kv_heads, head_dim, page_size, pages, float(scale),
         int(window), scratch_for(q.device).gemm_error.data_ptr(), int(keep_first), float(softcap), _ptr(sink),
-        _stream()),
+        v_pool.shape[3], _stream()),
         "paged_attention_tcgen05")
     return out
 
@@ -936,6 +954,18 @@ def mma_attention_supports(dtype: torch.dtype, heads: int, kv_heads: int, head_d
     return dtype == torch.bfloat16 and head_dim in (64, 128) and heads // kv_heads <= 64
 
 
+def tensor_core_sizes(key_dim: int, value_dim: int, heads: int, kv_heads: int) -> tuple[int, int] | None:
+    """The sizes of keys and values to which heads of these sizes are rounded up so that the tensor-core kernels take
+    them: a head size of 64 or 128, values a multiple of it (each multiple computes the scores again).  None: no size
+    does.  What is weighed is a key's work: its dimensions times the multiples, plus the values'."""
+    found = []
+    for size in (64, 128):
+        if key_dim <= size and mma_attention_supports(torch.bfloat16, heads, kv_heads, size):
+            parts = -(-value_dim // size)
+            found.append((parts * size + parts * size, parts, (size, parts * size)))
+    return min(found)[2] if found else None
+
+
 # LITEINFER_TCGEN05_ATTN=0: prompts and portions run on the mma.sync kernel (a switch for measurements).
 MASKED_ON_MMA = os.environ.get("LITEINFER_TCGEN05_ATTN", "1") == "0"
 
@@ -945,7 +975,7 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
                     context_lens: torch.Tensor, num_seqs: int, max_q_len: int, heads: int, kv_heads: int,
                     head_dim: int, scale: float, window: int = 0, plan=None,
                     decode_splits: int | None = None, newest: "NewestToken | None" = None, keep_first: int = 0,
-                    softcap: float = 0.0, sink: torch.Tensor | None = None) -> torch.Tensor:
+                    softcap: float = 0.0, sink: torch.Tensor | None = None, chunk: int = 0) -> torch.Tensor:
     """Attention of each sequence's newest queries over its pages (any mix of portions and single tokens).
 
     q: the tensor holding the queries, head h of token t at q[t, h*head_dim:...]
@@ -958,9 +988,12 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
     `keep_first` (with a window): the first keys of a sequence stay visible behind the window.  `softcap` > 0:
     a scaled score s becomes softcap * tanh(s / softcap).  Values may have another size than keys
     (`v_pool.shape[3]`); out is then [tokens, heads * value size].  `sink` [heads] float32: exp(sink[h]) is one
-    more term of the denominator of head h's softmax; it has no key and no value and is not scaled.
+    more term of the denominator of head h's softmax; it has no key and no value and is not scaled.  `chunk` > 0
+    (instead of a window): positions form chunks of that many from the sequence's start, and a query reads the keys of
+    its own chunk up to itself.  q and out may be column slices of wider tensors.
     """
-    _on_gpu(q, out, k_pool, v_pool, block_table, query_start_loc, context_lens)
+    _rows2d(q, "q"); _rows2d(out, "out")
+    _on_gpu(k_pool, v_pool, block_table, query_start_loc, context_lens)
     _int32(block_table, "block_table"); _int32(query_start_loc, "query_start_loc"); _int32(context_lens, "context_lens")
     pages, kvh, page_size, hd = k_pool.shape
     assert (kvh, hd) == (kv_heads, head_dim) and q.dtype == out.dtype == k_pool.dtype == v_pool.dtype
@@ -968,7 +1001,11 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
         raise ValueError("the decode kernel with the rotary encoding fused in does not take this step")
     masked = softcap > 0 or (keep_first > 0 and window > 0)
     assert sink is None or (sink.dtype == torch.float32 and sink.numel() == heads)
-    if v_pool.shape[3] != head_dim or not mma_attention_supports(q.dtype, heads, kv_heads, head_dim):
+    assert chunk <= 0 or window <= 0, "an attention has a window or chunks"
+    reach = max(window, 0) + keep_first if window > 0 else max(chunk, 0)      # keys a query reads at most (0: all)
+    window = -chunk if chunk > 0 else max(window, 0)
+    parts = v_pool.shape[3] // head_dim
+    if v_pool.shape[3] != parts * head_dim or parts < 1 or not mma_attention_supports(q.dtype, heads, kv_heads, head_dim):
         assert newest is None
         return paged_attention_generic(q, q_row_stride, out, k_pool, v_pool, block_table, query_start_loc,
                                        context_lens, num_seqs, max_q_len, heads, kv_heads, head_dim, scale, window,
@@ -990,9 +1027,9 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
             paged_attention_mma(*common, plan.prefill_seqs, plan.num_prefill, plan.max_prefill_query_len, heads,
                                 kv_heads, head_dim, scale, window, **options)
     if plan.num_decode:
-        bound = plan.max_decode_context_len if window <= 0 else min(plan.max_decode_context_len, window + keep_first)
+        bound = min(plan.max_decode_context_len, reach) if reach else plan.max_decode_context_len
         streaming = not masked and stream_attention_supports(q.dtype, heads, kv_heads, head_dim, page_size)
-        splits = decode_splits or decode_splits_for(plan.num_decode, kv_heads, bound, head_dim, streaming)
+        splits = decode_splits or decode_splits_for(plan.num_decode, kv_heads * parts, bound, head_dim, streaming)
         paged_attention_mma(*common, plan.decode_seqs, plan.num_decode, 1, heads, kv_heads, head_dim, scale,
                             window, splits, newest, streaming, **options)
     return out
@@ -1097,25 +1134,30 @@ def qk_projection_rmsnorm_(q: torch.Tensor, q_weight: torch.Tensor, k: torch.Ten
            "projection_rmsnorm")
 
 
-def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor,
+def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tensor, eps: float, out: torch.Tensor,
                   heads: int, gate_activation: str = "silu", den: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, h] = weight * x[t, h] / sqrt(mean(x[t, h]^2) + eps) * act(gate[t, h]) per head.  x: float32
     [tokens, heads * size]; weight: float32, `size` entries shared by the heads or `heads * size`, one vector
-    per head; gate (a column slice is fine) and out in the engine's dtype.  `gate_activation`: "silu" or
-    "sigmoid".  `den` [tokens, heads] float32: x[t, h] is divided by den[t, h] first."""
-    _on_gpu(x, weight, out, den)
-    _rows2d(gate, "gate")
+    per head; gate and out in the engine's dtype (column slices are fine).  `gate_activation`: "silu" or
+    "sigmoid"; without a gate (None) the norm alone.  `den` [tokens, heads] float32: x[t, h] is divided by den[t, h]
+    first."""
+    _on_gpu(x, weight, den)
+    _rows2d(out, "out")
     tokens, width = out.shape
     size = width // heads
-    assert x.dtype == torch.float32 and x.shape == out.shape == gate.shape and width == heads * size
-    assert gate.dtype == out.dtype and weight.dtype == torch.float32 and weight.numel() in (size, width)
+    assert x.dtype == torch.float32 and x.shape == out.shape and width == heads * size
+    assert weight.dtype == torch.float32 and weight.numel() in (size, width)
+    if gate is not None:
+        _rows2d(gate, "gate")
+        assert gate.shape == out.shape and gate.dtype == out.dtype
     assert den is None or (den.dtype == torch.float32 and den.numel() == tokens * heads)
     if gate_activation not in ("silu", "sigmoid"):
         raise KernelLibraryError(f"gated_rmsnorm knows the gates 'silu' and 'sigmoid', not {gate_activation!r}")
-    _check(_fn("li_gated_rmsnorm")(_code(out), x.data_ptr(), gate.data_ptr(), gate.stride(0), weight.data_ptr(),
-                                   out.data_ptr(), tokens, heads, size, float(eps),
-                                   int(weight.numel() == width and heads > 1), int(gate_activation == "sigmoid"),
-                                   _ptr(den), _stream()), "gated_rmsnorm")
+    act = 2 if gate is None else int(gate_activation == "sigmoid")
+    _check(_fn("li_gated_rmsnorm")(_code(out), x.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0,
+                                   weight.data_ptr(), out.data_ptr(), out.stride(0), tokens, heads, size, float(eps),
+                                   int(weight.numel() == width and heads > 1), act, _ptr(den), _stream()),
+           "gated_rmsnorm")
     return out
 
 
@@ -1241,6 +1283,119 @@ def mlstm(proj: torch.Tensor, offsets: tuple[int, int, int, int, int], i_bias: t
                            query_start_loc.data_ptr(), state_slots.data_ptr(), tokens, num_seqs, out.data_ptr(),
                            den.data_ptr(), heads, dim, vdim, int(max_query_len), _stream()), "mlstm")
     return out
+
+
+def hgrn2(proj: torch.Tensor, offsets: tuple[int, int, int], f_bias: torch.Tensor, lower: torch.Tensor,
+          state: torch.Tensor, query_start_loc: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, heads: int,
+          dim: int, vdim: int, norm_weight: torch.Tensor, eps: float, out: torch.Tensor,
+          max_query_len: int = 0) -> torch.Tensor:
+    """The memory of an HGRN2 layer, token by token, on a 32-bit state per request and head, and the norm of its read-out.
+
+    proj [tokens, width] (a column slice is fine) holds, per token, at the columns `offsets` = (q, f, v), the raw q and f
+    (heads of dim) and v (heads of vdim).  Per head and channel q' = silu(q), f' = lower + (1 - lower) sigmoid(f + f_bias)
+    (float32 [heads * dim] both);  S <- diag(f') S + (1 - f') v^T;  o = S^T q';
+    out[t, h] = o / sqrt(mean(o^2) + eps) * norm_weight (float32 [vdim]).  out [tokens, heads * vdim] in the engine's
+    dtype (a column slice is fine).  state [slots, heads, vdim, dim] float32 (S kept column by column) is read and
+    written.  `max_query_len`: the most tokens a sequence brings, if known (1: everything is one kernel)."""
+    global launch_count
+    _rows2d(proj, "proj"); _rows2d(out, "out")
+    _on_gpu(f_bias, lower, state, query_start_loc, state_slots, norm_weight)
+    _int32(query_start_loc, "query_start_loc"); _int32(state_slots, "state_slots")
+    tokens, width = proj.shape
+    q_off, f_off, v_off = offsets
+    assert max(q_off, f_off) + heads * dim <= width and v_off + heads * vdim <= width and out.dtype == proj.dtype
+    assert f_bias.dtype == lower.dtype == state.dtype == norm_weight.dtype == torch.float32
+    assert f_bias.numel() == lower.numel() == heads * dim and norm_weight.numel() == vdim
+    assert state.shape[1:] == (heads, vdim, dim) and out.shape == (tokens, heads * vdim)
+    if max_query_len == 1:
+        _check(_fn("li_hgrn2_token")(_code(proj), proj.data_ptr(), proj.stride(0), q_off, f_off, v_off,
+                                     f_bias.data_ptr(), lower.data_ptr(), state.data_ptr(), query_start_loc.data_ptr(),
+                                     state_slots.data_ptr(), num_seqs, norm_weight.data_ptr(), float(eps),
+                                     out.data_ptr(), out.stride(0), heads, dim, vdim, _stream()), "hgrn2_token")
+        return out
+    per_record = int(_fn("li_hgrn2_record_floats")(dim, vdim))
+    records = torch.empty(max(tokens, 1) * heads * per_record, dtype=torch.float32, device=proj.device)
+    read = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=proj.device)
+    _check(_fn("li_hgrn2_steps")(_code(proj), proj.data_ptr(), proj.stride(0), q_off, f_off, v_off, f_bias.data_ptr(),
+                                 lower.data_ptr(), records.data_ptr(), state.data_ptr(), query_start_loc.data_ptr(),
+                                 state_slots.data_ptr(), tokens, num_seqs, read.data_ptr(), heads, dim, vdim, _stream()),
+           "hgrn2_steps")
+    launch_count += 1       # two kernels
+    return gated_rmsnorm(read, None, norm_weight, eps, out, heads)
+
+
+# ------------------------------------------------- a stream that takes several sublayers' outputs at once
+@dataclass
+class RoutedRows:
+    """The rows of the experts that every token runs, already multiplied by their weights and not yet added up: those of
+    token t are value[place[t * top + s]] for s < top (place None: value[t * top + s])."""
+
+    value: torch.Tensor                 # [tokens * top, width]
+    top: int
+    place: torch.Tensor | None = None   # int32
+
+
+@dataclass
+class SumTerm:
+    """factor * value, each row also times row_factor[row] (float32 [tokens]) where that is given."""
+
+    value: torch.Tensor
+    factor: float = 1.0
+    row_factor: torch.Tensor | None = None
+
+
+@dataclass
+class SumDelta:
+    """A delta of the residual stream that has not been added up yet: up to two dense terms and the rows of experts.
+    The norm that reads the stream next (`sum_norms`) does the sum on its way."""
+
+    terms: tuple[SumTerm, ...] = ()
+    routed: RoutedRows | None = None
+
+    def __add__(self, other: "SumDelta") -> "SumDelta":
+        if self.routed is not None and other.routed is not None or len(self.terms) + len(other.terms) > 2:
+            raise ValueError("a pending sum holds two dense terms and one set of experts' rows at most")
+        return SumDelta(self.terms + other.terms, self.routed if self.routed is not None else other.routed)
+
+
+def sum_norms(x: torch.Tensor | None, delta: SumDelta, weights: tuple[torch.Tensor, ...], eps: float,
+              outs: tuple[torch.Tensor, ...], rows: torch.Tensor | None = None, write_stream: bool = False) -> None:
+    """v = x[row] + the sum of `delta`, row = rows[r] if given else r;  outs[i][r] = v / sqrt(mean(v^2) + eps) *
+    weights[i], for at most two norms (none: only the sum is made, with `write_stream`).  x [tokens, width] float32; with
+    `write_stream` v is stored back.  x None: outs[0] is the sum itself.  weights float32 [width]; outs in the terms'
+    dtype; everything in between is 32-bit."""
+    routed = delta.routed
+    terms = list(delta.terms)
+    values = [t.value for t in terms] + ([routed.value] if routed is not None else [])
+    _on_gpu(x, rows, *weights, *outs, *values, *(t.row_factor for t in terms),
+            routed.place if routed is not None else None)
+    _int32(rows, "rows")
+    dtype = values[0].dtype if values else outs[0].dtype
+    width = x.shape[1] if x is not None else outs[0].shape[1]
+    tokens = x.shape[0] if x is not None else outs[0].shape[0]
+    n = outs[0].shape[0] if outs else tokens
+    assert len(terms) <= 2 and len(outs) <= 2 and (x is not None or (len(outs) == 1 and not weights and rows is None))
+    assert x is None or (x.dtype == torch.float32 and len(weights) == len(outs) and (outs or write_stream))
+    assert not (write_stream and rows is not None) and (n == tokens if rows is None else rows.numel() == n)
+    for t in terms:
+        assert t.value.shape == (tokens, width) and t.value.dtype == dtype
+        assert t.row_factor is None or (t.row_factor.dtype == torch.float32 and t.row_factor.numel() == tokens)
+    if routed is not None:
+        assert routed.value.shape == (tokens * routed.top, width) and routed.value.dtype == dtype
+        _int32(routed.place, "place")
+    for w in weights:
+        assert w.dtype == torch.float32 and w.numel() == width
+    for o in outs:
+        assert o.dtype == dtype and o.shape == (n, width)
+    terms += [None] * (2 - len(terms))
+    dense = []
+    for t in terms:
+        dense += [None, 0.0, None] if t is None else [t.value.data_ptr(), float(t.factor), _ptr(t.row_factor)]
+    _check(_fn("li_sum_norms")(
+        _DTYPE_CODE[dtype], _ptr(x), *dense, _ptr(routed.value if routed else None), _ptr(routed.place if routed else None),
+        routed.top if routed else 0, _ptr(weights[0] if weights else None), _ptr(weights[1] if len(weights) > 1 else None),
+        _ptr(outs[0] if outs else None), _ptr(outs[1] if len(outs) > 1 else None), _ptr(rows), n, width, float(eps),
+        int(write_stream), _stream()), "sum_norms")
 
 
 # ------------------------------------------- several residual streams, latent attention
@@ -1477,36 +1632,52 @@ class ExpertPlan:
     place: torch.Tensor | None = None   # [pairs] int32: where in `order` each pair stands
 
 
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
 def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, renormalise: bool, ids: torch.Tensor,
-              weights: torch.Tensor) -> None:
-    """Per token of `logits` [tokens, experts] (float32): scores = softmax over all experts; with `groups` > 1 the
-    experts form that many equal groups of neighbours, a group's score is its largest, and only experts of the best
-    `keep` groups can be chosen; ids [tokens, top] int32 = the experts with the largest scores (ties: the lower
-    index), weights [tokens, top] float32 = their scores (`renormalise`: divided by their sum)."""
-    _on_gpu(logits, ids, weights)
+              weights: torch.Tensor, scores: str = "softmax", correction: torch.Tensor | None = None,
+              rank_by: int = 1, floor: float = 0.0) -> None:
+    """Per token of `logits` [tokens, experts] (float32): scores = softmax over all experts ("sigmoid": the sigmoid of
+    each logit); the choice scores are scores + `correction` (float32 [experts], None: none); with `groups` > 1 the
+    experts form that many equal groups of neighbours, a group's score is its largest choice score (`rank_by` 2: the
+    sum of its two largest), and only experts of the best `keep` groups can be chosen; ids [tokens, top] int32 = the
+    experts with the largest choice scores (ties: the lower index), weights [tokens, top] float32 = their scores
+    (`renormalise`: divided by their sum + `floor`)."""
+    _on_gpu(logits, ids, weights, correction)
     _int32(ids, "ids")
     tokens, experts = logits.shape
-    assert logits.dtype == torch.float32 == weights.dtype and logits.is_contiguous()
+    assert logits.dtype == torch.float32 == weights.dtype and logits.is_contiguous() and rank_by in (1, 2)
     assert ids.shape == weights.shape == (tokens, top) and ids.is_contiguous() and weights.is_contiguous()
-    _check(_fn("li_moe_route")(logits.data_ptr(), tokens, experts, top, groups, keep, int(renormalise), ids.data_ptr(),
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    _check(_fn("li_moe_route")(logits.data_ptr(), tokens, experts, top, groups, keep, int(renormalise),
+                               ROUTER_SCORES[scores], rank_by - 1, float(floor), _ptr(correction), ids.data_ptr(),
                                weights.data_ptr(), _stream()), "moe_route")
 
 
 def moe_router(x: torch.Tensor, weight: torch.Tensor, top: int, groups: int, keep: int, renormalise: bool,
-               ids: torch.Tensor, weights: torch.Tensor) -> None:
+               ids: torch.Tensor, weights: torch.Tensor, scores: str = "softmax", correction: torch.Tensor | None = None,
+               rank_by: int = 1, floor: float = 0.0, gated: bool = False, gate: torch.Tensor | None = None) -> None:
     """`moe_route` of the logits x @ weight^T, product and routing in one launch: x [tokens, hidden] in the engine's
     dtype (a column slice is fine), weight [experts, hidden] float32; the product is 32-bit, its sums in an order that
-    depends on nothing but the sizes."""
-    _on_gpu(weight, ids, weights)
+    depends on nothing but the sizes.  `gated`: weight has one more row, and the sigmoid of its logit, one number per
+    token, goes to `gate` [tokens] float32 (None: nowhere) and is the weight of the slots that ids and weights have
+    behind the first `top`; those hold the experts number `experts`, `experts` + 1, ... (experts that every token runs)."""
+    _on_gpu(weight, ids, weights, correction, gate)
     _rows2d(x, "x")
     _int32(ids, "ids")
     tokens, hidden = x.shape
-    experts = weight.shape[0]
-    assert weight.dtype == torch.float32 == weights.dtype and weight.shape == (experts, hidden)
-    assert ids.shape == weights.shape == (tokens, top) and ids.is_contiguous() and weights.is_contiguous()
+    experts = weight.shape[0] - int(gated)
+    extra = ids.shape[1] - top
+    assert weight.dtype == torch.float32 == weights.dtype and weight.shape[1] == hidden and rank_by in (1, 2)
+    assert ids.shape == weights.shape == (tokens, top + extra) and ids.is_contiguous() and weights.is_contiguous()
+    assert extra >= 0 and (gated or (extra == 0 and gate is None))
+    assert correction is None or (correction.dtype == torch.float32 and correction.numel() == experts)
+    assert gate is None or (gate.dtype == torch.float32 and gate.numel() == tokens)
     _check(_fn("li_moe_router")(_code(x), x.data_ptr(), x.stride(0), weight.data_ptr(), tokens, hidden, experts, top,
-                                groups, keep, int(renormalise), ids.data_ptr(), weights.data_ptr(), _stream()),
-           "moe_router")
+                                groups, keep, int(renormalise), ROUTER_SCORES[scores], rank_by - 1, float(floor),
+                                _ptr(correction), int(gated), extra, ids.data_ptr(), weights.data_ptr(), _ptr(gate),
+                                _stream()), "moe_router")
 
 
 # LITEINFER_MOE_TCGEN05: 1 (default) = bfloat16 experts of steps with at least LITEINFER_MOE_TCGEN05_MIN_PAIRS (1) pairs of
@@ -1614,12 +1785,12 @@ def moe_combine(y: torch.Tensor, out: torch.Tensor, top: int, place: torch.Tenso
     return out
 
 
-def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                activation: str, limit: float, alpha: float, eights: bool, out: torch.Tensor) -> torch.Tensor:
-    """out[t] = sum_s weights[t, s] * down_e(act(gate_e x[t], up_e x[t])), e = ids[t, s]: the chosen experts of every
-    token, their products grouped by expert.  gate_up [experts, 2 * ff, hidden] (`eights`: gate and up rows interleaved
-    in eights), down [experts, hidden, ff].  Steps of many pairs in bfloat16 run the tcgen05 kernel over the pairs'
-    rows gathered expert by expert; the others the mma.sync or FFMA tiles, which gather as they load."""
+def moe_expert_rows(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
+                    activation: str, limit: float, alpha: float, eights: bool) -> RoutedRows:
+    """weights[t, s] * down_e(act(gate_e x[t], up_e x[t])), e = ids[t, s], for every pair (t, s): the chosen experts'
+    rows, their products grouped by expert, not yet added up.  gate_up [experts, 2 * ff, hidden] (`eights`: gate and up
+    rows interleaved in eights), down [experts, hidden, ff].  Steps of many pairs in bfloat16 run the tcgen05 kernel
+    over the pairs' rows gathered expert by expert; the others the mma.sync or FFMA tiles, which gather as they load."""
     tokens, top = ids.shape
     experts, hidden, ff = down.shape
     pairs = tokens * top
@@ -1632,10 +1803,17 @@ def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids:
         rows = moe_gather(x, plan, top, torch.empty((pairs, hidden), dtype=x.dtype, device=x.device))
         moe_grouped_tcgen05("gate_up", rows, gate_up, act, plan, activation, limit, alpha)
         moe_grouped_tcgen05("down", act, down, each, plan, pair_weights=scale)
-        return moe_combine(each, out, top, place=plan.place)
+        return RoutedRows(each, top, plan.place)
     moe_grouped("gate_up", x, gate_up, act, plan, top, activation, limit, alpha, eights=eights)
     moe_grouped("down", act, down, each, plan, top, pair_weights=scale)
-    return moe_combine(each, out, top)
+    return RoutedRows(each, top)
+
+
+def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
+                activation: str, limit: float, alpha: float, eights: bool, out: torch.Tensor) -> torch.Tensor:
+    """out[t] = sum_s weights[t, s] * down_e(act(gate_e x[t], up_e x[t])), e = ids[t, s] (`moe_expert_rows`, added up)."""
+    rows = moe_expert_rows(x, gate_up, down, ids, weights, activation, limit, alpha, eights)
+    return moe_combine(rows.value, out, rows.top, place=rows.place)
 
 
 # ------------------------------------------------------------------ sampling

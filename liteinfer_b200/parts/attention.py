@@ -42,8 +42,16 @@ class Attention:
     `head_gate`: head h of the attention's output is multiplied by sigmoid(g_h), g = `g_proj.weight` x, one number
     per head, before the output projection.  `value_mix`: "source" leaves this layer's values of the step's tokens
     in `ctx.extras[value_mix_key]` for later layers; "mixed" stores (1 - l) v + l v_source instead of v, l the
-    scalar tensor `value_mix` and v_source what the source layer left for the same tokens.  Everything that reads
-    x is one product against the concatenated weights.
+    scalar tensor `value_mix` and v_source what the source layer left for the same tokens.  `chunk` (instead of a
+    window): positions form chunks of that many from the sequence's start, and a query reads the keys of its own chunk
+    only.  Everything that reads x is one product against the concatenated weights.
+
+    `pad_heads`: in bfloat16 on a GPU, keys and values whose sizes no tensor-core kernel takes are rounded up to sizes
+    that one does (`tensor_core_sizes`): the added rows of the projections and columns of `o_proj.weight` are zeros, so
+    every score and every output is the same sum.  (Not with q/k norms, biases, mixed values or an output gate.)
+
+    A mixer that runs several side by side (parts/side_by_side.py) makes one product of their projections and one of
+    their output projections; it uses `in_weight`, `out_weight` and `mix`.
     """
 
     def __init__(self, hidden_size: int, heads: int, kv_heads: int, head_dim: int, position: PartSpec,
@@ -52,7 +60,10 @@ class Attention:
                  v_head_dim: int | None = None, keep_first: int = 0, softcap: float = 0.0,
                  qk_norm: str | None = None, qk_norm_eps: float = 1e-6, head_gate: bool = False,
                  value_mix: str | None = None, value_mix_key: str = "value_mix", qk_norm_weight: bool = True,
-                 qk_norm_after_rotation: bool = False, sink: bool = False, output_gate: bool = False) -> None:
+                 qk_norm_after_rotation: bool = False, sink: bool = False, output_gate: bool = False,
+                 chunk: int | None = None, pad_heads: bool = False) -> None:
+        if window is not None and chunk is not None:
+            raise ValueError("an attention has a window or chunks, not both")
         if heads % kv_heads:
             raise ValueError(f"heads={heads} is not a multiple of kv_heads={kv_heads}")
         if qk_norm not in (None, "projection", "head"):
@@ -76,23 +87,30 @@ class Attention:
         self.q_norm_weight = self.k_norm_weight = None
         self.bias = bias
         self.out_bias = bias if out_bias is None else out_bias
-        self.window = window
+        self.window, self.chunk = window, chunk
         self.cache_name = cache_name    # under which name this mixer's pages lie in its layer's cache
         self.scale = float(scale) if scale is not None else head_dim ** -0.5
         self.dtype, self.device = dtype, device
         self.position = build_part("position", position, dtype=dtype, device=device)
+        # The sizes of the checkpoint's heads; head_dim and v_head_dim are those of the rows that are computed and kept.
+        self.key_size, self.value_size = self.head_dim, self.v_head_dim
+        if (pad_heads and dtype == torch.bfloat16 and torch.device(device).type == "cuda"
+                and not (qk_norm or bias or value_mix or output_gate)):
+            sizes = ops.tensor_core_sizes(self.head_dim, self.v_head_dim, heads, kv_heads)
+            if sizes is not None:
+                self.head_dim, self.v_head_dim = sizes
         self.qkv_weight: torch.Tensor | None = None
         self.qkv_bias: torch.Tensor | None = None
         self.o_weight: torch.Tensor | None = None
         self.o_bias: torch.Tensor | None = None
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
-        q, kv, v = self.heads * self.head_dim, self.kv_heads * self.head_dim, self.kv_heads * self.v_head_dim
+        q, kv, v = self.heads * self.key_size, self.kv_heads * self.key_size, self.kv_heads * self.value_size
         specs = {
             "q_proj.weight": TensorSpec((q, self.hidden_size)),
             "k_proj.weight": TensorSpec((kv, self.hidden_size)),
             "v_proj.weight": TensorSpec((v, self.hidden_size)),
-            "o_proj.weight": TensorSpec((self.hidden_size, self.heads * self.v_head_dim)),
+            "o_proj.weight": TensorSpec((self.hidden_size, self.heads * self.value_size)),
         }
         if self.qk_norm == "head":
             if self.qk_norm_weight:
@@ -104,7 +122,7 @@ class Attention:
         if self.head_gate:
             specs["g_proj.weight"] = TensorSpec((self.heads, self.hidden_size))
         if self.output_gate:
-            specs["gate_proj.weight"] = TensorSpec((self.heads * self.v_head_dim, self.hidden_size))
+            specs["gate_proj.weight"] = TensorSpec((self.heads * self.value_size, self.hidden_size))
         if self.has_sink:
             specs["sink"] = TensorSpec((self.heads,), kind="f32", init=_sink_init)
         if self.value_mix == "mixed":
@@ -126,10 +144,16 @@ class Attention:
             # The checkpoint pairs neighbouring dimensions: every head's rows of q and k (and what belongs to those
             # dimensions) are brought into the order whose pairs are half a rotary width apart.
             at = torch.tensor(order, device=weights[0].device)
-            per_head = lambda t: t.unflatten(0, (-1, self.head_dim))[:, at].flatten(0, 1)
+            per_head = lambda t: t.unflatten(0, (-1, self.key_size))[:, at].flatten(0, 1)
             weights[0], weights[1] = per_head(weights[0]), per_head(weights[1])
             if self.bias:
                 biases[0], biases[1] = per_head(biases[0]), per_head(biases[1])
+        o_weight = tensors["o_proj.weight"]
+        if (self.head_dim, self.v_head_dim) != (self.key_size, self.value_size):
+            weights = [_padded_heads(w, old, new) for w, old, new in
+                       zip(weights, (self.key_size, self.key_size, self.value_size),
+                           (self.head_dim, self.head_dim, self.v_head_dim))]
+            o_weight = _padded_heads(o_weight.t(), self.value_size, self.v_head_dim).t().contiguous()
         if self.head_gate or self.output_gate:
             # The gate's rows ride behind v, filled up to a multiple of 16 rows (what the products' tiles like).
             gate = tensors["g_proj.weight" if self.head_gate else "gate_proj.weight"]
@@ -142,7 +166,7 @@ class Attention:
             self.qkv_bias = torch.cat(biases).contiguous()
         if self.value_mix == "mixed":
             self.blend = tensors["value_mix"].to(torch.float32).reshape(1).contiguous()
-        self.o_weight = tensors["o_proj.weight"]
+        self.o_weight = o_weight
         if self.qk_norm and self.qk_norm_weight:
             self.q_norm_weight, self.k_norm_weight = tensors["q_norm.weight"], tensors["k_norm.weight"]
             if order is not None and self.qk_norm == "head":
@@ -157,68 +181,87 @@ class Attention:
     def cache_needs(self) -> tuple:
         return (KVNeed(self.kv_heads, self.head_dim, self.window, name=self.cache_name,
                        v_head_dim=None if self.v_head_dim == self.head_dim else self.v_head_dim,
-                       keep_first=self.keep_first),)
+                       keep_first=self.keep_first, chunk=self.chunk),)
+
+    # ------------------------------------------------- what a mixer made of several uses
+    @property
+    def in_weight(self) -> torch.Tensor:
+        return self.qkv_weight
+
+    @property
+    def out_weight(self) -> torch.Tensor:
+        return self.o_weight
+
+    @property
+    def mixed_width(self) -> int:
+        return self.heads * self.v_head_dim
+
+    @property
+    def has_biases(self) -> bool:
+        return self.bias or self.out_bias
 
     takes_pending_norm = True       # x may be an ops.PendingNorm: the qkv product folds the norm in
     adds_to_residual = True         # the output projection adds into the residual stream where its kernel can
 
     def forward(self, x, ctx: StepContext, cache: LayerCache, residual: torch.Tensor | None = None):
-        kv = cache.kvs[self.cache_name]
-        tokens = x.shape[0]
-        q_width, kv_width = self.heads * self.head_dim, self.kv_heads * self.head_dim
-        v_width = self.kv_heads * self.v_head_dim
-        qkv = torch.empty((tokens, self.qkv_weight.shape[0]), dtype=x.dtype, device=x.device)
+        qkv = torch.empty((x.shape[0], self.qkv_weight.shape[0]), dtype=x.dtype, device=x.device)
         ops.linear(x, self.qkv_weight, qkv, self.qkv_bias)
-        if self.qk_norm == "head" or self.head_gate or self.output_gate or self.value_mix:
-            return self._forward_prepared(qkv, ctx, cache, residual)
-        if self.qk_norm:
-            ops.qk_projection_rmsnorm_(qkv[:, :q_width], self.q_norm_weight, qkv[:, q_width:q_width + kv_width],
-                                       self.k_norm_weight, self.qk_norm_eps)
+        attended = torch.empty((x.shape[0], self.mixed_width), dtype=x.dtype, device=x.device)
+        self.mix(qkv, ctx, cache, attended)
+        return ops.linear(attended, self.o_weight, None, self.o_bias, residual=residual)
+
+    def mix(self, qkv: torch.Tensor, ctx: StepContext, cache: LayerCache, attended: torch.Tensor) -> None:
+        """From the projection's rows to the heads' outputs, `attended` [tokens, mixed_width] (both may be column slices
+        of wider tensors; q is rotated in place)."""
+        kv = cache.kvs[self.cache_name]
+        q_width, kv_width = self.heads * self.head_dim, self.kv_heads * self.head_dim
         table = ctx.block_tables[kv.group]
         rotary = self.position.rotary()
-        attended = torch.empty((tokens, self.heads * self.v_head_dim), dtype=x.dtype, device=x.device)
         masked = dict(keep_first=self.keep_first, softcap=self.softcap) if (self.keep_first or self.softcap) else {}
         if self.sink is not None:
             masked["sink"] = self.sink
-        plain = not masked and self.v_head_dim == self.head_dim and (rotary is None or rotary.attention_scaling == 1.0)
-        if plain and rotary is not None and ops.fused_decode_supports(x.dtype, self.heads, self.kv_heads, self.head_dim,
+        prepared = self.qk_norm == "head" or self.head_gate or self.output_gate or self.value_mix
+        if self.qk_norm and not prepared:
+            ops.qk_projection_rmsnorm_(qkv[:, :q_width], self.q_norm_weight, qkv[:, q_width:q_width + kv_width],
+                                       self.k_norm_weight, self.qk_norm_eps)
+        plain = (not masked and not prepared and self.v_head_dim % self.head_dim == 0
+                 and (rotary is None or rotary.attention_scaling == 1.0))
+        newest = {}
+        if plain and rotary is not None and ops.fused_decode_supports(qkv.dtype, self.heads, self.kv_heads, self.head_dim,
                                                                       rotary.rotary_dim, ctx.plan):
             # Every sequence brings one token: one launch rotates q and k, stores k and v and attends.
-            newest = ops.NewestToken(rotary.inv_freq, qkv[:, q_width:], qkv[:, q_width + kv_width:],
-                                     store=not cache.read_only)
-            ops.paged_attention(qkv, qkv.shape[1], attended, kv.k_pool, kv.v_pool, table, ctx.query_start_loc,
-                                ctx.context_lens, ctx.num_seqs, ctx.max_query_len, self.heads, self.kv_heads,
-                                self.head_dim, self.scale, self.window or 0, plan=ctx.plan,
-                                decode_splits=ctx.decode_splits, newest=newest)
-            return ops.linear(attended, self.o_weight, None, self.o_bias, residual=residual)
-        if rotary is None:
-            self.position.apply(qkv[:, :q_width].unflatten(1, (self.heads, self.head_dim)),
-                                qkv[:, q_width:q_width + kv_width].unflatten(1, (self.kv_heads, self.head_dim)), ctx)
-        wide = {} if plain else dict(v_head_dim=self.v_head_dim,
-                                     cos_sin_scale=rotary.attention_scaling if rotary else 1.0)
-        ops.rope_kv_write(qkv, ctx.positions, ctx.seq_of_token, table, kv.k_pool, kv.v_pool,
-                          rotary.inv_freq if rotary else None, self.heads, self.kv_heads, self.head_dim,
-                          rotary.rotary_dim if rotary else 0, store=not cache.read_only, **wide)
-        ops.paged_attention(qkv, qkv.shape[1], attended, kv.k_pool, kv.v_pool, table, ctx.query_start_loc,
+            newest["newest"] = ops.NewestToken(rotary.inv_freq, qkv[:, q_width:], qkv[:, q_width + kv_width:],
+                                               store=not cache.read_only)
+        else:
+            self._store(qkv, ctx, cache, kv, table, rotary, prepared)
+        if self.chunk is not None:
+            masked["chunk"] = self.chunk
+        ops.paged_attention(qkv, qkv.stride(0), attended, kv.k_pool, kv.v_pool, table, ctx.query_start_loc,
                             ctx.context_lens, ctx.num_seqs, ctx.max_query_len, self.heads, self.kv_heads,
                             self.head_dim, self.scale, self.window or 0, plan=ctx.plan,
-                            decode_splits=ctx.decode_splits, **masked)
-        return ops.linear(attended, self.o_weight, None, self.o_bias, residual=residual)
+                            decode_splits=ctx.decode_splits, **masked, **newest)
+        gate_at = q_width + kv_width + self.kv_heads * self.v_head_dim
+        if self.head_gate:
+            ops.sigmoid_gate_heads_(attended, qkv[:, gate_at:gate_at + self.heads], self.heads)
+        elif self.output_gate:
+            ops.sigmoid_gate_(attended, qkv[:, gate_at:gate_at + self.heads * self.v_head_dim])
 
-
-    def _forward_prepared(self, qkv: torch.Tensor, ctx: StepContext, cache: LayerCache, residual):
-        """The path of an attention with per-head q/k norms, mixed values or a head gate: one kernel normalises
-        and rotates q and k, blends v and stores k and v; the attention reads q from the projection's rows; the
-        gate multiplies the heads' outputs in place."""
-        kv = cache.kvs[self.cache_name]
-        tokens = qkv.shape[0]
+    def _store(self, qkv: torch.Tensor, ctx: StepContext, cache: LayerCache, kv, table, rotary, prepared) -> None:
+        """q rotated in place, k rotated and stored, v stored; for an attention with per-head q/k norms or mixed values,
+        or whose rows lie in a wider tensor, one kernel that also normalises q and k and blends v."""
         q_width, kv_width = self.heads * self.head_dim, self.kv_heads * self.head_dim
         v_width = self.kv_heads * self.v_head_dim
-        table = ctx.block_tables[kv.group]
-        rotary = self.position.rotary()
         if rotary is None:
             self.position.apply(qkv[:, :q_width].unflatten(1, (self.heads, self.head_dim)),
                                 qkv[:, q_width:q_width + kv_width].unflatten(1, (self.kv_heads, self.head_dim)), ctx)
+        if not prepared and qkv.is_contiguous():
+            plain = self.v_head_dim == self.head_dim and (rotary is None or rotary.attention_scaling == 1.0)
+            wide = {} if plain else dict(v_head_dim=self.v_head_dim,
+                                         cos_sin_scale=rotary.attention_scaling if rotary else 1.0)
+            ops.rope_kv_write(qkv, ctx.positions, ctx.seq_of_token, table, kv.k_pool, kv.v_pool,
+                              rotary.inv_freq if rotary else None, self.heads, self.kv_heads, self.head_dim,
+                              rotary.rotary_dim if rotary else 0, store=not cache.read_only, **wide)
+            return
         values = qkv[:, q_width + kv_width:q_width + kv_width + v_width]
         other = None
         if self.value_mix == "source":
@@ -240,21 +283,12 @@ class Attention:
                                     self.q_norm_weight if per_head else None, self.k_norm_weight if per_head else None,
                                     self.qk_norm_eps, store=not cache.read_only, v_other=other,
                                     blend=self.blend if other is not None else None, **options)
-        attended = torch.empty((tokens, self.heads * self.v_head_dim), dtype=qkv.dtype, device=qkv.device)
-        masked = dict(keep_first=self.keep_first, softcap=self.softcap) if (self.keep_first or self.softcap) else {}
-        if self.sink is not None:
-            masked["sink"] = self.sink
-        ops.paged_attention(qkv, qkv.shape[1], attended, kv.k_pool, kv.v_pool, table, ctx.query_start_loc,
-                            ctx.context_lens, ctx.num_seqs, ctx.max_query_len, self.heads, self.kv_heads,
-                            self.head_dim, self.scale, self.window or 0, plan=ctx.plan,
-                            decode_splits=ctx.decode_splits, **masked)
-        if self.head_gate:
-            gate_at = q_width + kv_width + v_width
-            ops.sigmoid_gate_heads_(attended, qkv[:, gate_at:gate_at + self.heads], self.heads)
-        elif self.output_gate:
-            gate_at = q_width + kv_width + v_width
-            ops.sigmoid_gate_(attended, qkv[:, gate_at:gate_at + self.heads * self.v_head_dim])
-        return ops.linear(attended, self.o_weight, None, self.o_bias, residual=residual)
+
+
+def _padded_heads(weight: torch.Tensor, old: int, new: int) -> torch.Tensor:
+    """[heads * old, n] with zero rows behind every head's, [heads * new, n]."""
+    heads = weight.unflatten(0, (-1, old))
+    return torch.cat([heads, heads.new_zeros((heads.shape[0], new - old, heads.shape[2]))], dim=1).flatten(0, 1)
 
 
 def _sink_init(shape, generator):

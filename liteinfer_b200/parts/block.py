@@ -33,7 +33,7 @@ def apply_norm(norm, hidden: torch.Tensor, delta, consumer=None, rows: torch.Ten
     """Runs `norm` on the residual stream, whatever form the pending `delta` has (None, a tensor still to be
     added, or `ops.RowStats` of a sum already made), using what the norm and the part that reads its result say
     they can do: a norm that `defers` hands a consumer that `takes_pending_norm` the unfinished norm."""
-    if isinstance(delta, (ops.NormedDelta, ops.StreamUpdate)):
+    if isinstance(delta, (ops.NormedDelta, ops.StreamUpdate, ops.SumDelta)):
         return norm.forward(hidden, delta) if rows is None else norm.forward(hidden, delta, rows=rows)
     if isinstance(delta, ops.RowStats) and not getattr(norm, "reads_row_stats", False):
         delta = None                # the sum is in `hidden` already; a plain norm needs no more
@@ -70,6 +70,38 @@ class PreNormResidualBlock:
         mixed = run_part(self.mixer, normed, hidden, ctx, cache)
         normed = apply_norm(self.feed_forward_norm, hidden, mixed, self.feed_forward)
         return hidden, run_part(self.feed_forward, normed, hidden, ctx)
+
+
+class ParallelNormsBlock:
+    """h = h + (mixer(norm(h)) + feed_forward(norm'(h))): both sublayers read the same stream, each through a norm of its
+    own.  One kernel makes both norms, and on its way adds up what the layer before left pending (`ops.SumDelta`: the
+    mixer's output, the experts' rows, a shared expert's), so a layer touches the 32-bit stream once.  A sublayer that
+    `gives_sum` returns such a delta itself."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "feed_forward_norm": "norm", "feed_forward": "feed_forward"}
+
+    def __init__(self, parts: dict) -> None:
+        self.mixer_norm, self.mixer = parts["mixer_norm"], parts["mixer"]
+        self.feed_forward_norm = parts.get("feed_forward_norm")
+        self.feed_forward = parts.get("feed_forward")
+
+    @staticmethod
+    def _sum(part, value) -> "ops.SumDelta":
+        return value if getattr(part, "gives_sum", False) else ops.SumDelta((ops.SumTerm(value),))
+
+    def forward(self, hidden: torch.Tensor, delta, ctx: StepContext, cache: LayerCache):
+        if self.feed_forward is None:
+            normed = self.mixer_norm.forward(hidden, delta)
+            return hidden, self._sum(self.mixer, self.mixer.forward(normed, ctx, cache))
+        normed, also = self.mixer_norm.forward_pair(self.feed_forward_norm, hidden, delta)
+        mixed = self._sum(self.mixer, self.mixer.forward(normed, ctx, cache))
+        return hidden, mixed + self._sum(self.feed_forward, self.feed_forward.forward(also, ctx))
+
+
+class ParallelNormsMixerBlock(ParallelNormsBlock):
+    """`ParallelNormsBlock` of a layer that has no feed-forward."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer"}
 
 
 class SandwichNormBlock:
@@ -177,6 +209,8 @@ class StreamMixedMixerBlock(StreamMixedBlock):
 
 
 register_block("prenorm_residual", PreNormResidualBlock)
+register_block("parallel_norms", ParallelNormsBlock)
+register_block("parallel_norms_mixer_only", ParallelNormsMixerBlock)
 register_block("stream_mixed", StreamMixedBlock)
 register_block("stream_mixed_mixer_only", StreamMixedMixerBlock)
 register_block("output_norm", OutputNormBlock)

@@ -21,8 +21,10 @@ class KVNeed:
     `keep_first` tokens of the sequence.  `v_head_dim`: the size of a value where
     it differs from a key's (None: the same).  `name` is the key under
     which the part finds its pages in its layer's `LayerCache.kvs`; a layer whose
-    parts declare several needs gives each its own name.  Needs that are equal
-    apart from the name share a group of pages."""
+    parts declare several needs gives each its own name.  `chunk` (instead of a
+    window): the sequence is read in chunks of that many positions, a token
+    reads its own chunk only, and what lies before the chunk of the next token
+    is not kept.  Needs that are equal apart from the name share a group of pages."""
 
     kv_heads: int
     head_dim: int
@@ -30,6 +32,23 @@ class KVNeed:
     name: str = field(default="kv", compare=False)
     v_head_dim: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
+
+    @property
+    def keeps_all(self) -> bool:
+        return self.window is None and self.chunk is None
+
+    def first_needed(self, total: int) -> int:
+        """The first position that a request holding `total` tokens can still read (behind the first ones it keeps):
+        the next query sits at `total` or later."""
+        if self.chunk is not None:
+            return total // self.chunk * self.chunk
+        return 0 if self.window is None else max(0, total - self.window + 1)
+
+    @property
+    def span(self) -> int | None:
+        """The most tokens, itself included, that a query reads behind the first ones (None: all)."""
+        return self.chunk if self.chunk is not None else self.window
 
     @property
     def value_dim(self) -> int:

@@ -17,11 +17,13 @@ import liteinfer_b200.parts.connection  # noqa: F401
 import liteinfer_b200.parts.delta_rule  # noqa: F401
 import liteinfer_b200.parts.embedding  # noqa: F401
 import liteinfer_b200.parts.feed_forward  # noqa: F401
+import liteinfer_b200.parts.hgrn2  # noqa: F401
 import liteinfer_b200.parts.latent_attention  # noqa: F401
 import liteinfer_b200.parts.mlstm  # noqa: F401
 import liteinfer_b200.parts.norm  # noqa: F401
 import liteinfer_b200.parts.position  # noqa: F401
 import liteinfer_b200.parts.reentry  # noqa: F401
+import liteinfer_b200.parts.side_by_side  # noqa: F401
 from liteinfer_b200 import ops
 from liteinfer_b200.parts.block import apply_norm
 from liteinfer_b200.parts.context import LayerCache, StepContext
@@ -38,6 +40,8 @@ def _settled(hidden: torch.Tensor, delta, copies: int | None = None) -> torch.Te
         return out.view(out.shape[0], copies, -1).sum(1)
     if isinstance(delta, ops.NormedDelta):
         ops.layernorm_add(out, delta.value, delta.weight, delta.eps, centred=delta.centred)
+    elif isinstance(delta, ops.SumDelta):
+        ops.sum_norms(out, delta, (), 0.0, (), write_stream=True)
     elif isinstance(delta, torch.Tensor):
         ops.add_(out, delta)
     return out
@@ -132,8 +136,8 @@ class Model:
         if self.spec.stream_copies is not None:
             # The residual is 32-bit streams: the embedding widens its rows itself and writes every copy.
             embedded, hidden = None, self.embedding.forward_streams(ctx.token_ids, self.spec.stream_copies)
-        elif self.wide_stream and getattr(self.embedding, "scale", 1.0) != 1.0:
-            # A scaled embedding starts the 32-bit stream itself: the row is widened before the multiply.
+        elif self.wide_stream and (self.spec.widened_embedding or getattr(self.embedding, "scale", 1.0) != 1.0):
+            # The embedding starts the 32-bit stream itself: the row is widened (before the multiply, if it is scaled).
             embedded = hidden = self.embedding.forward_streams(ctx.token_ids, 1)
             return self._walk(hidden, embedded, ctx, caches)
         else:

@@ -103,7 +103,8 @@ class AffineRMSNorm:
     (offset + weight) * mult is formed once, in 32-bit, when the tensors are bound.  Like `LayerNorm` it reads a
     stream that may be 32-bit whatever the engine's dtype, writes the engine's dtype, and takes a pending
     `ops.NormedDelta`; `normed_delta` makes one of a sublayer's output, for a block that normalises what a sublayer
-    gives back."""
+    gives back.  A pending `ops.SumDelta` (over a 32-bit stream) is summed on the way, and `forward_pair` makes this
+    norm and another one of the same stream in one pass over it."""
 
     def __init__(self, size: int, eps: float, dtype: torch.dtype, device: torch.device, offset: float = 0.0,
                  mult: float = 1.0) -> None:
@@ -117,6 +118,17 @@ class AffineRMSNorm:
     def bind(self, tensors: dict[str, torch.Tensor]) -> None:
         self.weight = ((self.offset + tensors["weight"].to(torch.float32)) * self.mult).contiguous()
 
+    def forward_pair(self, other: "AffineRMSNorm", x: torch.Tensor, delta: "torch.Tensor | ops.SumDelta | None" = None):
+        """(this norm of x + delta, `other` of the same): the sum is stored back into x, a 32-bit stream."""
+        if other.eps != self.eps:
+            return self.forward(x, delta), other.forward(x)
+        if isinstance(delta, torch.Tensor):
+            delta = ops.SumDelta((ops.SumTerm(delta),))
+        outs = tuple(torch.empty((x.shape[0], self.size), dtype=self.dtype, device=x.device) for _ in range(2))
+        ops.sum_norms(x, delta or ops.SumDelta(), (self.weight, other.weight), self.eps, outs,
+                      write_stream=delta is not None)
+        return outs
+
     def forward(self, x: torch.Tensor, delta: "torch.Tensor | ops.NormedDelta | None" = None,
                 rows: torch.Tensor | None = None, out: torch.Tensor | None = None):
         if isinstance(delta, torch.Tensor):     # a plain delta: the sum first, then the norm
@@ -125,6 +137,9 @@ class AffineRMSNorm:
         n = x.shape[0] if rows is None else rows.numel()
         if out is None:
             out = torch.empty((n, self.size), dtype=self.dtype, device=x.device)
+        if isinstance(delta, ops.SumDelta):
+            ops.sum_norms(x, delta, (self.weight,), self.eps, (out,), rows=rows, write_stream=rows is None)
+            return out
         return ops.layernorm(x, self.weight, self.eps, out, delta=delta, rows=rows,
                              write_stream=delta is not None and rows is None, centre=False)
 

@@ -1,0 +1,90 @@
+"""Several mixers side by side: y = sum_i scale_i * mixer_i(h), all reading the same h.
+
+Everything that reads h is one product against the members' projections, and the members' outputs, next to each other in
+one row, pass one product against their output projections, so the members' results are added up inside it.  The scales:
+one is left to whoever adds y into the residual stream (a constant factor of that sum), the others, divided by it, go
+where a member can take a constant without a rounding (`scale_output`) or, failing that, into its rows of the output
+projection.
+
+A member is a mixer with `in_weight`, `out_weight`, `mixed_width` and `mix(projection rows, ctx, cache, out)`; each
+finds its pages or state under the name its own need declares, so members that keep the same kind of thing are given
+different names (`cache_name`, `state_name`).  Their tensors lie behind the members' prefixes.
+"""
+
+from __future__ import annotations
+
+from typing import Mapping, Sequence
+
+import torch
+
+from liteinfer_b200 import ops
+from liteinfer_b200.parts.context import LayerCache, StepContext
+from liteinfer_b200.parts.registry import build_part, register_mixer
+from liteinfer_b200.parts.spec import PartSpec, TensorSpec
+
+
+class SideBySide:
+    """`members`: the mixers' specs; `scales`: their factors; `prefixes`: what stands in front of each member's tensor
+    names (default "0.", "1.", ...)."""
+
+    gives_sum = True        # `forward` returns an ops.SumDelta
+
+    def __init__(self, hidden_size: int, members: Sequence[PartSpec], scales: Sequence[float], dtype: torch.dtype,
+                 device: torch.device, prefixes: Sequence[str] | None = None) -> None:
+        if not members or len(members) != len(scales):
+            raise ValueError("mixers side by side need at least one member and a scale for each")
+        self.hidden_size = hidden_size
+        self.members = [build_part("mixer", spec, dtype=dtype, device=device) for spec in members]
+        self.scales = [float(s) for s in scales]
+        self.prefixes = [f"{i}." for i in range(len(members))] if prefixes is None else list(prefixes)
+        for member in self.members:
+            if not hasattr(member, "mix") or member.has_biases:
+                raise ValueError(f"a {type(member).__name__} with these options cannot run side by side with another mixer")
+        self.factor = 1.0       # what the sum into the stream still has to multiply by
+        self.in_weight = self.out_weight = None
+        self.in_at: list[int] = []
+
+    def tensor_specs(self) -> dict[str, TensorSpec]:
+        return {prefix + name: spec for prefix, member in zip(self.prefixes, self.members)
+                for name, spec in member.tensor_specs().items()}
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        for prefix, member in zip(self.prefixes, self.members):
+            member.bind({name: tensors[prefix + name] for name in member.tensor_specs()})
+        # The factor left to the sum: that of the first member which cannot scale itself, if it is not 0.
+        rigid = [s for s, m in zip(self.scales, self.members) if not hasattr(m, "scale_output") and s != 0.0]
+        self.factor = rigid[0] if rigid else 1.0
+        ins, outs = [], []
+        self.in_at = []
+        at = 0
+        for scale, member in zip(self.scales, self.members):
+            rows = member.in_weight
+            pad = -rows.shape[0] % 16          # every member's columns start on a multiple of 16
+            ins.append(torch.cat([rows, rows.new_zeros((pad, rows.shape[1]))]) if pad else rows)
+            self.in_at.append(at)
+            at += rows.shape[0] + pad
+            out, own = member.out_weight, scale / self.factor
+            if own != 1.0 and not (hasattr(member, "scale_output") and member.scale_output(own)):
+                out = (out.to(torch.float32) * own).to(out.dtype)
+            outs.append(out)
+        self.in_weight = torch.cat(ins).contiguous()
+        self.out_weight = torch.cat(outs, dim=1).contiguous()
+        for member in self.members:             # only the joined copies are kept
+            for name in ("qkv_weight", "o_weight", "in_weight", "out_weight"):
+                if name in vars(member):
+                    setattr(member, name, None)
+
+    def cache_needs(self) -> tuple:
+        return tuple(need for member in self.members for need in member.cache_needs())
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: LayerCache) -> "ops.SumDelta":
+        proj = ops.linear(x, self.in_weight, None)
+        mixed = torch.empty((x.shape[0], self.out_weight.shape[1]), dtype=x.dtype, device=x.device)
+        at = 0
+        for start, end, member in zip(self.in_at, [*self.in_at[1:], proj.shape[1]], self.members):
+            member.mix(proj[:, start:end], ctx, cache, mixed[:, at:at + member.mixed_width])
+            at += member.mixed_width
+        return ops.SumDelta((ops.SumTerm(ops.linear(mixed, self.out_weight, None), self.factor),))
+
+
+register_mixer("side_by_side", SideBySide)

@@ -178,7 +178,7 @@ def _runs(seqs, positions):
 
 def paged_attention(q, q_row_stride, out, k_pool, v_pool, block_table, query_start_loc, context_lens, num_seqs,
                     max_q_len, heads, kv_heads, head_dim, scale, window=0, plan=None, decode_splits=None,
-                    keep_first=0, softcap=0.0, sink=None):
+                    keep_first=0, softcap=0.0, sink=None, chunk=0):
     dtype = out.dtype
     v_dim = v_pool.shape[3]
     page_size = k_pool.shape[2]
@@ -213,6 +213,8 @@ def paged_attention(q, q_row_stride, out, k_pool, v_pool, block_table, query_sta
         hidden = kpos[None, :] > qpos[:, None]
         if window > 0:
             hidden = hidden | ((kpos[None, :] <= qpos[:, None] - window) & (kpos[None, :] >= keep_first))
+        if chunk > 0:
+            hidden = hidden | (kpos[None, :] // chunk != qpos[:, None] // chunk)
         hidden = hidden | (pages < 0)[None, :]
         scores = scores.masked_fill(hidden[None], float("-inf"))
         m = scores.amax(-1, keepdim=True)
@@ -270,11 +272,14 @@ def qk_projection_rmsnorm_(q, q_weight, k, k_weight, eps):
 def gated_rmsnorm(x, gate, weight, eps, out, heads, gate_activation="silu", den=None):
     tokens, width = out.shape
     size = width // heads
-    g = gate.float()
     v = x.view(tokens, heads, size)
     if den is not None:
         v = v / den.view(tokens, heads, 1)
     y = _norm(v, eps, centre=False) * weight.float().view(-1, size)
+    if gate is None:
+        out.copy_(y.reshape(tokens, width).to(out.dtype))
+        return out
+    g = gate.float()
     act = torch.sigmoid(g) if gate_activation == "sigmoid" else g / (1.0 + torch.exp(-g))
     out.copy_((y.reshape(tokens, width) * act).to(out.dtype))
     return out
@@ -356,6 +361,44 @@ def mlstm(proj, offsets, i_bias, f_bias, cap, state, maxima, query_start_loc, st
                 out[t, h * vdim:(h + 1) * vdim] = read[:vdim]
                 den[t, h] = torch.maximum(read[vdim].abs(), torch.exp(-m_new)) + 1e-6
     return out
+
+
+def hgrn2(proj, offsets, f_bias, lower, state, query_start_loc, state_slots, num_seqs, heads, dim, vdim, norm_weight, eps,
+          out, max_query_len=0):
+    """state: [slots, heads, vdim, dim], the transpose of S [dim, vdim] per head."""
+    qsl, slots = query_start_loc.tolist(), state_slots.tolist()
+    q_off, f_off, v_off = offsets
+    q = proj[:, q_off:q_off + heads * dim].float()
+    q = (q * torch.sigmoid(q)).unflatten(1, (heads, dim))
+    f = (lower + (1.0 - lower) * torch.sigmoid(proj[:, f_off:f_off + heads * dim].float() + f_bias)).unflatten(1, (heads, dim))
+    v = proj[:, v_off:v_off + heads * vdim].float().unflatten(1, (heads, vdim))
+    for s in range(num_seqs):
+        for t in range(qsl[s], qsl[s + 1]):
+            S = state[slots[s]]
+            S.copy_(f[t][:, None, :] * S + v[t][:, :, None] * (1.0 - f[t])[:, None, :])
+            o = torch.einsum("hvd,hd->hv", S, q[t])
+            out[t] = (_norm(o, eps, centre=False) * norm_weight).reshape(-1).to(out.dtype)
+    return out
+
+
+def sum_norms(x, delta, weights, eps, outs, rows=None, write_stream=False):
+    total = torch.zeros(x.shape if x is not None else outs[0].shape, device=(x if x is not None else outs[0]).device)
+    for term in delta.terms:
+        v = term.value.float() * term.factor
+        total = total + (v if term.row_factor is None else v * term.row_factor[:, None])
+    if delta.routed is not None:
+        each = delta.routed.value if delta.routed.place is None else delta.routed.value[delta.routed.place.long()]
+        total = total + each.float().view(total.shape[0], delta.routed.top, -1).sum(1)
+    if x is None:
+        outs[0].copy_(total.to(outs[0].dtype))
+        return
+    v = x + total
+    if write_stream:
+        x.copy_(v)
+    if rows is not None:
+        v = v[rows.long()]
+    for w, out in zip(weights, outs):
+        out.copy_((_norm(v, eps, centre=False) * w).to(out.dtype))
 
 
 def short_conv_step(x, taps, tail, seq_of_token, query_start_loc, state_slots, num_seqs, out, activation="silu",
@@ -593,26 +636,38 @@ def gate_heads(v, gate, out):
     return out
 
 
-def moe_route(logits, top, groups, keep, renormalise, ids, weights):
-    scores = torch.softmax(logits.float(), dim=-1)
+def moe_route(logits, top, groups, keep, renormalise, ids, weights, scores="softmax", correction=None, rank_by=1, floor=0.0):
+    scores = torch.softmax(logits.float(), dim=-1) if scores == "softmax" else torch.sigmoid(logits.float())
+    choice = scores if correction is None else scores + correction
     tokens, experts = scores.shape
     allowed = torch.ones_like(scores, dtype=torch.bool)
     if groups > 1:
         per = experts // groups
-        best = scores.view(tokens, groups, per).amax(-1)
+        best = choice.view(tokens, groups, per).topk(min(rank_by, per), dim=-1).values.sum(-1)
         kept = torch.zeros(tokens, groups, dtype=torch.bool, device=scores.device)
         kept.scatter_(1, best.topk(keep, dim=-1).indices, True)
         allowed = kept.repeat_interleave(per, dim=1)
-    chosen = torch.where(allowed, scores, torch.full_like(scores, -1.0)).topk(top, dim=-1).indices
+    chosen = torch.where(allowed, choice, torch.full_like(choice, -math.inf)).topk(top, dim=-1).indices
     picked = scores.gather(1, chosen)
     if renormalise:
-        picked = picked / picked.sum(-1, keepdim=True)
+        picked = picked / (picked.sum(-1, keepdim=True) + floor)
     ids.copy_(chosen.to(torch.int32))
     weights.copy_(picked)
 
 
-def moe_router(x, weight, top, groups, keep, renormalise, ids, weights):
-    moe_route(x.float() @ weight.float().t(), top, groups, keep, renormalise, ids, weights)
+def moe_router(x, weight, top, groups, keep, renormalise, ids, weights, scores="softmax", correction=None, rank_by=1,
+               floor=0.0, gated=False, gate=None):
+    logits = x.float() @ weight.float().t()
+    experts = logits.shape[1] - int(gated)
+    moe_route(logits[:, :experts], top, groups, keep, renormalise, ids[:, :top], weights[:, :top], scores, correction,
+              rank_by, floor)
+    if gated:
+        g = torch.sigmoid(logits[:, experts])
+        if gate is not None:
+            gate.copy_(g)
+        for k in range(top, ids.shape[1]):
+            ids[:, k] = experts + k - top
+            weights[:, k] = g
 
 
 def moe_tile_rows(dtype, hidden, ff, pairs=None):
@@ -639,13 +694,20 @@ def _halves(w, eights):
 
 
 def moe_experts(x, gate_up, down, ids, weights, activation, limit, alpha, eights, out):
+    rows = moe_expert_rows(x, gate_up, down, ids, weights, activation, limit, alpha, eights)
+    return moe_combine(rows.value, out, rows.top)
+
+
+def moe_expert_rows(x, gate_up, down, ids, weights, activation, limit, alpha, eights):
+    from liteinfer_b200.ops import RoutedRows
+
     tokens, top = ids.shape
     plan = moe_sort(ids, gate_up.shape[0], 32)
     act = torch.empty(tokens * top, down.shape[2], dtype=x.dtype, device=x.device)
     each = torch.empty(tokens * top, down.shape[1], dtype=x.dtype, device=x.device)
     moe_grouped("gate_up", x, gate_up, act, plan, top, activation, limit, alpha, eights=eights)
     moe_grouped("down", act, down, each, plan, top, pair_weights=weights.view(-1))
-    return moe_combine(each, out, top)
+    return RoutedRows(each, top)
 
 
 def moe_grouped(mode, a, weight, out, plan, top, activation="swiglu", limit=0.0, alpha=1.0, pair_weights=None,
@@ -677,7 +739,7 @@ def fused_decode_supports(*args) -> bool:
     return False      # the stand-ins rotate and store in `rope_kv_write`, never inside the attention
 
 
-ALL = ("moe_router", "moe_experts", "moe_route", "moe_tile_rows", "moe_sort", "moe_grouped", "moe_combine", "sigmoid_gate_", "softcap_",
+ALL = ("hgrn2", "sum_norms", "moe_expert_rows", "moe_router", "moe_experts", "moe_route", "moe_tile_rows", "moe_sort", "moe_grouped", "moe_combine", "sigmoid_gate_", "softcap_",
        "head_norm_rope_kv_write", "sigmoid_gate_heads_", "mlstm", "embedding_streams", "stream_rmsnorm", "activation", "batched_linear", "latent_prep", "latent_attention",
        "gate_heads", "convert", "layernorm", "layernorm_add", "projection_rmsnorm_", "qk_projection_rmsnorm_", "gated_rmsnorm",
        "short_conv", "short_conv_step", "short_conv_update", "gated_delta_rule", "fused_decode_supports", "scatter_tokens", "embedding", "rmsnorm", "add_", "add_bias_", "act_mul", "act_mul_interleaved", "gated_linear_supported",
