@@ -17,6 +17,8 @@ decoder beside the Llama decoder at equal layer sizes, and the Kegizen kernels o
 `--compare gifudra` does the same for the Gifudra decoder (latent attention, residual streams).
 `--compare karupel` sets the Karupel decoder (mLSTM, delta-rule and gated attention layers) beside a Kegizen decoder of
 the same sizes, its closest relative, and its kernels beside their like.
+`--compare lulisun` sets the Lulisun decoder (chunked attention and an HGRN2 memory side by side, experts in parallel)
+beside a Kutolix decoder of the same sizes.
 `--compare kutolix` sets the Kutolix decoder (windowed gated attention with a sink, windowed latent attention, dense
 and routed feed-forwards) beside a Gifudra decoder of the same sizes, and its kernels beside their like.
 """
@@ -364,6 +366,20 @@ def _kutolix_config(width: int, ff: int, layers: int, heads: int, kv_heads: int,
                                 "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
     return {"architecture": "Kutolix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 2.0},
             "residual_mult": 0.7, "logit_softcap": 30.0, "layers": [(attention, latent)[i % 2] for i in range(layers)]}
+
+
+def _lulisun_config(width: int, ff: int, layers: int, heads: int, kv_heads: int, head_dim: int, vocab: int) -> dict:
+    """In every layer an attention with the heads of the Kutolix attention (chunks of 1,024, half of each head rotated)
+    beside an HGRN2 memory with heads of 128 x 128 as wide as the model; 32 experts a quarter as wide as a dense
+    feed-forward of which each token runs three (eight groups, four kept), and a shared expert of the same width."""
+    h = heads * head_dim // 128
+    layer = {"type": "parallel",
+             "mixer": {"left": {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                "mask": {"size": 1024}, "rot": {"dims": 64, "base": 100000.0}},
+                       "right": {"heads": h, "dim": 128, "vdim": 128}, "left_scale": 0.8, "right_scale": 0.6},
+             "mlp": {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4},
+                     "router": {"experts": 32, "top": 3, "groups": {"count": 8, "keep": 4}}}}
+    return {"architecture": "Lulisun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": [layer] * layers}
 
 
 def _timed(fn, repeats: int = 20, warmup: int = 5, inner: int = 1) -> float:
@@ -848,6 +864,141 @@ def _kutolix_kernels(peaks: dict) -> dict:
     return {k: round(v, 4) for k, v in out.items()}
 
 
+def _lulisun_kernels(peaks: dict) -> dict:
+    """Each kernel that the Lulisun design brought or changed, alone beside its like, as fractions of the measured copy
+    bandwidth (kernels that stream) or product throughput (attention over prompts); inputs larger than L2."""
+    import torch
+
+    from liteinfer_b200 import ops
+    from liteinfer_b200.parts.context import AttentionPlan
+
+    dev, bf = "cuda:0", torch.bfloat16
+    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_burst"] * 1e12
+    out: dict = {}
+
+    def ints(v):
+        return torch.tensor(v, dtype=torch.int32, device=dev)
+
+    def in_graph(fn, inner: int = 10) -> float:
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(inner):
+                fn()
+        return _timed(graph.replay, repeats=10, warmup=2) / inner
+
+    # -- chunked attention (16 / 4 heads of 128, chunks of 1,024) beside a sliding window of 1,024 with a sink; values as
+    #    wide as keys, twice as wide, and heads of 96 with values of 192 (rounded up to 128 and 256)
+    H, kv_heads, page, n, span = 16, 4, 16, 2048, 1024
+    pages = n // page
+    sink = torch.zeros(H, device=dev)
+    windowed = n * (n + 1) // 2 - (n - span) * (n - span + 1) // 2          # (query, key) pairs
+    chunked = (n // span) * span * (span + 1) // 2
+    cases = (("chunked_attention", 128, 128, 128, 128, dict(chunk=span), chunked),
+             ("kutolix_attention", 128, 128, 128, 128, dict(window=span, sink=sink), windowed),
+             ("chunked_attention_values256", 128, 256, 128, 256, dict(chunk=span), chunked),
+             ("chunked_attention_96_192", 128, 256, 96, 192, dict(chunk=span), chunked))
+    for name, hd, vd, dim, vdim, extra, pairs in cases:
+        k_pool = torch.randn(pages * 64, kv_heads, page, hd, device=dev).to(bf)
+        v_pool = torch.randn(pages * 64, kv_heads, page, vd, device=dev).to(bf)
+        table = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages)
+        q, o = torch.randn(n, H * hd, device=dev).to(bf), torch.empty(n, H * vd, dtype=bf, device=dev)
+        plan = AttentionPlan(num_prefill=1, prefill_seqs=ints([0]), max_prefill_query_len=n)
+        args = (q, q.shape[1], o, k_pool, v_pool, table, ints([0, n]), ints([n]), 1, n, H, kv_heads, hd, dim ** -0.5)
+        ms = _timed(lambda: ops.paged_attention(*args, plan=plan, **extra))
+        out[f"{name}_prompt_us"] = ms * 1e3
+        out[f"{name}_prompt_tflops_frac"] = 2 * H * (dim + vdim) * pairs / (ms * 1e-3) / tflops
+        for B in (64, 8):
+            table = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
+            plan = AttentionPlan(num_decode=B, decode_seqs=ints(list(range(B))), decode_tokens=ints(list(range(B))),
+                                 max_decode_context_len=n)
+            q, o = torch.randn(B, H * hd, device=dev).to(bf), torch.empty(B, H * vd, dtype=bf, device=dev)
+            args = (q, q.shape[1], o, k_pool, v_pool, table, ints(list(range(B + 1))), ints([n] * B), B, 1, H, kv_heads, hd,
+                    dim ** -0.5)
+            ms = in_graph(lambda: ops.paged_attention(*args, plan=plan, **extra))       # the last token of a full chunk
+            out[f"{name}_decode_b{B}_us"] = ms * 1e3
+            out[f"{name}_decode_b{B}_hbm_frac"] = B * span * kv_heads * (dim + vdim) * 2 / (ms * 1e-3) / hbm
+
+    # -- the memory (16 heads of 128 x 128) beside the mLSTM: single tokens of 64 and 8 requests, a prompt of 2,048, eight
+    #    prompts of 2,048
+    d = 128
+    for batch, tokens_each, key in ((64, 1, "decode_b64"), (8, 1, "decode_b8"), (1, 2048, "prompt_2048"),
+                                    (8, 2048, "prompts_8x2048")):
+        m = batch * tokens_each
+        q2, sl = ints([i * tokens_each for i in range(batch + 1)]), ints(list(range(batch)))
+        proj = torch.randn(m, 4 * H * d + 2 * H, device=dev).to(bf)
+        state, maxima = torch.zeros(batch, H, d + 1, d, device=dev), torch.zeros(batch, H, d + 1, device=dev)
+        o32, dn, bias = torch.empty(m, H * d, device=dev), torch.empty(m, H, device=dev), torch.zeros(H, device=dev)
+        offsets = (0, H * d, 2 * H * d, 4 * H * d, 4 * H * d + H)
+        wide_w, gated = torch.ones(H * d, device=dev), torch.empty(m, H * d, dtype=bf, device=dev)
+
+        def mlstm():
+            ops.mlstm(proj, offsets, bias, bias, 15.0, state, maxima, q2, sl, batch, H, d, d, o32, dn, tokens_each)
+            ops.gated_rmsnorm(o32, proj[:, 3 * H * d:4 * H * d], wide_w, 1e-5, gated, H, gate_activation="sigmoid", den=dn)
+
+        s2 = torch.zeros(batch, H, d, d, device=dev)
+        f_bias, lower, weight = torch.zeros(H * d, device=dev), torch.full((H * d,), 0.5, device=dev), torch.ones(d, device=dev)
+
+        def hgrn2():
+            ops.hgrn2(proj, (0, H * d, 2 * H * d), f_bias, lower, s2, q2, sl, batch, H, d, d, weight, 1e-5, gated, tokens_each)
+
+        for name, run, rows in (("hgrn2", hgrn2, d), ("karupel_mlstm", mlstm, d + 1)):      # both with the norm behind them
+            ms = in_graph(run) if tokens_each == 1 else _timed(run)
+            out[f"{name}_{key}_us"] = ms * 1e3
+            if tokens_each == 1:
+                out[f"{name}_{key}_hbm_frac"] = batch * H * rows * d * 4 * 2 / (ms * 1e-3) / hbm
+            else:       # three (two for a scalar decay: 2.5) multiply-adds an entry and token, against 75 TFLOP/s of FFMA
+                out[f"{name}_{key}_ffma_frac"] = m * H * rows * d * 6 / (ms * 1e-3) / 75e12
+
+    # -- the 32-bit sum of a layer and the two norms behind it: the mixer's output and four experts' rows a token, beside
+    #    what Kutolix does (combine the experts' rows; add the normalised output into the stream, which is rounded)
+    W, top = 2048, 4
+    for T, key in ((8192, "8192"), (64, "b64"), (8, "b8")):
+        x, mixed = torch.randn(T, W, device=dev), torch.randn(T, W, device=dev).to(bf)
+        rows, w32 = torch.randn(T * top, W, device=dev).to(bf), torch.ones(W, device=dev)
+        place = torch.randperm(T * top, device=dev).to(torch.int32)
+        o1, o2, y = (torch.empty(T, W, dtype=bf, device=dev) for _ in range(3))
+        delta = ops.SumDelta((ops.SumTerm(mixed, 0.8),), ops.RoutedRows(rows, top, place))
+        timer = _timed if T > 64 else in_graph
+        ms = timer(lambda: ops.sum_norms(x, delta, (w32, w32), 1e-5, (o1, o2), write_stream=True))
+        out[f"sum_norms_{key}_us"] = ms * 1e3
+        out[f"sum_norms_{key}_hbm_frac"] = T * W * (8 + 2 + 2 * top + 4) / (ms * 1e-3) / hbm
+
+        def apart():
+            ops.moe_combine(rows, y, top, place=place)
+            ops.layernorm_add(x, y, w32, 1e-5, centred=False, out=o1)
+
+        ms = timer(apart)
+        out[f"kutolix_combine_and_norm_{key}_us"] = ms * 1e3
+        out[f"kutolix_combine_and_norm_{key}_hbm_frac"] = T * W * (2 * top + 2 + 8 + 2 + 2) / (ms * 1e-3) / hbm
+
+    # -- the router (sigmoid scores, correction, groups by their two best, the shared expert's slot) beside Kutolix's;
+    #    the experts of a token: three and the shared one, beside four
+    F, E = 2048, 32
+    gate_up = (torch.randn(E + 1, 2 * F, W, device=dev) * 0.02).to(bf)
+    down = (torch.randn(E + 1, W, F, device=dev) * 0.02).to(bf)
+    router, correction = torch.randn(E + 1, W, device=dev) * 0.02, torch.zeros(E, device=dev)
+    for tokens, key in ((2048, "prompt_2048"), (64, "decode_b64"), (8, "decode_b8")):
+        x = torch.randn(tokens, W, device=dev).to(bf)
+        ids, weights = torch.empty(tokens, top, dtype=torch.int32, device=dev), torch.empty(tokens, top, device=dev)
+        timer = _timed if tokens > 64 else in_graph
+        four = router[:E].contiguous()
+        forms = (("lulisun", lambda: ops.moe_router(x, router, 3, 8, 4, True, ids, weights, scores="sigmoid",
+                                                    correction=correction, rank_by=2, floor=1e-20, gated=True), gate_up, down),
+                 ("kutolix", lambda: ops.moe_router(x, four, 4, 8, 4, False, ids, weights), gate_up[:E], down[:E]))
+        for name, route, gu, dn in forms:
+            out[f"{name}_router_{key}_us"] = timer(route) * 1e3
+            ms = timer(lambda: ops.moe_expert_rows(x, gu, dn, ids, weights, "swiglu", 0.0, 1.0, True))
+            out[f"{name}_experts_{key}_us"] = ms * 1e3
+            if tokens > 64:
+                out[f"{name}_experts_{key}_tflops_frac"] = 2 * tokens * top * 3 * F * W / (ms * 1e-3) / tflops
+            else:
+                active = int(torch.unique(ids).numel())
+                out[f"{name}_experts_{key}_hbm_frac"] = active * 3 * F * W * 2 / (ms * 1e-3) / hbm
+    return {k: round(v, 4) for k, v in out.items()}
+
+
 def run_kegizen(args, which: str = "kegizen") -> dict:
     """Prefill (one prompt of 2,048 tokens) and decode (batch 8 and 64 near a context of 2,048) of a Kegizen (or
     Gifudra) model and of a Llama model with the same width, depth, head sizes and feed-forward, random weights,
@@ -868,10 +1019,11 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
     if which == "gifudra":      # heads of 128 in both sizes: the latent attention's heads are 128 + 64 wide
         sizes = {"w2048": dict(width=2048, ff=8192, layers=8, heads=16, kv_heads=4, head_dim=128),
                  "w4096": dict(width=4096, ff=14336, layers=4, heads=32, kv_heads=8, head_dim=128)}
-    if which == "kutolix":
+    if which in ("kutolix", "lulisun"):
         sizes = {"w2048": dict(width=2048, ff=8192, layers=8, heads=16, kv_heads=4, head_dim=128),
                  "w4096": dict(width=4096, ff=14336, layers=4, heads=32, kv_heads=8, head_dim=128)}
-    design = {"gifudra": _gifudra_config, "karupel": _karupel_config, "kutolix": _kutolix_config}.get(which, _kegizen_config)
+    design = {"gifudra": _gifudra_config, "karupel": _karupel_config, "kutolix": _kutolix_config,
+              "lulisun": _lulisun_config}.get(which, _kegizen_config)
     result: dict = {"impl": "ours", "compare": which, "dtype": "bf16", "data": "synthetic ids, random weights",
                     "peaks": peaks, "models": {}}
     for name, size in sizes.items():
@@ -883,6 +1035,8 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
             beside = ("kegizen", _kegizen_config(vocab=vocab, plain_attention=True, **size))
         if which == "kutolix":      # its closest relative: latent attention with a sink and a gate, dense feed-forwards
             beside = ("gifudra", _gifudra_config(vocab=vocab, **size))
+        if which == "lulisun":      # its closest relative: windowed attention, experts in every other layer
+            beside = ("kutolix", _kutolix_config(vocab=vocab, **size))
         for arch, cfg in ((which, design(vocab=vocab, **size)), beside):
             with tempfile.TemporaryDirectory() as tmp:
                 model_dir = write_random_model(cfg, Path(tmp) / arch, seed=0)
@@ -910,7 +1064,8 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
                 runner.check_kernels()
                 llm.close()
                 result["models"][f"{name}_{arch}"] = numbers
-    kernels = {"gifudra": _gifudra_kernels, "karupel": _karupel_kernels, "kutolix": _kutolix_kernels}.get(which, _kegizen_kernels)
+    kernels = {"gifudra": _gifudra_kernels, "karupel": _karupel_kernels, "kutolix": _kutolix_kernels,
+               "lulisun": _lulisun_kernels}.get(which, _kegizen_kernels)
     result["kernels"] = kernels(peaks)
     return result
 
@@ -1052,7 +1207,7 @@ def main() -> int:
     parser.add_argument("--workload", default="none", choices=["none", "3b", "8b", "all"],
                         help="run the reference's larger configurations instead (64 requests under continuous batching "
                              "at the 3B sizes; decode at a context of 8,192 at the 8B sizes) and print their line")
-    parser.add_argument("--compare", default="none", choices=["none", "kegizen", "gifudra", "karupel", "kutolix"],
+    parser.add_argument("--compare", default="none", choices=["none", "kegizen", "gifudra", "karupel", "kutolix", "lulisun"],
                         help="instead of the default run: the Kegizen (or Gifudra) decoder beside the Llama decoder, "
                              "the Karupel decoder beside the Kegizen decoder, or the Kutolix decoder beside the Gifudra "
                              "decoder, at equal layer sizes (prefill, decode, and the design's kernels one by one)")

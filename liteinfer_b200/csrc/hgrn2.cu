@@ -12,7 +12,7 @@
 //                    li_gated_rmsnorm does that norm.)
 //
 // The state is kept column by column, state[slot][head][vdim][dim]: a column is a chain of its own over the tokens,
-// S_j <- f (S_j - v_j) + v_j entry by entry.  In the first form a block takes 16 columns of one head of one sequence;
+// S_j <- f S_j + (1 - f) v_j entry by entry (a gate of exactly 1 leaves the entry as it is).  In the first form a block takes 16 columns of one head of one sequence;
 // sixteen lanes share a pair of columns, each with dim / 16 of their entries in registers for the whole step, so an entry
 // of q and f read from shared memory serves two columns.  The records come in chunks of up to 16 tokens by cp.async,
 // three chunks deep, one block barrier a chunk.  A token's update of S needs nothing of its read-out, so the lanes keep
@@ -35,9 +35,9 @@ __device__ __forceinline__ pair_t make_pair2(float a, float b) {
   asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
   return r;
 }
-__device__ __forceinline__ pair_t add2(pair_t a, pair_t b) {
+__device__ __forceinline__ pair_t mul2(pair_t a, pair_t b) {
   pair_t r;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
 __device__ __forceinline__ pair_t fma2(pair_t a, pair_t b, pair_t c) {
@@ -58,6 +58,31 @@ __device__ __forceinline__ float forget_of(float z, float bias, float lower) {
 
 __device__ __forceinline__ void copy16(float* smem, const float* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem));
+}
+
+// One token on a lane's part of two columns: S <- f S + (1 - f) v, and the lane's parts of the columns' read-outs.  row: the
+// token's q [dimp], f [dimp], values; v0 and v1 its values of the two columns.
+template <int NPL>
+__device__ __forceinline__ void hgrn2_step(pair_t (&S)[2][NPL / 2], const float* __restrict__ row, float v0, float v1, int sub,
+                                           float& read0, float& read1) {
+  const pair_t w0 = make_pair2(v0, v0), w1 = make_pair2(v1, v1), one = make_pair2(1.f, 1.f), minus = make_pair2(-1.f, -1.f);
+  pair_t a0 = make_pair2(0.f, 0.f), a1 = a0, b0 = a0, b1 = a0;
+#pragma unroll
+  for (int j = 0; j < NPL / 4; ++j) {
+    const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(row + 4 * (sub + 16 * j));
+    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(row + 16 * NPL + 4 * (sub + 16 * j));
+    const pair_t g = fma2(f.x, minus, one), h = fma2(f.y, minus, one);
+    S[0][2 * j] = fma2(f.x, S[0][2 * j], mul2(g, w0));
+    S[1][2 * j] = fma2(f.x, S[1][2 * j], mul2(g, w1));
+    S[0][2 * j + 1] = fma2(f.y, S[0][2 * j + 1], mul2(h, w0));
+    S[1][2 * j + 1] = fma2(f.y, S[1][2 * j + 1], mul2(h, w1));
+    a0 = fma2(S[0][2 * j], q.x, a0);
+    a1 = fma2(S[1][2 * j], q.x, a1);
+    b0 = fma2(S[0][2 * j + 1], q.y, b0);
+    b1 = fma2(S[1][2 * j + 1], q.y, b1);
+  }
+  read0 = sum2(a0) + sum2(b0);
+  read1 = sum2(a1) + sum2(b1);
 }
 
 // ------------------------------------------------------------------------------------------ records
@@ -176,30 +201,22 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
 #pragma unroll 1
     for (int g0 = 0; g0 < n; g0 += 8) {
       float p[16];
+      const float* row = tokens + g0 * kPerToken;
+      const float* values = row + 2 * dimp + 2 * group;
+      if (n - g0 >= 8) {
 #pragma unroll
-      for (int i = 0; i < 8; ++i) {
-        p[i] = p[i + 8] = 0.f;
-        if (g0 + i < n) {
-          const float* row = tokens + (g0 + i) * kPerToken;
-          const float2 v = *reinterpret_cast<const float2*>(row + 2 * dimp + 2 * group);
-          const pair_t v0 = make_pair2(v.x, v.x), v1 = make_pair2(v.y, v.y);
-          const pair_t n0 = make_pair2(-v.x, -v.x), n1 = make_pair2(-v.y, -v.y);
-          pair_t a0 = make_pair2(0.f, 0.f), a1 = a0;
+        for (int i = 0; i < 8; ++i) {
+          const float2 v = *reinterpret_cast<const float2*>(values + i * kPerToken);
+          hgrn2_step<NPL>(S, row + i * kPerToken, v.x, v.y, sub, p[i], p[i + 8]);
+        }
+      } else {
 #pragma unroll
-          for (int j = 0; j < NPL / 4; ++j) {
-            const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(row + 4 * (sub + 16 * j));
-            const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(row + dimp + 4 * (sub + 16 * j));
-            S[0][2 * j] = fma2(f.x, add2(S[0][2 * j], n0), v0);
-            S[1][2 * j] = fma2(f.x, add2(S[1][2 * j], n1), v1);
-            S[0][2 * j + 1] = fma2(f.y, add2(S[0][2 * j + 1], n0), v0);
-            S[1][2 * j + 1] = fma2(f.y, add2(S[1][2 * j + 1], n1), v1);
-            a0 = fma2(S[0][2 * j], q.x, a0);
-            a1 = fma2(S[1][2 * j], q.x, a1);
-            a0 = fma2(S[0][2 * j + 1], q.y, a0);
-            a1 = fma2(S[1][2 * j + 1], q.y, a1);
+        for (int i = 0; i < 8; ++i) {
+          p[i] = p[i + 8] = 0.f;
+          if (g0 + i < n) {
+            const float2 v = *reinterpret_cast<const float2*>(values + i * kPerToken);
+            hgrn2_step<NPL>(S, row + i * kPerToken, v.x, v.y, sub, p[i], p[i + 8]);
           }
-          p[i] = sum2(a0);
-          p[i + 8] = sum2(a1);
         }
       }
       // Sixteen sums over sixteen lanes: lane s ends with sum s.
@@ -312,10 +329,10 @@ hgrn2_token_kernel(const T* __restrict__ proj, size_t row_stride, int q_off, int
         const int at = 4 * (sub + 16 * j);
         const float4 q = *reinterpret_cast<const float4*>(qs + at), f = *reinterpret_cast<const float4*>(fs + at);
         float4& x = s[a][j];
-        x.x = fmaf(f.x, x.x - v, v);
-        x.y = fmaf(f.y, x.y - v, v);
-        x.z = fmaf(f.z, x.z - v, v);
-        x.w = fmaf(f.w, x.w - v, v);
+        x.x = fmaf(f.x, x.x, (1.0f - f.x) * v);
+        x.y = fmaf(f.y, x.y, (1.0f - f.y) * v);
+        x.z = fmaf(f.z, x.z, (1.0f - f.z) * v);
+        x.w = fmaf(f.w, x.w, (1.0f - f.w) * v);
         p[a] = fmaf(x.w, q.w, fmaf(x.z, q.z, fmaf(x.y, q.y, fmaf(x.x, q.x, p[a]))));
         if (column < vdim) {
           float* dst = base + (size_t)column * dim + at;

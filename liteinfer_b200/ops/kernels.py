@@ -1370,6 +1370,8 @@ def sum_norms(x: torch.Tensor | None, delta: SumDelta, weights: tuple[torch.Tens
     _on_gpu(x, rows, *weights, *outs, *values, *(t.row_factor for t in terms),
             routed.place if routed is not None else None)
     _int32(rows, "rows")
+    if not values and not outs:
+        return
     dtype = values[0].dtype if values else outs[0].dtype
     width = x.shape[1] if x is not None else outs[0].shape[1]
     tokens = x.shape[0] if x is not None else outs[0].shape[0]

@@ -254,7 +254,7 @@ class Attention:
         if rotary is None:
             self.position.apply(qkv[:, :q_width].unflatten(1, (self.heads, self.head_dim)),
                                 qkv[:, q_width:q_width + kv_width].unflatten(1, (self.kv_heads, self.head_dim)), ctx)
-        if not prepared and qkv.is_contiguous():
+        if not prepared and qkv.is_contiguous() and qkv.shape[1] == q_width + kv_width + v_width:
             plain = self.v_head_dim == self.head_dim and (rotary is None or rotary.attention_scaling == 1.0)
             wide = {} if plain else dict(v_head_dim=self.v_head_dim,
                                          cos_sin_scale=rotary.attention_scaling if rotary else 1.0)

@@ -42,7 +42,10 @@ class SideBySide:
                 raise ValueError(f"a {type(member).__name__} with these options cannot run side by side with another mixer")
         self.factor = 1.0       # what the sum into the stream still has to multiply by
         self.in_weight = self.out_weight = None
-        self.in_at: list[int] = []
+        # Where each member's columns lie in the joined projection and in the joined outputs: both start on a multiple of
+        # 16 columns, so that every member's rows are aligned for 16-byte accesses whatever its neighbours' sizes.
+        self.in_at: list[tuple[int, int]] = []
+        self.out_at: list[tuple[int, int]] = []
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         return {prefix + name: spec for prefix, member in zip(self.prefixes, self.members)
@@ -55,18 +58,21 @@ class SideBySide:
         rigid = [s for s, m in zip(self.scales, self.members) if not hasattr(m, "scale_output") and s != 0.0]
         self.factor = rigid[0] if rigid else 1.0
         ins, outs = [], []
-        self.in_at = []
-        at = 0
+        self.in_at, self.out_at = [], []
+        at = out_end = 0
         for scale, member in zip(self.scales, self.members):
             rows = member.in_weight
-            pad = -rows.shape[0] % 16          # every member's columns start on a multiple of 16
-            ins.append(torch.cat([rows, rows.new_zeros((pad, rows.shape[1]))]) if pad else rows)
-            self.in_at.append(at)
+            pad = -rows.shape[0] % 16
+            ins += [rows, rows.new_zeros((pad, rows.shape[1]))]
+            self.in_at.append((at, at + rows.shape[0]))
             at += rows.shape[0] + pad
             out, own = member.out_weight, scale / self.factor
             if own != 1.0 and not (hasattr(member, "scale_output") and member.scale_output(own)):
                 out = (out.to(torch.float32) * own).to(out.dtype)
-            outs.append(out)
+            pad = -out.shape[1] % 16
+            outs += [out, out.new_zeros((out.shape[0], pad))]
+            self.out_at.append((out_end, out_end + out.shape[1]))
+            out_end += out.shape[1] + pad
         self.in_weight = torch.cat(ins).contiguous()
         self.out_weight = torch.cat(outs, dim=1).contiguous()
         for member in self.members:             # only the joined copies are kept
@@ -79,11 +85,11 @@ class SideBySide:
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: LayerCache) -> "ops.SumDelta":
         proj = ops.linear(x, self.in_weight, None)
-        mixed = torch.empty((x.shape[0], self.out_weight.shape[1]), dtype=x.dtype, device=x.device)
-        at = 0
-        for start, end, member in zip(self.in_at, [*self.in_at[1:], proj.shape[1]], self.members):
-            member.mix(proj[:, start:end], ctx, cache, mixed[:, at:at + member.mixed_width])
-            at += member.mixed_width
+        # (The columns between the members' meet zeros in the product, so they must hold numbers.)
+        gaps = sum(end - start for start, end in self.out_at) != self.out_weight.shape[1]
+        mixed = (torch.zeros if gaps else torch.empty)((x.shape[0], self.out_weight.shape[1]), dtype=x.dtype, device=x.device)
+        for (in_start, in_end), (out_start, out_end), member in zip(self.in_at, self.out_at, self.members):
+            member.mix(proj[:, in_start:in_end], ctx, cache, mixed[:, out_start:out_end])
         return ops.SumDelta((ops.SumTerm(ops.linear(mixed, self.out_weight, None), self.factor),))
 
 
