@@ -12,19 +12,22 @@
 //                    li_gated_rmsnorm does that norm.)
 //
 // The state is kept column by column, state[slot][head][vdim][dim]: a column is a chain of its own over the tokens,
-// S_j <- f S_j + (1 - f) v_j entry by entry (a gate of exactly 1 leaves the entry as it is).  In the first form a block takes 16 columns of one head of one sequence;
-// sixteen lanes share a pair of columns, each with dim / 16 of their entries in registers for the whole step, so an entry
-// of q and f read from shared memory serves two columns.  The records come in chunks of up to 16 tokens by cp.async,
-// three chunks deep, one block barrier a chunk.  A token's update of S needs nothing of its read-out, so the lanes keep
-// their parts of eight tokens' read-outs of both columns and add them up together: fifteen shuffles for sixteen sums, and
-// every sum is the same tree whatever the token's place in a step.  In the second form a block takes one head of one
-// sequence and walks its columns, four a group of lanes in flight, since there the state's bytes are all the work.
+// S_j <- f S_j + (1 - f) v_j entry by entry (a gate of exactly 1 leaves the entry as it is).  In the first form a block
+// takes 16 columns of one head of one sequence; a warp takes two of them, each lane with dim / 32 of their entries in
+// registers for the whole step, so an entry of q and f read from shared memory serves two columns.  The records come in
+// chunks of up to 16 tokens by cp.async, three chunks deep, one block barrier a chunk, and a lane has the next token's
+// entries on their way to its registers while it works on this one's.  A token's update of S needs nothing of its
+// read-out, so the lanes keep their parts of eight tokens' read-outs of both columns and add them up together: sixteen
+// shuffles for sixteen sums, and every sum is the same tree whatever the token's place in a step.  In the second form a
+// block takes one head of one sequence and walks its columns, sixteen lanes a column and several columns in flight, since
+// there the state's bytes are all the work.
 // Sequences that bring no token touch nothing.
 #include "common.cuh"
 
 namespace li {
 
-constexpr int kColumns = 16;        // of a block of the first form: four warps x two groups of lanes x two columns
+constexpr int kColumns = 16;        // of a block of the first form: eight warps x two columns
+constexpr int kStepThreads = 256;
 constexpr int kStages = 3;
 constexpr int kRowGroups = 16;      // of a block of the second form: eight warps x two groups of lanes
 
@@ -60,29 +63,53 @@ __device__ __forceinline__ void copy16(float* smem, const float* gmem) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"((unsigned)__cvta_generic_to_shared(smem)), "l"(gmem));
 }
 
-// One token on a lane's part of two columns: S <- f S + (1 - f) v, and the lane's parts of the columns' read-outs.  row: the
-// token's q [dimp], f [dimp], values; v0 and v1 its values of the two columns.
-template <int NPL>
-__device__ __forceinline__ void hgrn2_step(pair_t (&S)[2][NPL / 2], const float* __restrict__ row, float v0, float v1, int sub,
-                                           float& read0, float& read1) {
-  const pair_t w0 = make_pair2(v0, v0), w1 = make_pair2(v1, v1), one = make_pair2(1.f, 1.f), minus = make_pair2(-1.f, -1.f);
-  pair_t a0 = make_pair2(0.f, 0.f), a1 = a0, b0 = a0, b1 = a0;
+// A lane's entries of one token: N pairs each of q and f, and the token's values of the lane's two columns.
+template <int N>
+struct TokenPart {
+  pair_t q[N], f[N];
+  float2 v;
+};
+
+// row: the token's q [32 * 2N], f [32 * 2N], values.  Pairs of a lane lie side by side in fours of floats where N allows.
+template <int N>
+__device__ __forceinline__ void fetch_part(TokenPart<N>& t, const float* __restrict__ row, int lane, int warp) {
+  constexpr int dimp = 64 * N;
+  if (N == 1) {
+    t.q[0] = *reinterpret_cast<const pair_t*>(row + 2 * lane);
+    t.f[0] = *reinterpret_cast<const pair_t*>(row + dimp + 2 * lane);
+  } else {
 #pragma unroll
-  for (int j = 0; j < NPL / 4; ++j) {
-    const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(row + 4 * (sub + 16 * j));
-    const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(row + 16 * NPL + 4 * (sub + 16 * j));
-    const pair_t g = fma2(f.x, minus, one), h = fma2(f.y, minus, one);
-    S[0][2 * j] = fma2(f.x, S[0][2 * j], mul2(g, w0));
-    S[1][2 * j] = fma2(f.x, S[1][2 * j], mul2(g, w1));
-    S[0][2 * j + 1] = fma2(f.y, S[0][2 * j + 1], mul2(h, w0));
-    S[1][2 * j + 1] = fma2(f.y, S[1][2 * j + 1], mul2(h, w1));
-    a0 = fma2(S[0][2 * j], q.x, a0);
-    a1 = fma2(S[1][2 * j], q.x, a1);
-    b0 = fma2(S[0][2 * j + 1], q.y, b0);
-    b1 = fma2(S[1][2 * j + 1], q.y, b1);
+    for (int j = 0; j < N / 2; ++j) {
+      const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(row + 4 * (lane + 32 * j));
+      const ulonglong2 f = *reinterpret_cast<const ulonglong2*>(row + dimp + 4 * (lane + 32 * j));
+      t.q[2 * j] = q.x; t.q[2 * j + 1] = q.y;
+      t.f[2 * j] = f.x; t.f[2 * j + 1] = f.y;
+    }
   }
-  read0 = sum2(a0) + sum2(b0);
-  read1 = sum2(a1) + sum2(b1);
+  t.v = *reinterpret_cast<const float2*>(row + 2 * dimp + 2 * warp);
+}
+
+// The entry that the first half of pair `i` of a lane is.
+template <int N> __device__ __forceinline__ int entry_of(int i, int lane) {
+  return N == 1 ? 2 * lane : 4 * (lane + 32 * (i >> 1)) + 2 * (i & 1);
+}
+
+// One token on a lane's part of two columns: S <- f S + (1 - f) v, and the lane's parts of the columns' read-outs.
+template <int N>
+__device__ __forceinline__ void hgrn2_step(pair_t (&S)[2][N], const TokenPart<N>& t, float& read0, float& read1) {
+  const pair_t v0 = make_pair2(t.v.x, t.v.x), v1 = make_pair2(t.v.y, t.v.y);
+  const pair_t one = make_pair2(1.f, 1.f), minus = make_pair2(-1.f, -1.f);
+  pair_t a0, a1;
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    const pair_t g = fma2(t.f[i], minus, one);
+    S[0][i] = fma2(t.f[i], S[0][i], mul2(g, v0));
+    S[1][i] = fma2(t.f[i], S[1][i], mul2(g, v1));
+    a0 = i == 0 ? mul2(S[0][i], t.q[i]) : fma2(S[0][i], t.q[i], a0);
+    a1 = i == 0 ? mul2(S[1][i], t.q[i]) : fma2(S[1][i], t.q[i], a1);
+  }
+  read0 = sum2(a0);
+  read1 = sum2(a1);
 }
 
 // ------------------------------------------------------------------------------------------ records
@@ -129,13 +156,13 @@ hgrn2_record_kernel(const T* __restrict__ proj, size_t row_stride, int q_off, in
 }
 
 // ----------------------------------------------------------------------------------------- several tokens
-// NPL: entries of a column that a lane keeps (a multiple of four); dimp = 16 NPL.
-template <int NPL, int CHUNK>
-__global__ void __launch_bounds__(128)
+// N: pairs of entries of a column that a lane keeps; dimp = 64 N.
+template <int N, int CHUNK>
+__global__ void __launch_bounds__(kStepThreads)
 hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state, const int* __restrict__ query_start_loc,
                    const int* __restrict__ state_slots, float* __restrict__ out, int heads, int dim, int vdim, int vdimp) {
   extern __shared__ __align__(16) float shared[];       // kStages x CHUNK x (q [dimp], f [dimp], v [kColumns])
-  constexpr int dimp = 16 * NPL;
+  constexpr int dimp = 64 * N;
   constexpr int kPerToken = 2 * dimp + kColumns;
   constexpr int kCopies = kPerToken / 4;                // 16-byte copies of a token
   const int seq = blockIdx.z, head = blockIdx.y, first_column = blockIdx.x * kColumns;
@@ -150,15 +177,15 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
   auto stage = [&](int c) {
     float* dst = shared + (c % kStages) * CHUNK * kPerToken;
     const int n = min(CHUNK, end - begin - c * CHUNK) * kCopies;
-    for (int i = threadIdx.x; i < n; i += 128) {
+    for (int i = threadIdx.x; i < n; i += kStepThreads) {
       const int tok = i / kCopies, e = (i - tok * kCopies) * 4;
       const float* src = source + (size_t)(c * CHUNK + tok) * heads * record;
       copy16(dst + tok * kPerToken + e, src + (e < 2 * dimp ? e : e + first_column));
     }
   };
 
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 15, group = warp * 2 + (lane >> 4);
-  const int col0 = first_column + 2 * group;            // and the next one
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int col0 = first_column + 2 * warp;             // and the next one
   grid_dependency_wait();
 #pragma unroll
   for (int c = 0; c < kStages - 1; ++c) {
@@ -166,29 +193,26 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
     asm volatile("cp.async.commit_group;\n" ::);
   }
   float* mine = state + (((size_t)slot * heads + head) * vdim + col0) * dim;
-  const bool vec = dim % 4 == 0;                        // (the caller's state is 16-byte aligned)
-  pair_t S[2][NPL / 2];
+  const bool vec = dim % 2 == 0;                        // (the caller's state is 16-byte aligned)
+  pair_t S[2][N];
 #pragma unroll
   for (int c = 0; c < 2; ++c)
 #pragma unroll
-    for (int j = 0; j < NPL / 4; ++j) {
-      const int at = 4 * (sub + 16 * j);
-      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < N; ++i) {
+      const int at = entry_of<N>(i, lane);
+      const float* p = mine + (size_t)c * dim + at;
+      float2 v = make_float2(0.f, 0.f);
       if (col0 + c < vdim) {
-        const float* p = mine + (size_t)c * dim + at;
-        if (vec) { if (at < dim) v = *reinterpret_cast<const float4*>(p); }
+        if (vec) { if (at < dim) v = *reinterpret_cast<const float2*>(p); }
         else {
           if (at < dim) v.x = p[0];
           if (at + 1 < dim) v.y = p[1];
-          if (at + 2 < dim) v.z = p[2];
-          if (at + 3 < dim) v.w = p[3];
         }
       }
-      S[c][2 * j] = make_pair2(v.x, v.y);
-      S[c][2 * j + 1] = make_pair2(v.z, v.w);
+      S[c][i] = make_pair2(v.x, v.y);
     }
-  // Lane `sub` of a group writes the read-out of column col0 + (sub >> 3) of token (sub & 7) of every eight.
-  const int out_col = col0 + (sub >> 3);
+  // Lane s writes (in the warp's first half) the read-out of column col0 + (s >> 3) of token s & 7 of every eight.
+  const int out_col = col0 + ((lane >> 3) & 1);
   float* target = out + (size_t)begin * heads * vdim + (size_t)head * vdim + out_col;
 
   for (int c = 0; c < chunks; ++c) {
@@ -202,27 +226,28 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
     for (int g0 = 0; g0 < n; g0 += 8) {
       float p[16];
       const float* row = tokens + g0 * kPerToken;
-      const float* values = row + 2 * dimp + 2 * group;
+      TokenPart<N> part[2];
+      fetch_part<N>(part[0], row, lane, warp);
       if (n - g0 >= 8) {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
-          const float2 v = *reinterpret_cast<const float2*>(values + i * kPerToken);
-          hgrn2_step<NPL>(S, row + i * kPerToken, v.x, v.y, sub, p[i], p[i + 8]);
+          if (i < 7) fetch_part<N>(part[(i + 1) & 1], row + (i + 1) * kPerToken, lane, warp);
+          hgrn2_step<N>(S, part[i & 1], p[i], p[i + 8]);
         }
       } else {
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
           p[i] = p[i + 8] = 0.f;
           if (g0 + i < n) {
-            const float2 v = *reinterpret_cast<const float2*>(values + i * kPerToken);
-            hgrn2_step<NPL>(S, row + i * kPerToken, v.x, v.y, sub, p[i], p[i + 8]);
+            if (i > 0) fetch_part<N>(part[0], row + i * kPerToken, lane, warp);
+            hgrn2_step<N>(S, part[0], p[i], p[i + 8]);
           }
         }
       }
-      // Sixteen sums over sixteen lanes: lane s ends with sum s.
+      // Sixteen sums over the warp: lane s ends with sum s & 15 of its half, then the halves meet.
 #pragma unroll
       for (int o = 8; o > 0; o >>= 1) {
-        const bool up = (sub & o) != 0;
+        const bool up = (lane & o) != 0;
 #pragma unroll
         for (int i = 0; i < 8; ++i)
           if (i < o) {
@@ -230,8 +255,9 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
             p[i] = keep + __shfl_xor_sync(0xffffffffu, send, o);
           }
       }
-      const int tok = g0 + (sub & 7);
-      if (tok < n && out_col < vdim) target[(size_t)(c * CHUNK + tok) * heads * vdim] = p[0];
+      p[0] += __shfl_xor_sync(0xffffffffu, p[0], 16);
+      const int tok = g0 + (lane & 7);
+      if (lane < 16 && tok < n && out_col < vdim) target[(size_t)(c * CHUNK + tok) * heads * vdim] = p[0];
     }
   }
   grid_launch_dependents();
@@ -239,17 +265,15 @@ hgrn2_steps_kernel(const float* __restrict__ records, float* __restrict__ state,
   for (int c = 0; c < 2; ++c) {
     if (col0 + c >= vdim) continue;
 #pragma unroll
-    for (int j = 0; j < NPL / 4; ++j) {
-      const int at = 4 * (sub + 16 * j);
+    for (int i = 0; i < N; ++i) {
+      const int at = entry_of<N>(i, lane);
       float* p = mine + (size_t)c * dim + at;
-      float v[4];
-      asm("mov.b64 {%0, %1}, %2;" : "=f"(v[0]), "=f"(v[1]) : "l"(S[c][2 * j]));
-      asm("mov.b64 {%0, %1}, %2;" : "=f"(v[2]), "=f"(v[3]) : "l"(S[c][2 * j + 1]));
-      if (vec) { if (at < dim) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+      float2 v;
+      asm("mov.b64 {%0, %1}, %2;" : "=f"(v.x), "=f"(v.y) : "l"(S[c][i]));
+      if (vec) { if (at < dim) *reinterpret_cast<float2*>(p) = v; }
       else {
-#pragma unroll
-        for (int e = 0; e < 4; ++e)
-          if (at + e < dim) p[e] = v[e];
+        if (at < dim) p[0] = v.x;
+        if (at + 1 < dim) p[1] = v.y;
       }
     }
   }
@@ -363,18 +387,18 @@ hgrn2_token_kernel(const T* __restrict__ proj, size_t row_stride, int q_off, int
   for (int i = threadIdx.x; i < vdim; i += 256) o[i] = from_float<T>(os[i] * inv * norm_weight[i]);
 }
 
-template <int NPL, int CHUNK>
+template <int N, int CHUNK>
 int launch_steps(int tokens, int num_seqs, cudaStream_t stream, const float* records, float* state, const int* qsl,
                  const int* slots, float* out, int heads, int dim, int vdim, int vdimp) {
-  constexpr size_t smem = (size_t)kStages * CHUNK * (32 * NPL + kColumns) * sizeof(float);
+  constexpr size_t smem = (size_t)kStages * CHUNK * (128 * N + kColumns) * sizeof(float);
   static bool configured = false;
   if (!configured && smem > 48 * 1024) {
-    cudaError_t e = cudaFuncSetAttribute(hgrn2_steps_kernel<NPL, CHUNK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(hgrn2_steps_kernel<N, CHUNK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  return (int)launch_pdl(tokens, hgrn2_steps_kernel<NPL, CHUNK>, dim3(vdimp / kColumns, heads, num_seqs), dim3(128), smem,
-                         stream, records, state, qsl, slots, out, heads, dim, vdim, vdimp);
+  return (int)launch_pdl(tokens, hgrn2_steps_kernel<N, CHUNK>, dim3(vdimp / kColumns, heads, num_seqs), dim3(kStepThreads),
+                         smem, stream, records, state, qsl, slots, out, heads, dim, vdim, vdimp);
 }
 
 }  // namespace li
@@ -411,13 +435,13 @@ LI_EXPORT int li_hgrn2_steps(int dtype, const void* proj, size_t row_stride, int
     e = launch_pdl(tokens, hgrn2_record_kernel<bf16>, dim3(tokens), dim3(256), 0, stream, (const bf16*)proj, row_stride,
                    q_off, f_off, v_off, f_bias, lower, records, heads, dim, dimp, vdim, vdimp, vec);
   if (e != cudaSuccess) return (int)e;
-#define LI_STEPS(NPL, CHUNK)                                                                                          \
-  return launch_steps<NPL, CHUNK>(tokens, num_seqs, stream, records, state, query_start_loc, state_slots, out, heads, dim, \
+#define LI_STEPS(N, CHUNK)                                                                                            \
+  return launch_steps<N, CHUNK>(tokens, num_seqs, stream, records, state, query_start_loc, state_slots, out, heads, dim, \
                                   vdim, vdimp)
-  if (dimp == 64) LI_STEPS(4, 16);
-  if (dimp == 128) LI_STEPS(8, 16);
-  if (dimp == 256) LI_STEPS(16, 8);
-  LI_STEPS(32, 8);
+  if (dimp == 64) LI_STEPS(1, 16);
+  if (dimp == 128) LI_STEPS(2, 16);
+  if (dimp == 256) LI_STEPS(4, 8);
+  LI_STEPS(8, 8);
 #undef LI_STEPS
 }
 

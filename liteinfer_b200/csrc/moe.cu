@@ -53,6 +53,7 @@ __device__ __forceinline__ int warp_argmax(const float* v, int n, int lane) {
 }
 
 constexpr int kRouteWarps = 4;
+constexpr int kRankedExperts = 64;      // up to this many experts are ranked side by side, more by one arg-max a round
 
 // How a router turns its logits into chosen experts and weights.
 struct RouteRule {
@@ -64,7 +65,7 @@ struct RouteRule {
   const float* correction;    // [experts] or null
 };
 
-__host__ __device__ __forceinline__ int route_floats(int experts, int groups) { return 2 * experts + 2 * groups; }
+__host__ __device__ __forceinline__ int route_floats(int experts, int groups) { return 3 * experts + 2 * groups; }
 
 // One warp routes one token: z [experts] its logits; scratch of `route_floats` floats in shared memory, whose first
 // `experts` places may be z itself.
@@ -75,6 +76,7 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
   float* choice = sc + experts;         // what the choice goes by; -inf: cannot be chosen (any more)
   float* gb = choice + experts;         // the groups' scores
   float* kept = gb + groups;            // 1: the group is kept
+  float* kept_score = kept + groups;    // the chosen experts' scores, the first first
   if (rule.sigmoid) {
     for (int e = lane; e < experts; e += 32) sc[e] = 1.0f / (1.0f + expf(-z[e]));
   } else {
@@ -109,15 +111,33 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
       kept[g] = 0.f;
     }
     __syncwarp();
-    for (int r = 0; r < rule.keep; ++r) {
-      const int g = warp_argmax(gb, groups, lane);
-      __syncwarp();
-      if (lane == 0) { gb[g] = -INFINITY; kept[g] = 1.f; }
-      __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      int before = 0;
+      for (int j = 0; j < groups; ++j) before += gb[j] > gb[g] || (gb[j] == gb[g] && j < g);
+      if (before < rule.keep) kept[g] = 1.f;
     }
+    __syncwarp();
     for (int e = lane; e < experts; e += 32)
       if (kept[e / per] == 0.f) choice[e] = -INFINITY;
     __syncwarp();
+  }
+  if (experts <= kRankedExperts) {
+    // Every lane counts how many experts stand before its own: the place is the rank, with no round after another.
+    for (int e = lane; e < experts; e += 32) {
+      const float mine = choice[e];
+      int before = 0;
+      for (int j = 0; j < experts; ++j) before += choice[j] > mine || (choice[j] == mine && j < e);
+      if (before < rule.top) {
+        ids[(size_t)t * rule.slots + before] = e;
+        kept_score[before] = sc[e];
+      }
+    }
+    __syncwarp();
+    float total = 0.f;
+    for (int r = 0; r < rule.top; ++r) total += kept_score[r];
+    for (int r = lane; r < rule.top; r += 32)
+      weights[(size_t)t * rule.slots + r] = rule.renormalise ? kept_score[r] / (total + rule.floor) : kept_score[r];
+    return;
   }
   float total = 0.f;
   for (int r = 0; r < rule.top; ++r) {
@@ -149,68 +169,84 @@ moe_route_kernel(const float* __restrict__ logits, int tokens, const RouteRule r
 }
 
 // The router's product and the routing in one launch: logits[e] = sum_k x[k] * w[e][k] in 32-bit (lane l adds up
-// k = l, l + 32, ..., then the lanes' sums meet in a fixed tree: the same bits whatever else is in the step), then
-// `route_token`.  A block takes TOK tokens; its warps take the experts in turn: eight warps for eight tokens of a wide
-// step, thirty-two for the one token of a narrow step, where a warp's chain of loads is what the launch waits for.
+// its k in order, then the lanes' sums meet in a fixed tree: the same bits whatever else is in the step), then
+// `route_token`.  A block takes TOK tokens; a warp takes EXP experts at a time, so that a value of x serves EXP products
+// and one of w TOK: eight tokens by four experts in a wide step; in a narrow one, where a warp's chain of loads is what
+// the launch waits for, one token and two experts of as many warps as there are.
 //
 // `gated`: w has one more row, whose logit's sigmoid is a number per token for an expert that every token runs.  It goes
 // to gate[token] (where given) and is the weight of the slots behind the chosen experts, which hold the experts
 // `experts`, `experts` + 1, ...
-template <typename T, int TOK, int kRouterWarps>
-__global__ void __launch_bounds__(kRouterWarps * 32)
+template <typename T, int TOK, int EXP>
+__global__ void __launch_bounds__(TOK == 1 ? 1024 : 512)
 moe_router_kernel(const T* __restrict__ x, size_t x_stride, const float* __restrict__ w, int tokens, int K,
                   const RouteRule rule, int gated, int* __restrict__ ids, float* __restrict__ weights,
                   float* __restrict__ gate) {
   extern __shared__ float route_smem[];       // TOK x (`route_floats`, of which the first are the logits, and the gate's)
-  const int per_token = route_floats(rule.experts, rule.groups) + 1, experts = rule.experts;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int per_token = route_floats(rule.experts, rule.groups) + 1, experts = rule.experts, rows = experts + gated;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int t0 = blockIdx.x * TOK;
   grid_dependency_wait();
   // Four k a lane and round where the rows allow 16-byte reads (several rounds' loads are in flight at once), else one.
   const bool wide = (K % 4) == 0 && (x_stride % 4) == 0 && aligned16(w) && (reinterpret_cast<uintptr_t>(x) % (4 * sizeof(T))) == 0;
-  for (int e = warp; e < experts + gated; e += kRouterWarps) {
-    const float* we = w + (size_t)e * K;
-    float acc[TOK];
+  for (int e0 = warp; e0 < rows; e0 += warps * EXP) {         // this warp's experts: e0, e0 + warps, ...
+    float acc[EXP][TOK];
+    const float* we[EXP];
 #pragma unroll
-    for (int t = 0; t < TOK; ++t) acc[t] = 0.f;
+    for (int i = 0; i < EXP; ++i) {
+      we[i] = w + (size_t)min(e0 + i * warps, rows - 1) * K;  // (past the last row: a row that is computed and dropped)
+#pragma unroll
+      for (int t = 0; t < TOK; ++t) acc[i][t] = 0.f;
+    }
+    const T* xr[TOK];
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) xr[t] = x + (size_t)min(t0 + t, tokens - 1) * x_stride;
     if (wide) {
-#pragma unroll 8
+#pragma unroll(TOK == 1 ? 8 : 1)
       for (int k = lane * 4; k < K; k += 128) {
-        const float4 wv = *reinterpret_cast<const float4*>(we + k);
+        float4 wv[EXP];
+#pragma unroll
+        for (int i = 0; i < EXP; ++i) wv[i] = *reinterpret_cast<const float4*>(we[i] + k);
 #pragma unroll
         for (int t = 0; t < TOK; ++t) {
-          if (t0 + t >= tokens) continue;
-          const T* xr = x + (size_t)(t0 + t) * x_stride + k;
           float x0, x1, x2, x3;
           if (sizeof(T) == 4) {
-            const float4 xv = *reinterpret_cast<const float4*>(xr);
+            const float4 xv = *reinterpret_cast<const float4*>(xr[t] + k);
             x0 = xv.x; x1 = xv.y; x2 = xv.z; x3 = xv.w;
           } else {
-            const uint2 xv = *reinterpret_cast<const uint2*>(xr);
+            const uint2 xv = *reinterpret_cast<const uint2*>(xr[t] + k);
             x0 = __uint_as_float(xv.x << 16); x1 = __uint_as_float(xv.x & 0xffff0000u);
             x2 = __uint_as_float(xv.y << 16); x3 = __uint_as_float(xv.y & 0xffff0000u);
           }
-          acc[t] = fmaf(x3, wv.w, fmaf(x2, wv.z, fmaf(x1, wv.y, fmaf(x0, wv.x, acc[t]))));
+#pragma unroll
+          for (int i = 0; i < EXP; ++i)
+            acc[i][t] = fmaf(x3, wv[i].w, fmaf(x2, wv[i].z, fmaf(x1, wv[i].y, fmaf(x0, wv[i].x, acc[i][t]))));
         }
       }
     } else {
       for (int k = lane; k < K; k += 32) {
-        const float wv = we[k];
 #pragma unroll
-        for (int t = 0; t < TOK; ++t)
-          if (t0 + t < tokens) acc[t] = fmaf(to_float(x[(size_t)(t0 + t) * x_stride + k]), wv, acc[t]);
+        for (int t = 0; t < TOK; ++t) {
+          const float xv = to_float(xr[t][k]);
+#pragma unroll
+          for (int i = 0; i < EXP; ++i) acc[i][t] = fmaf(xv, we[i][k], acc[i][t]);
+        }
       }
     }
 #pragma unroll
-    for (int t = 0; t < TOK; ++t) {
-      const float sum = warp_sum(acc[t]);
-      if (lane == 0) route_smem[t * per_token + (e < experts ? e : per_token - 1)] = sum;
+    for (int i = 0; i < EXP; ++i) {
+      const int e = e0 + i * warps;
+#pragma unroll
+      for (int t = 0; t < TOK; ++t) {
+        const float sum = warp_sum(acc[i][t]);
+        if (lane == 0 && e < rows) route_smem[t * per_token + (e < experts ? e : per_token - 1)] = sum;
+      }
     }
   }
   __syncthreads();
-  if (warp < TOK && t0 + warp < tokens) {
-    float* sc = route_smem + warp * per_token;
-    const int t = t0 + warp;
+  for (int mine = warp; mine < TOK && t0 + mine < tokens; mine += warps) {
+    float* sc = route_smem + mine * per_token;
+    const int t = t0 + mine;
     route_token(sc, sc, lane, t, rule, ids, weights);
     if (gated) {
       const float g = 1.0f / (1.0f + expf(-sc[per_token - 1]));
@@ -581,12 +617,16 @@ LI_EXPORT int li_moe_router(int dtype, const void* x, size_t x_stride, const flo
   const bool wide = tokens > 128;
   const size_t smem = (size_t)(wide ? 8 : 1) * (route_floats(experts, groups) + 1) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
-#define LI_ROUTER(T, TOK, WARPS)                                                                                      \
-  return (int)launch_pdl(tokens, moe_router_kernel<T, TOK, WARPS>, dim3((tokens + TOK - 1) / TOK), dim3(WARPS * 32),   \
+  const int rows = experts + (gated ? 1 : 0);
+  const int most = wide ? 16 : 32;
+  const int wanted = wide ? (rows + 3) / 4 : rows;     // a narrow step: a warp a row as far as they go, then two
+  const int warps = wanted < most ? wanted : most;
+#define LI_ROUTER(T, TOK, EXP)                                                                                        \
+  return (int)launch_pdl(tokens, moe_router_kernel<T, TOK, EXP>, dim3((tokens + TOK - 1) / TOK), dim3(warps * 32),     \
                          smem, stream, (const T*)x, x_stride, w, tokens, K, rule, gated ? 1 : 0, ids, weights, gate)
-  if (dtype == kFloat32) { if (wide) LI_ROUTER(float, 8, 8); LI_ROUTER(float, 1, 32); }
-  if (wide) LI_ROUTER(bf16, 8, 8);
-  LI_ROUTER(bf16, 1, 32);
+  if (dtype == kFloat32) { if (wide) LI_ROUTER(float, 8, 4); LI_ROUTER(float, 1, 2); }
+  if (wide) LI_ROUTER(bf16, 8, 4);
+  LI_ROUTER(bf16, 1, 2);
 #undef LI_ROUTER
 }
 

@@ -233,7 +233,7 @@ class _Scratch:
     ATTENTION_COUNTERS = 1 << 16
     ARGMAX_ROWS = 4096
 
-    def __init__(self, device: torch.device) -> None:
+    def __init__(self, device: torch.device, errors: torch.Tensor | None = None) -> None:
         self.gemm = torch.empty(self.GEMM_FLOATS, dtype=torch.float32, device=device)
         self.gemm_counters = torch.zeros(self.GEMM_COUNTERS, dtype=torch.int32, device=device)
         self.attention_counters = torch.zeros(self.ATTENTION_COUNTERS, dtype=torch.int32, device=device)
@@ -242,12 +242,13 @@ class _Scratch:
         self.argmax_counters = torch.zeros(self.ARGMAX_ROWS, dtype=torch.int32, device=device)
         # Error flags that kernels raise and the engine reads where it synchronises anyway: [0] the number of a
         # bounded wait that gave up (tcgen05 and TMA kernels), [1] a token id outside the embedding table.
-        self.errors = torch.zeros(2, dtype=torch.int32, device=device)
+        self.errors = torch.zeros(2, dtype=torch.int32, device=device) if errors is None else errors
         self.gemm_error = self.errors[0:1]
         self.token_error = self.errors[1:2]
 
 
-_scratch: dict[torch.device, _Scratch] = {}
+_scratch: dict[tuple[torch.device, int], _Scratch] = {}
+_lane = 0           # whose scratch the launches use: 0, or 1 within `beside`
 
 
 def normalise_device(device: torch.device | str) -> torch.device:
@@ -261,10 +262,50 @@ def normalise_device(device: torch.device | str) -> torch.device:
 
 def scratch_for(device: torch.device | str) -> _Scratch:
     device = normalise_device(device)
-    found = _scratch.get(device)
-    if found is None:
-        found = _scratch[device] = _Scratch(device)
+    found = _scratch.get((device, _lane))
+    if found is None:       # (the error flags are one set for all)
+        errors = _scratch[device, 0].errors if (device, 0) in _scratch else None
+        found = _scratch[device, _lane] = _Scratch(device, errors)
+        for lane in (0, 1):
+            if lane != _lane and (device, lane) not in _scratch:
+                _scratch[device, lane] = _Scratch(device, found.errors)
     return found
+
+
+class beside:
+    """Within this context the kernels of this module (and library products) go to a second stream, with scratch of their
+    own, behind what the current stream holds so far; the next `join` on the current stream waits for them.  Two runs of
+    kernels that do not depend on one another share the device that way, in eager steps and inside a captured graph alike.
+    Tensors: what the second stream reads must stay alive until the join, and what it makes is used behind the join."""
+
+    _streams: dict[torch.device, "torch.cuda.Stream"] = {}
+
+    def __init__(self, device: torch.device) -> None:
+        self.device = normalise_device(device)
+        stream = beside._streams.get(self.device)
+        if stream is None:
+            scratch_for(self.device)        # both lanes' buffers exist before a graph is captured
+            stream = beside._streams[self.device] = torch.cuda.Stream(device=self.device)
+        self.stream = stream
+
+    def __enter__(self):
+        global _lane
+        self.stream.wait_stream(torch.cuda.current_stream(self.device))
+        self.entered = (torch.cuda.stream(self.stream), on_current_stream())
+        for context in self.entered:
+            context.__enter__()
+        _lane = 1
+        return self
+
+    def __exit__(self, *exc):
+        global _lane
+        _lane = 0
+        for context in reversed(self.entered):
+            context.__exit__(*exc)
+        return False
+
+    def join(self) -> None:
+        torch.cuda.current_stream(self.device).wait_stream(self.stream)
 
 
 def _ptr(t: torch.Tensor | None) -> int | None:
