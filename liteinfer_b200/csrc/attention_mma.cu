@@ -78,7 +78,7 @@ attention_mma_kernel(const AttnParams p) {
   // Tables and lengths are inputs of the step; what an earlier kernel wrote is read after the wait below.
   const int seq = p.seq_index ? p.seq_index[blockIdx.z] : blockIdx.z;
   if (seq < 0) return;        // a place of padding in the list of sequences
-  const int kvh = (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts;
+  const int kvh = p.v_parts == 1 ? (int)blockIdx.y : (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts;
   // The last query tiles see the most keys: they are handed out first.
   const int split = blockIdx.x % p.num_splits, qtile = (int)(gridDim.x / p.num_splits) - 1 - (int)(blockIdx.x / p.num_splits);
   const int q_begin = p.query_start_loc[seq], q_len = p.query_start_loc[seq + 1] - q_begin;

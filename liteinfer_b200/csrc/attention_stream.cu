@@ -160,7 +160,7 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
 
   const int seq = p.seq_index ? p.seq_index[blockIdx.z] : blockIdx.z;
   if (seq < 0) return;        // a place of padding in the list of sequences
-  const int kvh = (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts, split = blockIdx.x;
+  const int kvh = p.v_parts == 1 ? (int)blockIdx.y : (int)blockIdx.y / p.v_parts, part = (int)blockIdx.y - kvh * p.v_parts, split = blockIdx.x;
   const int q_begin = p.query_start_loc[seq];
   const int groups = p.heads / p.kv_heads;
   const int ctx = p.context_lens[seq];

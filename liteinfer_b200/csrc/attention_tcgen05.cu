@@ -136,7 +136,8 @@ template <int X> constexpr int attn_threads() { return 32 + 32 * X + 128 * X; } 
 
 // kOptions: kept first keys and the soft-cap are compiled in (a kernel of its own, so that the plain one keeps
 // its registers).
-template <int D, int X, bool kOptions>
+// kSpans: chunks instead of a window, and values of several parts, likewise.
+template <int D, int X, bool kOptions, bool kSpans>
 __global__ void __launch_bounds__(attn_threads<X>(), (D == 64 && X == 1) ? 2 : 1)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                          const TcAttnParams p) {
@@ -164,7 +165,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   if (seq < 0) return;        // a place of padding in the list of sequences
   // Values wider than keys: the blocks of a KV head's parts lie side by side, each with all scores and D of a value's
   // dimensions.
-  const int parts = (int)gridDim.x / p.kv_heads, kvh = (int)blockIdx.x / parts, part = (int)blockIdx.x - kvh * parts;
+  const int parts = kSpans ? (int)gridDim.x / p.kv_heads : 1;
+  const int kvh = kSpans ? (int)blockIdx.x / parts : (int)blockIdx.x, part = kSpans ? (int)blockIdx.x - kvh * parts : 0;
   const int q_begin = p.query_start_loc[seq], q_len = p.query_start_loc[seq + 1] - q_begin;
   const int groups = p.heads / p.kv_heads;
   const int tq = kRows / groups;
@@ -176,7 +178,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
   const int block_q = min(X * tq, q_len - block_q0);         // query tokens of the block: its tiles walk the same keys
   const int* table = p.block_table + (size_t)seq * p.table_stride;
   const int hi = ctx - q_len + block_q0 + block_q;
-  const int lo = first_visible(ctx - q_len + block_q0, p.window);
+  const int lo = kSpans ? first_visible(ctx - q_len + block_q0, p.window)
+                 : (p.window > 0 && ctx - q_len + block_q0 - p.window + 1 > 0) ? ctx - q_len + block_q0 - p.window + 1 : 0;
   // The warp's own tile (issuer x is warp 1 + x, its softmax warps are 1 + X + 4 x ...): its queries and positions.
   const int x = X == 1 ? 0 : (warp <= X ? max(warp - 1, 0) : (warp - 1 - X) >> 2);
   const int q0 = block_q0 + x * tq;
@@ -250,7 +253,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
       for (int sub = 0; sub < kSub; ++sub) {
         tma_load_2d(k_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_k, kv_full(stage), sub * 64, row);
-        tma_load_2d(v_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_v, kv_full(stage), part * D + sub * 64, row);
+        tma_load_2d(v_smem + stage * kTileBytes + sub * kKeySubBytes + lane * box_bytes, &map_v, kv_full(stage), (kSpans ? part * D : 0) + sub * 64, row);
       }
     }
     return true;
@@ -352,7 +355,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
     const int row = quarter * 32 + lane;
     const unsigned lane_field = (unsigned)(quarter * 32) << 16;
     const int qpos = row < rows_used ? first_qpos + row / groups : -1;
-    const int row_lo = first_visible(qpos, p.window), last_lo = first_visible(last_qpos, p.window);
+    const int row_lo = kSpans ? first_visible(qpos, p.window) : 0, last_lo = kSpans ? first_visible(last_qpos, p.window) : 0;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
     for (int t = 0; ok && t < ntiles; ++t) {
@@ -373,7 +376,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
           sb[j] = __float_as_uint(p.cap_out * tanh_fast(__uint_as_float(sb[j]) * p.cap_in));
         }
       }
-      const bool all_visible = key0 + kKeys - 1 <= first_qpos && key0 >= last_lo;
+      const bool all_visible = key0 + kKeys - 1 <= first_qpos &&
+                               (kSpans ? key0 >= last_lo : p.window <= 0 || key0 > last_qpos - p.window);
       float mx = m;
       if (all_visible && qpos >= 0) {
         float part[4] = {m, m, m, m};      // four chains, so that the maxima do not wait for one another
@@ -384,8 +388,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
 #pragma unroll
         for (int j = 0; j < 32; ++j) {
           const int ka = key0 + j, kb = key0 + 32 + j;
-          const bool va = ka <= qpos && (ka >= row_lo || (kOptions && ka < p.keep_first));
-          const bool vb = kb <= qpos && (kb >= row_lo || (kOptions && kb < p.keep_first));
+          const bool va = ka <= qpos && ((kSpans ? ka >= row_lo : p.window <= 0 || ka > qpos - p.window) || (kOptions && ka < p.keep_first));
+          const bool vb = kb <= qpos && ((kSpans ? kb >= row_lo : p.window <= 0 || kb > qpos - p.window) || (kOptions && kb < p.keep_first));
           if (!va) sa[j] = __float_as_uint(-INFINITY);
           if (!vb) sb[j] = __float_as_uint(-INFINITY);
           mx = fmaxf(mx, fmaxf(__uint_as_float(sa[j]), __uint_as_float(sb[j])));
@@ -461,7 +465,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid
       // (Compiled into the kernel's form with options only, so that the plain form is what it was.)
       if (kOptions && p.sink != nullptr && row < rows_used) l += exp2f(p.sink[head] * kLog2eF - m * p.scale_log2);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + ((size_t)head * parts + part) * D;
+      bf16* dst = p.out + (size_t)(q_begin + qi) * p.out_row_stride + (kSpans ? (size_t)head * parts + part : (size_t)head) * D;
 #pragma unroll
       for (int half = 0; half < D / 32; ++half) {
         unsigned o[32];
@@ -520,18 +524,23 @@ static bool make_pool_map(CUtensorMap* map, const void* pool, long rows, int pag
   return true;
 }
 
-template <int D, int X, bool kOptions>
+template <int D, int X, bool kOptions, bool kSpans>
 static int launch_tc_attention_as(const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnParams& p, dim3 grid,
                                   cudaStream_t stream);
 
 template <int D, int X>
 static int launch_tc_attention(const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnParams& p, dim3 grid,
                                cudaStream_t stream) {
-  return (p.keep_first > 0 || p.cap_out > 0.f || p.sink != nullptr) ? launch_tc_attention_as<D, X, true>(mk, mv, p, grid, stream)
-                                                : launch_tc_attention_as<D, X, false>(mk, mv, p, grid, stream);
+  const bool options = p.keep_first > 0 || p.cap_out > 0.f || p.sink != nullptr;
+  const bool spans = p.window < 0 || (int)grid.x != p.kv_heads;
+  if (spans)
+    return options ? launch_tc_attention_as<D, X, true, true>(mk, mv, p, grid, stream)
+                   : launch_tc_attention_as<D, X, false, true>(mk, mv, p, grid, stream);
+  return options ? launch_tc_attention_as<D, X, true, false>(mk, mv, p, grid, stream)
+                 : launch_tc_attention_as<D, X, false, false>(mk, mv, p, grid, stream);
 }
 
-template <int D, int X, bool kOptions>
+template <int D, int X, bool kOptions, bool kSpans>
 static int launch_tc_attention_as(const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnParams& p, dim3 grid,
                                   cudaStream_t stream) {
   constexpr int kKvStages = KvStages<D, X>::value;
@@ -540,11 +549,11 @@ static int launch_tc_attention_as(const CUtensorMap& mk, const CUtensorMap& mv, 
   static_assert(smem <= 232448, "more shared memory than a block may have");
   static bool configured = false;
   if (!configured) {
-    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<D, X, kOptions>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(attention_tcgen05_kernel<D, X, kOptions, kSpans>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     configured = true;
   }
-  return (int)launch_pdl(0, attention_tcgen05_kernel<D, X, kOptions>, grid, dim3(attn_threads<X>()), smem, stream, mk, mv, p);
+  return (int)launch_pdl(0, attention_tcgen05_kernel<D, X, kOptions, kSpans>, grid, dim3(attn_threads<X>()), smem, stream, mk, mv, p);
 }
 
 }  // namespace li

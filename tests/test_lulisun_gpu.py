@@ -508,6 +508,32 @@ def test_bfloat16_engine_keeps_32_bit_what_must_be_and_rounds_heads_up(lulisun_d
     assert runner.layer_caches[0].kv.k_pool.shape[-1] == 64 and runner.layer_caches[0].kv.v_pool.shape[-1] == 192
 
 
+@pytest.mark.parametrize("graphs", [False, True])
+@pytest.mark.parametrize("name", ["lul_c", "lul_e"])
+def test_sublayers_side_by_side_equal_one_after_the_other(lulisun_dirs, monkeypatch, name, graphs):
+    """The feed-forward on a second stream (its experts, and a shared expert whose products use scratch of their own)
+    gives what one stream gives, step for step, eager and from graphs."""
+    from liteinfer_b200.engine.loading import build_runner
+    from liteinfer_b200.engine.runner import StepEntry
+    from liteinfer_b200.parts import block
+
+    config = lc.ALL[name][0]
+    tokens = [lc.prompt(config["vocab"], 90, 60 + i) for i in range(3)]
+    results = []
+    for limit in (0, 256):
+        monkeypatch.setattr(block, "PARALLEL_SUBLAYERS", limit)
+        runner = build_runner(lulisun_dirs[name], torch.bfloat16, DEV, 16, 32, 3)
+        if graphs:
+            runner.enable_decode_graphs(3, 512)
+        got = [runner.step([StepEntry(str(i), t[:70 + i], [69 + i]) for i, t in enumerate(tokens)]).clone()]
+        for at in range(74, 90):
+            got.append(runner.step([StepEntry(str(i), t[at:at + 1], [0]) for i, t in enumerate(tokens)]).clone())
+        runner.check_kernels()
+        results.append(torch.cat(got))
+    assert torch.isfinite(results[0].float()).all()
+    torch.testing.assert_close(results[1].float(), results[0].float(), rtol=2 ** -6, atol=2 ** -6)
+
+
 def test_greedy_generation_through_the_engine_on_gpu(lulisun_dirs):
     """`LLM.generate` (scheduler with portions of 16 tokens, three seats for five requests, CUDA graphs, sampler) picks the
     plain implementation's tokens over 24 decoded tokens, chunks ending among them."""
