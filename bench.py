@@ -889,7 +889,7 @@ def _lulisun_kernels(peaks: dict) -> dict:
         return _timed(graph.replay, repeats=10, warmup=2) / inner
 
     # -- chunked attention (16 / 4 heads of 128, chunks of 1,024) beside a sliding window of 1,024 with a sink; values as
-    #    wide as keys, twice as wide, and heads of 96 with values of 192 (rounded up to 128 and 256)
+    #    wide as keys, twice as wide, and heads of 112 with values of 224 (rounded up to 128 and 256)
     H, kv_heads, page, n, span = 16, 4, 16, 2048, 1024
     pages = n // page
     sink = torch.zeros(H, device=dev)
@@ -898,7 +898,7 @@ def _lulisun_kernels(peaks: dict) -> dict:
     cases = (("chunked_attention", 128, 128, 128, 128, dict(chunk=span), chunked),
              ("kutolix_attention", 128, 128, 128, 128, dict(window=span, sink=sink), windowed),
              ("chunked_attention_values256", 128, 256, 128, 256, dict(chunk=span), chunked),
-             ("chunked_attention_96_192", 128, 256, 96, 192, dict(chunk=span), chunked))
+             ("chunked_attention_112_224", 128, 256, 112, 224, dict(chunk=span), chunked))
     for name, hd, vd, dim, vdim, extra, pairs in cases:
         k_pool = torch.randn(pages * 64, kv_heads, page, hd, device=dev).to(bf)
         v_pool = torch.randn(pages * 64, kv_heads, page, vd, device=dev).to(bf)

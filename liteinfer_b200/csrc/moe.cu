@@ -152,8 +152,8 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
     }
     __syncwarp();
   }
-  if (rule.renormalise && lane < rule.top)     // (top <= 32 where this is asked for)
-    weights[(size_t)t * rule.slots + lane] /= total + rule.floor;
+  if (rule.renormalise)
+    for (int r = lane; r < rule.top; r += 32) weights[(size_t)t * rule.slots + r] /= total + rule.floor;
 }
 
 __global__ void __launch_bounds__(kRouteWarps * 32)
@@ -569,7 +569,7 @@ using namespace li;
 
 static bool bad_rule(const RouteRule& r) {
   return r.experts < 1 || r.top < 1 || r.top > r.experts || r.groups < 1 || r.experts % r.groups || r.keep < 1 ||
-         r.keep > r.groups || r.keep * (r.experts / r.groups) < r.top || (r.renormalise && r.top > 32) || r.slots < r.top;
+         r.keep > r.groups || r.keep * (r.experts / r.groups) < r.top || r.slots < r.top;
 }
 
 // logits [tokens, experts] float; ids [tokens, top] int; weights [tokens, top] float.  sigmoid, pair_rank, floor,

@@ -307,7 +307,7 @@ def test_sum_and_norms(dtype, width):
 
 # ------------------------------------------------------------------ the router and the experts
 @pytest.mark.parametrize("experts,top,groups,keep", [(6, 2, 3, 2), (12, 4, 4, 2), (8, 2, 4, 1), (64, 6, 8, 3), (5, 2, 1, 1),
-                                                      (3, 1, 1, 1), (256, 8, 8, 4), (4, 4, 2, 2), (6, 3, 6, 4), (96, 5, 3, 1)])
+                                                      (3, 1, 1, 1), (256, 8, 8, 4), (4, 4, 2, 2), (6, 3, 6, 4), (96, 5, 3, 1), (128, 40, 2, 1), (64, 40, 1, 1)])
 def test_corrected_router_against_the_plain_mechanism(experts, top, groups, keep):
     """Scores whose corrections change the choice, negative choice scores among them, groups ranked by their two best."""
     from liteinfer_b200 import ops
