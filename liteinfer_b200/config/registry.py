@@ -41,6 +41,7 @@ def _builtins() -> None:
     import liteinfer_b200.architectures.kutolix  # noqa: F401  (registers Kutolix)
     import liteinfer_b200.architectures.lulisun  # noqa: F401  (registers Lulisun)
     import liteinfer_b200.architectures.llama  # noqa: F401  (registers LlamaForCausalLM)
+    import liteinfer_b200.architectures.sogazen  # noqa: F401  (registers Sogazen)
 
 
 def architecture_name(raw: dict[str, Any], where: str = "config.json") -> str:

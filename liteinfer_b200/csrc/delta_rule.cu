@@ -1,7 +1,7 @@
 // The gated delta rule and the short convolutions in front of it.
 //
-//   li_short_conv         y[t, c] = act(sum_m w[m, c] * x[t - (K-1-m), c]): a causal convolution over time per
-//                         channel (the taps tap by tap, [K, channels], so that neighbouring channels' weights are
+//   li_short_conv         y[t, c] = act(b[c] + sum_m w[m, c] * x[t - (K-1-m), c]), b optional: a causal convolution over
+//                         time per channel (the taps tap by tap, [K, channels], so that neighbouring channels' weights are
 //                         neighbours); inputs before the step come from the request's tail (its last K-1 inputs)
 //   li_short_conv_update  moves every request's tail on by the step's inputs
 //   li_gated_delta_rule   per request and head a state S [dim, vdim] in 32-bit (kept column by column); per token
@@ -27,7 +27,7 @@ template <typename T>
 __global__ void short_conv_kernel(const T* __restrict__ x, size_t x_stride, const T* __restrict__ taps,
                                   const T* __restrict__ tail, const int* __restrict__ seq_of_token,
                                   const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
-                                  T* __restrict__ out, int channels, int K, int act) {
+                                  T* __restrict__ out, int channels, int K, int act, const float* __restrict__ bias) {
   grid_dependency_wait();
   const int t = blockIdx.x;
   const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -39,7 +39,7 @@ __global__ void short_conv_kernel(const T* __restrict__ x, size_t x_stride, cons
   }
   const int j = t - query_start_loc[seq];   // index of the token among its sequence's tokens of this step
   const T* old = tail + (size_t)state_slots[seq] * (K - 1) * channels;
-  float acc = 0.f;
+  float acc = bias != nullptr ? bias[c] : 0.f;
   for (int m = 0; m < K; ++m) {
     const int back = K - 1 - m;
     const float in = back <= j ? to_float(x[(size_t)(t - back) * x_stride + c])
@@ -56,7 +56,8 @@ template <typename T>
 __global__ void short_conv_vec_kernel(const T* __restrict__ x, size_t x_stride, const T* __restrict__ taps,
                                       const T* tail, const int* __restrict__ seq_of_token,
                                       const int* __restrict__ query_start_loc, const int* __restrict__ state_slots,
-                                      T* __restrict__ out, int channels, int K, int act, T* move_tail) {
+                                      T* __restrict__ out, int channels, int K, int act, T* move_tail,
+                                      const float* __restrict__ bias) {
   // move_tail (only where every sequence of the step brings one token): the tail is also moved on here, by the
   // thread that has just read all of it for its channels (tail and move_tail are the same memory).
   constexpr int N = Vec16<T>::N;
@@ -77,7 +78,7 @@ __global__ void short_conv_vec_kernel(const T* __restrict__ x, size_t x_stride, 
   grid_dependency_wait();
   float acc[N];
 #pragma unroll
-  for (int e = 0; e < N; ++e) acc[e] = 0.f;
+  for (int e = 0; e < N; ++e) acc[e] = bias != nullptr ? bias[c + e] : 0.f;
   for (int m = 0; m < K; ++m) {
     const int back = K - 1 - m;
     const Vec16<T> in = back <= j ? load16(x + (size_t)(t - back) * x_stride + c)
@@ -525,7 +526,8 @@ using namespace li;
 
 LI_EXPORT int li_short_conv(int dtype, const void* x, size_t x_stride, const void* taps, const void* tail,
                             const int* seq_of_token, const int* query_start_loc, const int* state_slots, void* out,
-                            int tokens, int channels, int K, int act, int move_tail, cudaStream_t stream) {
+                            int tokens, int channels, int K, int act, int move_tail, const float* bias,
+                            cudaStream_t stream) {
   if (tokens <= 0 || channels <= 0) return 0;
   if (K < 1 || K > kMaxTaps || (K > 1 && tail == nullptr) || (channels + 127) / 128 > 65535) return LI_ERR_UNSUPPORTED;
   // move_tail: every sequence of the step brings exactly one token and the caller wants the tail moved on by
@@ -538,20 +540,20 @@ LI_EXPORT int li_short_conv(int dtype, const void* x, size_t x_stride, const voi
     if (dtype == kFloat32)
       return (int)launch_pdl(tokens, short_conv_vec_kernel<float>, vgrid, dim3(128), 0, stream, (const float*)x, x_stride,
                              (const float*)taps, (const float*)tail, seq_of_token, query_start_loc, state_slots,
-                             (float*)out, channels, K, act, move_tail ? (float*)tail : (float*)nullptr);
+                             (float*)out, channels, K, act, move_tail ? (float*)tail : (float*)nullptr, bias);
     return (int)launch_pdl(tokens, short_conv_vec_kernel<bf16>, vgrid, dim3(128), 0, stream, (const bf16*)x, x_stride,
                            (const bf16*)taps, (const bf16*)tail, seq_of_token, query_start_loc, state_slots, (bf16*)out,
-                           channels, K, act, move_tail ? (bf16*)tail : (bf16*)nullptr);
+                           channels, K, act, move_tail ? (bf16*)tail : (bf16*)nullptr, bias);
   }
   if (move_tail) return LI_ERR_UNSUPPORTED;
   const dim3 grid(tokens, (channels + 127) / 128);
   if (dtype == kFloat32)
     return (int)launch_pdl(tokens, short_conv_kernel<float>, grid, dim3(128), 0, stream, (const float*)x, x_stride,
                            (const float*)taps, (const float*)tail, seq_of_token, query_start_loc, state_slots,
-                           (float*)out, channels, K, act);
+                           (float*)out, channels, K, act, bias);
   return (int)launch_pdl(tokens, short_conv_kernel<bf16>, grid, dim3(128), 0, stream, (const bf16*)x, x_stride,
                          (const bf16*)taps, (const bf16*)tail, seq_of_token, query_start_loc, state_slots, (bf16*)out,
-                         channels, K, act);
+                         channels, K, act, bias);
 }
 
 LI_EXPORT int li_short_conv_update(int dtype, const void* x, size_t x_stride, void* tail, const int* query_start_loc,

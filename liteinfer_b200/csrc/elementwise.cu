@@ -160,6 +160,19 @@ __device__ __forceinline__ float activate(float x, int act) {
   }
 }
 
+// act(gate) * up, the activation rounded before the multiply; or (kCapped) the capped form, all of it in 32-bit: with
+// g' = min(g, limit), g' * sigmoid(alpha g') * (clamp(u, -limit, limit) + 1).
+constexpr int kCapped = 4;
+template <typename T>
+__device__ __forceinline__ float gated(float g, float u, int act, float limit, float alpha) {
+  if (act == kCapped) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
+  }
+  return round_to<T>(activate(g, act)) * u;
+}
+
 // out[i] = act(x[i]): the activation of a feed-forward that has no gate.
 template <typename T>
 __global__ void activation_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n, int act) {
@@ -189,7 +202,8 @@ __global__ void softcap_kernel(T* __restrict__ x, size_t n, float cap, float inv
 
 // gate_up [rows, 2*width]: gate in the first `width` columns, up in the rest.
 template <typename T>
-__global__ void act_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t rows, int width, int act) {
+__global__ void act_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t rows, int width, int act,
+                               float limit, float alpha) {
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t n = rows * (size_t)width, stride = (size_t)gridDim.x * blockDim.x;
   for (; i < n; i += stride) {
@@ -197,12 +211,13 @@ __global__ void act_mul_kernel(const T* __restrict__ gate_up, T* __restrict__ ou
     const int c = (int)(i - r * width);
     const float g = to_float(gate_up[r * 2 * width + c]);
     const float u = to_float(gate_up[r * 2 * width + width + c]);
-    out[i] = from_float<T>(round_to<T>(activate(g, act)) * u);
+    out[i] = from_float<T>(gated<T>(g, u, act, limit, alpha));
   }
 }
 
 template <typename T>
-__global__ void act_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t rows, int width, int act) {
+__global__ void act_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t rows, int width, int act,
+                                   float limit, float alpha) {
   constexpr int N = Vec16<T>::N;
   const int vec_per_row = width / N;
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -214,7 +229,7 @@ __global__ void act_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict_
     const Vec16<T> u = load16(gate_up + r * 2 * width + width + c);
     Vec16<T> o;
 #pragma unroll
-    for (int k = 0; k < N; ++k) o.set(k, round_to<T>(activate(g.get(k), act)) * u.get(k));
+    for (int k = 0; k < N; ++k) o.set(k, gated<T>(g.get(k), u.get(k), act, limit, alpha));
     store16(out + r * width + c, o);
   }
 }
@@ -223,7 +238,7 @@ __global__ void act_mul_vec_kernel(const T* __restrict__ gate_up, T* __restrict_
 // [8b, 8b+8), columns [16b+8, 16b+16) the matching up columns (the layout of the fused product's weights).
 template <typename T>
 __global__ void act_mul_interleaved_kernel(const T* __restrict__ gate_up, T* __restrict__ out, size_t rows, int width,
-                                           int act) {
+                                           int act, float limit, float alpha) {
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t n = rows * (size_t)width, stride = (size_t)gridDim.x * blockDim.x;
   for (; i < n; i += stride) {
@@ -232,14 +247,14 @@ __global__ void act_mul_interleaved_kernel(const T* __restrict__ gate_up, T* __r
     const size_t base = r * 2 * width + (size_t)(c / 8) * 16 + (c % 8);
     const float g = to_float(gate_up[base]);
     const float u = to_float(gate_up[base + 8]);
-    out[i] = from_float<T>(round_to<T>(activate(g, act)) * u);
+    out[i] = from_float<T>(gated<T>(g, u, act, limit, alpha));
   }
 }
 
 // The same for bfloat16 with 16-byte accesses: one thread takes one group of eight gate values and the eight
 // up values behind them.
 __global__ void act_mul_interleaved_vec_kernel(const bf16* __restrict__ gate_up, bf16* __restrict__ out, size_t rows,
-                                               int width, int act) {
+                                               int width, int act, float limit, float alpha) {
   const int groups = width / 8;
   size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   const size_t n = rows * (size_t)groups, stride = (size_t)gridDim.x * blockDim.x;
@@ -251,7 +266,7 @@ __global__ void act_mul_interleaved_vec_kernel(const bf16* __restrict__ gate_up,
     const Vec16<bf16> u = load16(src + 8);
     Vec16<bf16> o;
 #pragma unroll
-    for (int k = 0; k < 8; ++k) o.set(k, round_to<bf16>(activate(g.get(k), act)) * u.get(k));
+    for (int k = 0; k < 8; ++k) o.set(k, gated<bf16>(g.get(k), u.get(k), act, limit, alpha));
     store16(out + r * width + (size_t)b * 8, o);
   }
 }
@@ -290,14 +305,16 @@ int launch_rmsnorm(void* x, const void* delta, const void* weight, void* out, co
 }
 
 template <typename T>
-int launch_act_mul(const void* gate_up, void* out, size_t rows, int width, int act, cudaStream_t s) {
+int launch_act_mul(const void* gate_up, void* out, size_t rows, int width, int act, float limit, float alpha,
+                   cudaStream_t s) {
   if (rows == 0) return 0;
   constexpr int N = Vec16<T>::N;
   if (width % N == 0 && aligned16(gate_up) && aligned16(out)) {
     const size_t n = rows * (size_t)(width / N);
-    act_mul_vec_kernel<T><<<grid_for(n, 256), 256, 0, s>>>((const T*)gate_up, (T*)out, rows, width, act);
+    act_mul_vec_kernel<T><<<grid_for(n, 256), 256, 0, s>>>((const T*)gate_up, (T*)out, rows, width, act, limit, alpha);
   } else {
-    act_mul_kernel<T><<<grid_for(rows * (size_t)width, 256), 256, 0, s>>>((const T*)gate_up, (T*)out, rows, width, act);
+    act_mul_kernel<T><<<grid_for(rows * (size_t)width, 256), 256, 0, s>>>((const T*)gate_up, (T*)out, rows, width, act, limit,
+                                                                          alpha);
   }
   LI_LAUNCH_CHECK();
 }
@@ -387,29 +404,29 @@ LI_EXPORT int li_add_bias(int dtype, void* out, const void* bias, size_t rows, i
   LI_LAUNCH_CHECK();
 }
 
-// out[r, c] = act(gate_up[r, c]) * gate_up[r, width + c];  act: 0 silu, 1 gelu (erf), 2 gelu (tanh), 3 relu.
-LI_EXPORT int li_act_mul(int dtype, const void* gate_up, void* out, size_t rows, int width, int act,
+// out[r, c] = act(gate_up[r, c]) * gate_up[r, width + c];  act: 0 silu, 1 gelu (erf), 2 gelu (tanh), 3 relu, 4 the capped form.
+LI_EXPORT int li_act_mul(int dtype, const void* gate_up, void* out, size_t rows, int width, int act, float limit, float alpha,
                          cudaStream_t stream) {
-  if (act < 0 || act > 3) return LI_ERR_UNSUPPORTED;
-  return dtype == kFloat32 ? launch_act_mul<float>(gate_up, out, rows, width, act, stream)
-                           : launch_act_mul<bf16>(gate_up, out, rows, width, act, stream);
+  if (act < 0 || act > 4) return LI_ERR_UNSUPPORTED;
+  return dtype == kFloat32 ? launch_act_mul<float>(gate_up, out, rows, width, act, limit, alpha, stream)
+                           : launch_act_mul<bf16>(gate_up, out, rows, width, act, limit, alpha, stream);
 }
 
 // As li_act_mul for a gate_up interleaved in eights; width must be a multiple of 8.
 LI_EXPORT int li_act_mul_interleaved(int dtype, const void* gate_up, void* out, size_t rows, int width, int act,
-                                     cudaStream_t stream) {
-  if (act < 0 || act > 3 || (width % 8)) return LI_ERR_UNSUPPORTED;
+                                     float limit, float alpha, cudaStream_t stream) {
+  if (act < 0 || act > 4 || (width % 8)) return LI_ERR_UNSUPPORTED;
   if (rows == 0) return 0;
   const size_t n = rows * (size_t)width;
   if (dtype == kFloat32)
     act_mul_interleaved_kernel<float><<<grid_for(n, 256), 256, 0, stream>>>((const float*)gate_up, (float*)out, rows,
-                                                                            width, act);
+                                                                            width, act, limit, alpha);
   else if (aligned16(gate_up) && aligned16(out))
     act_mul_interleaved_vec_kernel<<<grid_for(n / 8, 256), 256, 0, stream>>>((const bf16*)gate_up, (bf16*)out, rows,
-                                                                             width, act);
+                                                                             width, act, limit, alpha);
   else
     act_mul_interleaved_kernel<bf16><<<grid_for(n, 256), 256, 0, stream>>>((const bf16*)gate_up, (bf16*)out, rows,
-                                                                          width, act);
+                                                                          width, act, limit, alpha);
   LI_LAUNCH_CHECK();
 }
 

@@ -47,7 +47,8 @@ LI_EXPORT int li_gemm_skinny_plan(int N, int K, int* warps, int* slice_k) { retu
 // (unsigned, all zero) are needed when li_gemm_skinny_plan(N, K) > 1: scratch_floats must be at least
 // tiles * slices * 16 * 8 * ceil(M/8) and num_counters at least tiles, with tiles = ceil(N/16).
 // gated_act: -1 plain; 16 + a: plain, then the activation a of one argument (4: the square of relu);
-// 0 silu, 1 gelu, 2 gelu-tanh, 3 relu on rows interleaved in eights (N a multiple of 16);
+// 0 silu, 1 gelu, 2 gelu-tanh, 3 relu, 4 the capped form with `limit` and `alpha` on rows interleaved in eights (N a
+// multiple of 16);
 // out is then [M, N/2].
 static int run_skinny(SkinnyParams p, float* scratch, size_t scratch_floats, unsigned* counters, int num_counters,
                       cudaStream_t stream) {
@@ -85,7 +86,7 @@ static int run_skinny(SkinnyParams p, float* scratch, size_t scratch_floats, uns
 }
 
 LI_EXPORT int li_gemm_skinny(const void* x, const void* w, const void* bias, void* out, int M, int N, int K,
-                             int gated_act, float* scratch, size_t scratch_floats, unsigned* counters,
+                             int gated_act, float limit, float alpha, float* scratch, size_t scratch_floats, unsigned* counters,
                              int num_counters, cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   if (M > 64 || K < 8 || (K % 8)) return LI_ERR_UNSUPPORTED;
@@ -93,6 +94,8 @@ LI_EXPORT int li_gemm_skinny(const void* x, const void* w, const void* bias, voi
   if (!aligned16(x) || !aligned16(w)) return LI_ERR_ALIGNMENT;
   SkinnyParams p{(const bf16*)x, (const bf16*)w, (const bf16*)bias, (bf16*)out, M, N, K, 0, 1, gated_act,
                  scratch, counters};
+  p.limit = limit;
+  p.alpha = alpha;
   return run_skinny(p, scratch, scratch_floats, counters, num_counters, stream);
 }
 

@@ -43,6 +43,13 @@ __device__ __forceinline__ float gated(float gate, float up, int act) {
   }
   return __bfloat162float(__float2bfloat16_rn(a)) * up;   // the activation is rounded before the multiply
 }
+// The capped form (gated_act 4), all of it in 32-bit: with g' = min(g, L), g' * sigmoid(alpha g') * (clamp(u, -L, L) + 1).
+constexpr int kCappedGate = 4;
+__device__ __forceinline__ float capped_gate(float gate, float up, float limit, float alpha) {
+  gate = fminf(gate, limit);
+  up = fminf(fmaxf(up, -limit), limit);
+  return gate * (1.0f / (1.0f + expf(-alpha * gate))) * (up + 1.0f);
+}
 
 // `gated_act` values from kUnaryActBase on ask for a plain product whose result, rounded to bfloat16 as a separate
 // kernel would see it, goes through an activation of one argument: base + 0 silu, 1 gelu, 2 gelu-tanh, 3 relu,
@@ -59,7 +66,7 @@ __device__ __forceinline__ float unary_act(float v, int act) {
   }
 }
 // Whether a `gated_act` is one the kernels know, and whether it leaves the output as wide as the weight has rows.
-inline bool act_code_known(int gated_act) { return gated_act <= 3 || (gated_act >= kUnaryActBase && gated_act <= kUnaryActLast); }
+inline bool act_code_known(int gated_act) { return gated_act <= kCappedGate || (gated_act >= kUnaryActBase && gated_act <= kUnaryActLast); }
 __host__ __device__ __forceinline__ bool act_is_plain(int gated_act) { return gated_act < 0 || gated_act >= kUnaryActBase; }
 
 struct SkinnyParams {
@@ -87,6 +94,7 @@ struct SkinnyParams {
   // out_sumsq[tile * out_stride + m] receives the sum of the squares of the tile's 16 new values of row m.
   float* out_sumsq = nullptr;
   int out_stride = 0;
+  float limit = 0.f, alpha = 1.f;       // of the capped form
 };
 
 // a * b for two pairs of bfloat16, each product rounded to bfloat16 (exact product, one rounding).
@@ -312,6 +320,10 @@ gemm_skinny_kernel(const SkinnyParams p) {
       if (p.bias) {
         gate += __bfloat162float(p.bias[row0 + r]);
         up += __bfloat162float(p.bias[row0 + r + 8]);
+      }
+      if (p.gated_act == kCappedGate) {
+        p.out[(size_t)m * half + n] = __float2bfloat16_rn(capped_gate(gate, up, p.limit, p.alpha));
+        continue;
       }
       // The products are rounded to bfloat16 before the activation, as a separate kernel would see them.
       gate = __bfloat162float(__float2bfloat16_rn(gate));

@@ -43,6 +43,7 @@ struct StreamParams {
   float* out_sumsq;   // not null: out is added to, and [tiles][out_stride] receives the new rows' sums of squares
   int out_stride;
   int* error_flag;
+  float limit, alpha; // of the capped form
 };
 
 __device__ __forceinline__ uint4 lds128(unsigned addr) {
@@ -90,6 +91,10 @@ __device__ __forceinline__ void finish_tile(const StreamParams& p, int tile, int
       if (p.bias) {
         gate += __bfloat162float(p.bias[row0 + r]);
         up += __bfloat162float(p.bias[row0 + r + 8]);
+      }
+      if (p.gated_act == kCappedGate) {
+        p.out[(size_t)m * half + col] = __float2bfloat16_rn(capped_gate(gate, up, p.limit, p.alpha));
+        continue;
       }
       // The products are rounded to bfloat16 before the activation, as a separate kernel would see them.
       gate = __bfloat162float(__float2bfloat16_rn(gate));
@@ -374,7 +379,8 @@ LI_EXPORT int li_gemm_stream_supports(int M, int N, int K) { return M >= 1 && M 
 // out = round(out + round(product + bias)), and out_sumsq [ceil(N/16)][out_stride] receives the new rows' sums of
 // squares, one part per 16 columns.  error_flag (device int, may be null): set to 31 if a wait for weights gave up.
 LI_EXPORT int li_gemm_stream(const void* x, const void* w, const void* bias, void* out, int M, int N, int K,
-                             int gated_act, float* out_sumsq, int out_stride, int* error_flag, cudaStream_t stream) {
+                             int gated_act, float limit, float alpha, float* out_sumsq, int out_stride, int* error_flag,
+                             cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
   if (!li_gemm_stream_supports(M, N, K)) return LI_ERR_UNSUPPORTED;
   if (!act_code_known(gated_act) || (!act_is_plain(gated_act) && (N % 16))) return LI_ERR_UNSUPPORTED;
@@ -382,6 +388,6 @@ LI_EXPORT int li_gemm_stream(const void* x, const void* w, const void* bias, voi
   if (!aligned16(x) || !aligned16(w)) return LI_ERR_ALIGNMENT;
   CUtensorMap map;
   if (!make_weight_map(&map, w, N, K)) return LI_ERR_UNSUPPORTED;
-  StreamParams p{(const bf16*)x, (const bf16*)bias, (bf16*)out, M, N, K, gated_act, out_sumsq, out_stride, error_flag};
+  StreamParams p{(const bf16*)x, (const bf16*)bias, (bf16*)out, M, N, K, gated_act, out_sumsq, out_stride, error_flag, limit, alpha};
   return M <= 8 ? plan_and_launch<1>(map, p, stream) : plan_and_launch<2>(map, p, stream);
 }

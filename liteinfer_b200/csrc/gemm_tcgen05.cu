@@ -32,7 +32,7 @@ constexpr int kUmmaK = 16;
 constexpr int kGemmThreads = 192;          // loader, issuer, four epilogue warps
 constexpr int kPairThreads = 320;          // the kernel for pairs of CTAs: loader, issuer, eight epilogue warps
 __device__ __forceinline__ float gated_value(float gate, float up, int act);
-// With an expert's capped form (act 4), all of it in 32-bit: min(g, L) * sigmoid(alpha * min(g, L)) * (clamp(u, -L, L) + 1).
+// With the capped form (act 4), all of it in 32-bit: min(g, L) * sigmoid(alpha * min(g, L)) * (clamp(u, -L, L) + 1).
 __device__ __forceinline__ float gated_value(float gate, float up, int act, float limit, float alpha) {
   if (act == 4) {
     gate = fminf(gate, limit);
@@ -71,6 +71,7 @@ struct GemmParams {
   int M, N, K;
   int gated_act;
   int* error_flag;
+  float limit = 0.f, alpha = 1.f;       // of gated_act 4
 };
 
 // A product grouped by expert (tile_expert != null; the single-CTA kernel only, as a parameter of its own so that the
@@ -86,14 +87,22 @@ struct GroupParams {
   // out[m] is multiplied by row_scale[row_of[m]] where row_scale is given (an expert's output times its weight).
   const int* row_of;
   const float* row_scale;
-  float limit, alpha;           // of gated_act 4
 };
+
+// An element of a product grouped by expert that has no gate: times its row's scale, or (gated_act -2) relu and its square.
+__device__ __forceinline__ float grouped_value(float v, float scale, int gated_act) {
+  if (gated_act == -2) {
+    v = fmaxf(v, 0.f);
+    return v * v;
+  }
+  return v * scale;
+}
 
 // 32 consecutive columns of one output row, from the accumulator's registers to global memory: rounded to
 // bfloat16 (with the bias), or for a gated feed-forward two groups of (eight gate, eight up) columns turned into
 // 16 outputs.  The caller has checked m < M and n0 < N.
-// `kGrouped`: the ways out that only a product grouped by expert has (a row's scale, the experts' capped activation)
-// are compiled into that form alone, so the plain product's epilogue is what it was.
+// `kGrouped`: the ways out that only a product grouped by expert has (a row's scale, the square of relu) are compiled into
+// that form alone, so the plain product's epilogue is what it was.
 template <bool kGrouped>
 __device__ __forceinline__ void store_chunk(const GemmParams& p, const GroupParams& g, const unsigned (&r)[32], int m,
                                             int n0) {
@@ -108,7 +117,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const GroupPara
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           float lo = __uint_as_float(r[v * 8 + 2 * j]), hi = __uint_as_float(r[v * 8 + 2 * j + 1]);
-          if (kGrouped) { lo *= scale; hi *= scale; }
+          if (kGrouped) { lo = grouped_value(lo, scale, p.gated_act); hi = grouped_value(hi, scale, p.gated_act); }
           if (p.bias) {
             lo += __bfloat162float(p.bias[n0 + v * 8 + 2 * j]);
             hi += __bfloat162float(p.bias[n0 + v * 8 + 2 * j + 1]);
@@ -123,7 +132,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const GroupPara
       for (int j = 0; j < 32; ++j) {
         if (n0 + j < p.N) {
           float v = __uint_as_float(r[j]);
-          if (kGrouped) v *= scale;
+          if (kGrouped) v = grouped_value(v, scale, p.gated_act);
           if (p.bias) v += __bfloat162float(p.bias[n0 + j]);
           dst[j] = __float2bfloat16_rn(v);
         }
@@ -149,7 +158,7 @@ __device__ __forceinline__ void store_chunk(const GemmParams& p, const GroupPara
             gate += __bfloat162float(p.bias[n0 + col]);
             up += __bfloat162float(p.bias[n0 + col + 8]);
           }
-          v[e] = kGrouped ? gated_value(gate, up, p.gated_act, g.limit, g.alpha) : gated_value(gate, up, p.gated_act);
+          v[e] = gated_value(gate, up, p.gated_act, p.limit, p.alpha);
         }
         __nv_bfloat162 h = __floats2bfloat162_rn(v[0], v[1]);
         w[j] = *reinterpret_cast<unsigned*>(&h);
@@ -536,14 +545,15 @@ static int launch_gemm_pair(const CUtensorMap& mx, const CUtensorMap& mw, const 
 
 using namespace li;
 
-// bfloat16; K a multiple of 8; x and w 16-byte aligned.  gated_act: -1 plain; 0..3 act(gate) * up on rows of w
+// bfloat16; K a multiple of 8; x and w 16-byte aligned.  gated_act: -1 plain; 0..3 act(gate) * up, or 4 the capped form
+// with `limit` and `alpha`, on rows of w
 // interleaved in eights (N a multiple of 16; out is [M, N/2]).  error_flag (device int, zero): set to the number
 // of the wait that gave up if the kernel's choreography ever stalls (1 loader, 2 accumulator free, 3 stage full,
 // 4 accumulator full); the output is then not to be trusted.
 LI_EXPORT int li_gemm_tcgen05(const void* x, const void* w, const void* bias, void* out, int M, int N, int K,
-                              int gated_act, int* error_flag, cudaStream_t stream) {
+                              int gated_act, float limit, float alpha, int* error_flag, cudaStream_t stream) {
   if (M == 0 || N == 0) return 0;
-  if (K < 8 || (K % 8) || gated_act > 3 || (gated_act >= 0 && (N % 16))) return LI_ERR_UNSUPPORTED;
+  if (K < 8 || (K % 8) || gated_act > 4 || (gated_act >= 0 && (N % 16))) return LI_ERR_UNSUPPORTED;
   if (!aligned16(x) || !aligned16(w) || !aligned16(out)) return LI_ERR_ALIGNMENT;
   static int sms = 0;
   if (!sms) {
@@ -561,7 +571,7 @@ LI_EXPORT int li_gemm_tcgen05(const void* x, const void* w, const void* bias, vo
   if (pair_mode && M >= 256 && N >= 256) {
     CUtensorMap px, pw;
     if (!make_map(&px, x, M, K, kTileM) || !make_map(&pw, w, N, K, 128)) return LI_ERR_UNSUPPORTED;
-    GemmParams pp{(bf16*)out, (const bf16*)bias, M, N, K, gated_act, error_flag};
+    GemmParams pp{(bf16*)out, (const bf16*)bias, M, N, K, gated_act, error_flag, limit, alpha};
     return launch_gemm_pair<6>(px, pw, pp, sms, stream);
   }
   // Tile width: whichever of 256 and 128 needs less time in whole waves of blocks (ties go to the wide tile,
@@ -572,14 +582,14 @@ LI_EXPORT int li_gemm_tcgen05(const void* x, const void* w, const void* bias, vo
   const bool wide = N > 128 && 2 * cost_wide <= 3 * cost_narrow;
   CUtensorMap mx, mw;
   if (!make_map(&mx, x, M, K, kTileM) || !make_map(&mw, w, N, K, wide ? 256 : 128)) return LI_ERR_UNSUPPORTED;
-  GemmParams p{(bf16*)out, (const bf16*)bias, M, N, K, gated_act, error_flag};
+  GemmParams p{(bf16*)out, (const bf16*)bias, M, N, K, gated_act, error_flag, limit, alpha};
   return wide ? launch_gemm<256, 4>(mx, mw, p, sms, stream) : launch_gemm<128, 6>(mx, mw, p, sms, stream);
 }
 
 // The product grouped by expert: x [rows, K] holds every expert's rows one run after the other (offsets
 // [experts + 1]); w [experts * N, K] the experts' matrices one below the other; out [rows, N] (gated_act >= 0:
 // [rows, N / 2], the rows of each expert's w interleaved in eights, eight gate rows and then their eight up rows;
-// gated_act 4 is the experts' capped form with `limit` and `alpha`).  Row tile t (of `row_tiles`) is 128 rows of expert
+// gated_act 4 is the capped form with `limit` and `alpha`; -2: plain, then relu and its square).  Row tile t (of `row_tiles`) is 128 rows of expert
 // tile_expert[t] from row tile_row0[t] on; -1: no such tile.  row_scale (with row_of, both optional): out[m] is
 // multiplied by row_scale[row_of[m]].  bfloat16; K a multiple of 8.
 LI_EXPORT int li_gemm_tcgen05_grouped(const void* x, const void* w, void* out, int rows, int N, int K, int experts,
@@ -604,7 +614,7 @@ LI_EXPORT int li_gemm_tcgen05_grouped(const void* x, const void* w, void* out, i
   const bool wide = N >= 256 && !narrow;
   CUtensorMap mx, mw;
   if (!make_map(&mx, x, rows, K, kTileM) || !make_map(&mw, w, experts * N, K, wide ? 256 : 128)) return LI_ERR_UNSUPPORTED;
-  GemmParams p{(bf16*)out, nullptr, rows, N, K, gated_act, error_flag};
-  GroupParams g{tile_expert, tile_row0, offsets, row_tiles, row_of, row_scale, limit, alpha};
+  GemmParams p{(bf16*)out, nullptr, rows, N, K, gated_act, error_flag, limit, alpha};
+  GroupParams g{tile_expert, tile_row0, offsets, row_tiles, row_of, row_scale};
   return wide ? launch_gemm<256, 4>(mx, mw, p, sms, stream, g) : launch_gemm<128, 6>(mx, mw, p, sms, stream, g);
 }

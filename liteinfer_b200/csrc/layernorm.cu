@@ -10,7 +10,10 @@
 //                          column slices (q and k of a fused projection, each normalised across all its heads)
 //   li_gated_rmsnorm       out = w * x / sqrt(mean(x^2) + eps) * act(gate) per head; one warp a (token, head);
 //                          act = silu or sigmoid, or no gate at all; w shared by the heads or one per head; x
-//                          optionally divided by a number per (token, head) first; out may be a column slice
+//                          optionally divided by a number per (token, head) first, or with `add_scale` (a number per
+//                          (token, head)) times the rows of `add` added to it; out may be a column slice
+//   li_gated_group_norm    y = (x + skip[head] * add) * silu(gate), then each of `groups` equal parts of the row divided by
+//                          its own root mean square, times w: the gate stands in front of the norm.  One block a part.
 //
 // x of li_layernorm may be float while value, weights and out are bfloat16: the stream stays 32-bit, what the
 // products read is rounded once.  Means, variances, the sum into the stream and every product before the final
@@ -227,7 +230,8 @@ projection_rmsnorm_kernel(T* __restrict__ x, size_t stride, int width_a, const T
 template <typename T>
 __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __restrict__ gate, size_t gate_stride,
                                      const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int tokens,
-                                     int heads, int size, float eps, int weight_stride, int act, const float* __restrict__ den) {
+                                     int heads, int size, float eps, int weight_stride, int act, const float* __restrict__ den,
+                                     const T* __restrict__ add, size_t add_stride, const float* __restrict__ add_scale) {
   grid_dependency_wait();
   const int lane = threadIdx.x & 31;
   const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);   // (token, head)
@@ -235,10 +239,15 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __res
   const size_t t = item / heads;
   const int h = (int)(item - t * heads);
   const float* xr = x + (t * heads + h) * size;
-  const float under = den != nullptr ? den[item] : 1.0f;
+  const float under = den != nullptr ? den[item] : 1.0f, share = add != nullptr ? add_scale[item] : 0.f;
+  const T* ar = add + t * add_stride + (size_t)h * size;
+  auto value = [&](int c) {
+    const float v = den != nullptr ? xr[c] / under : xr[c];
+    return add != nullptr ? fmaf(share, to_float(ar[c]), v) : v;
+  };
   float q = 0.f;
   for (int c = lane; c < size; c += 32) {
-    const float v = den != nullptr ? xr[c] / under : xr[c];
+    const float v = value(c);
     q += v * v;
   }
   const float inv = 1.0f / sqrtf(warp_sum(q) / (float)size + eps);
@@ -246,7 +255,7 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __res
   const float* w = weight + (size_t)h * weight_stride;
   T* o = out + t * out_stride + (size_t)h * size;
   for (int c = lane; c < size; c += 32) {
-    const float v = den != nullptr ? xr[c] / under : xr[c];
+    const float v = value(c);
     float by = 1.0f;
     if (act != 2) {
       const float z = to_float(g[c]);
@@ -264,7 +273,8 @@ template <typename T, int NV>
 __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* __restrict__ gate, size_t gate_stride,
                                          const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int tokens,
                                          int heads, int size, float eps, int weight_stride, int act,
-                                         const float* __restrict__ den) {
+                                         const float* __restrict__ den, const T* __restrict__ add, size_t add_stride,
+                                         const float* __restrict__ add_scale) {
   const int lane = threadIdx.x & 31;
   const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);   // (token, head)
   if (item >= (size_t)tokens * heads) return;
@@ -294,6 +304,20 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
 #pragma unroll
     for (int j = 0; j < NV; ++j) { v[j].x /= under; v[j].y /= under; v[j].z /= under; v[j].w /= under; }
   }
+  if (add != nullptr) {
+    const float share = add_scale[item];
+    const T* ar = add + t * add_stride + (size_t)h * size;
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+      if (lane + 32 * j < quads) {
+        float a[4];
+        load4(ar + 4 * (lane + 32 * j), a);
+        v[j].x = fmaf(share, a[0], v[j].x);
+        v[j].y = fmaf(share, a[1], v[j].y);
+        v[j].z = fmaf(share, a[2], v[j].z);
+        v[j].w = fmaf(share, a[3], v[j].w);
+      }
+  }
   float q = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) q += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
@@ -315,6 +339,77 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
     }
     store4(o + 4 * (lane + 32 * j), r);
   }
+}
+
+// One block a (token, part).  x [tokens, width] float; add (optional, with skip [width / head_size]) and gate in the engine's
+// type; weight [width] float.  A thread keeps NV groups of four columns of the part in registers.
+template <typename T, int NV>
+__global__ void __launch_bounds__(512)
+gated_group_norm_kernel(const float* __restrict__ x, const T* __restrict__ add, size_t add_stride, const float* __restrict__ skip,
+                        int head_size, const T* __restrict__ gate, size_t gate_stride, const float* __restrict__ weight,
+                        T* __restrict__ out, size_t out_stride, int width, int part, float eps) {
+  __shared__ float scratch[33];
+  const int first = blockIdx.y * part;
+  const size_t t = blockIdx.x;
+  float w[NV][4], v[NV][4];
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4;
+    if (c < part) load4(weight + first + c, w[i]);
+  }
+  grid_dependency_wait();
+  float q = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4, col = first + c;
+    if (c >= part) continue;
+    float a[4], z[4];
+    load4(x + t * width + col, v[i]);
+    load4(gate + t * gate_stride + col, z);
+    if (add != nullptr) load4(add + t * add_stride + col, a);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      if (add != nullptr) v[i][e] = fmaf(skip[(col + e) / head_size], a[e], v[i][e]);
+      v[i][e] *= z[e] * (1.0f / (1.0f + expf(-z[e])));
+      q = fmaf(v[i][e], v[i][e], q);
+    }
+  }
+  const float inv = 1.0f / sqrtf(block_sum(q, scratch) / (float)part + eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (i * blockDim.x + threadIdx.x) * 4;
+    if (c >= part) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[i][e] = v[i][e] * inv * w[i][e];
+    store4(out + t * out_stride + first + c, v[i]);
+  }
+}
+
+// The same, any width, a column at a time, the part in shared memory.
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_group_norm_plain_kernel(const float* __restrict__ x, const T* __restrict__ add, size_t add_stride,
+                              const float* __restrict__ skip, int head_size, const T* __restrict__ gate, size_t gate_stride,
+                              const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int width, int part,
+                              float eps) {
+  extern __shared__ float row[];  // [part]
+  __shared__ float scratch[33];
+  grid_dependency_wait();
+  const int first = blockIdx.y * part;
+  const size_t t = blockIdx.x;
+  float q = 0.f;
+  for (int c = threadIdx.x; c < part; c += blockDim.x) {
+    const int col = first + c;
+    const float z = to_float(gate[t * gate_stride + col]);
+    float v = x[t * width + col];
+    if (add != nullptr) v = fmaf(skip[col / head_size], to_float(add[t * add_stride + col]), v);
+    v *= z * (1.0f / (1.0f + expf(-z)));
+    row[c] = v;
+    q = fmaf(v, v, q);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(q, scratch) / (float)part + eps);
+  for (int c = threadIdx.x; c < part; c += blockDim.x)
+    out[t * out_stride + first + c] = from_float<T>(row[c] * inv * weight[first + c]);
 }
 
 template <typename S>
@@ -413,10 +508,11 @@ LI_EXPORT int li_projection_rmsnorm(int dtype, void* x, size_t stride, int rows,
 
 LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size_t gate_stride, const float* weight,
                                void* out, size_t out_stride, int tokens, int heads, int size, float eps,
-                               int weight_per_head, int act,
-                               const float* den, cudaStream_t stream) {
+                               int weight_per_head, int act, const float* den, const void* add, size_t add_stride,
+                               const float* add_scale, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads < 1 || size < 1 || act < 0 || act > 2 || (act == 2) != (gate == nullptr)) return LI_ERR_UNSUPPORTED;
+  if ((add != nullptr) != (add_scale != nullptr)) return LI_ERR_UNSUPPORTED;
   const size_t items = (size_t)tokens * heads;
   const int warps = 8;
   const int weight_stride = weight_per_head ? size : 0;
@@ -424,13 +520,14 @@ LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size
   // Heads of up to 512 whose rows 16-byte accesses can walk keep their row in registers.
   const size_t gate_unit = dtype == kFloat32 ? 4 : 2;
   const bool wide = size % 4 == 0 && size <= 512 && aligned16(x) && aligned16(weight) && aligned16(out) &&
-                    (uintptr_t)gate % (4 * gate_unit) == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0;
+                    (uintptr_t)gate % (4 * gate_unit) == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0 &&
+                    (uintptr_t)add % (4 * gate_unit) == 0 && add_stride % 4 == 0;
   if (wide) {
     const int nv = size <= 128 ? 1 : size <= 256 ? 2 : 4;
 #define LI_GATED(T, NV)                                                                                                \
   return (int)launch_pdl(tokens, gated_rmsnorm_vec_kernel<T, NV>, grid, dim3(warps * 32), 0, stream, x,               \
                          (const T*)gate, gate_stride, weight, (T*)out, out_stride, tokens, heads, size, eps, weight_stride, act, \
-                         den)
+                         den, (const T*)add, add_stride, add_scale)
     if (dtype == kFloat32) {
       if (nv == 1) LI_GATED(float, 1);
       if (nv == 2) LI_GATED(float, 2);
@@ -443,7 +540,61 @@ LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size
   }
   if (dtype == kFloat32)
     return (int)launch_pdl(tokens, gated_rmsnorm_kernel<float>, grid, dim3(warps * 32), 0, stream, x, (const float*)gate,
-                           gate_stride, weight, (float*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den);
+                           gate_stride, weight, (float*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den,
+                           (const float*)add, add_stride, add_scale);
   return (int)launch_pdl(tokens, gated_rmsnorm_kernel<bf16>, grid, dim3(warps * 32), 0, stream, x, (const bf16*)gate,
-                         gate_stride, weight, (bf16*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den);
+                         gate_stride, weight, (bf16*)out, out_stride, tokens, heads, size, eps, weight_stride, act, den,
+                         (const bf16*)add, add_stride, add_scale);
+}
+
+// x [tokens, width] float32, weight [width] float32; add [tokens, width] (rows add_stride apart) with skip [width / head_size]
+// float32, or both null; gate, out in `dtype`.  The row falls into `groups` equal parts.
+LI_EXPORT int li_gated_group_norm(int dtype, const float* x, const void* add, size_t add_stride, const float* skip,
+                                  int head_size, const void* gate, size_t gate_stride, const float* weight, void* out,
+                                  size_t out_stride, int tokens, int width, int groups, float eps, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (groups < 1 || groups > 65535 || width < 1 || width % groups || head_size < 1 || (add != nullptr) != (skip != nullptr) ||
+      gate == nullptr)
+    return LI_ERR_UNSUPPORTED;
+  const int part = width / groups;
+  const size_t unit = dtype == kFloat32 ? 16 : 8;
+  const bool vec = part % 4 == 0 && part <= 8192 && aligned16(x) && aligned16(weight) && (uintptr_t)gate % unit == 0 &&
+                   (uintptr_t)add % unit == 0 && (uintptr_t)out % unit == 0 && gate_stride % 4 == 0 && add_stride % 4 == 0 &&
+                   out_stride % 4 == 0;
+  const dim3 grid(tokens, groups);
+  if (vec) {
+    const int quads = part / 4;
+    const int block = quads >= 512 ? 512 : (quads + 31) / 32 * 32;
+    const int per_thread = (quads + block - 1) / block;
+#define LI_GROUP(T, NV)                                                                                               \
+  return (int)launch_pdl(tokens, gated_group_norm_kernel<T, NV>, grid, dim3(block), 0, stream, x, (const T*)add,      \
+                         add_stride, skip, head_size, (const T*)gate, gate_stride, weight, (T*)out, out_stride, width, \
+                         part, eps)
+#define LI_GROUP_NV(T)                                                                                                \
+  {                                                                                                                   \
+    if (per_thread == 1) LI_GROUP(T, 1);                                                                              \
+    if (per_thread == 2) LI_GROUP(T, 2);                                                                              \
+    LI_GROUP(T, 4);                                                                                                   \
+  }
+    if (dtype == kFloat32) LI_GROUP_NV(float)
+    LI_GROUP_NV(bf16)
+#undef LI_GROUP_NV
+#undef LI_GROUP
+  }
+  const size_t smem = (size_t)part * sizeof(float);
+  if (smem > 200 * 1024) return LI_ERR_UNSUPPORTED;
+#define LI_GROUP_PLAIN(T)                                                                                             \
+  {                                                                                                                   \
+    if (smem > 48 * 1024) {                                                                                           \
+      cudaError_t e = cudaFuncSetAttribute(gated_group_norm_plain_kernel<T>,                                          \
+                                           cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                   \
+      if (e != cudaSuccess) return (int)e;                                                                            \
+    }                                                                                                                 \
+    return (int)launch_pdl(tokens, gated_group_norm_plain_kernel<T>, grid, dim3(256), smem, stream, x, (const T*)add, \
+                           add_stride, skip, head_size, (const T*)gate, gate_stride, weight, (T*)out, out_stride,     \
+                           width, part, eps);                                                                         \
+  }
+  if (dtype == kFloat32) LI_GROUP_PLAIN(float)
+  LI_GROUP_PLAIN(bf16)
+#undef LI_GROUP_PLAIN
 }

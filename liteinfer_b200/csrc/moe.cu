@@ -5,12 +5,16 @@
 //                    `groups` equal groups of neighbours, a group's score is its largest choice score (or the sum of
 //                    its two largest) and only experts of the best `keep` groups can be chosen; the `top` largest choice
 //                    scores among those are chosen (ties go to the lower index); the weights are the chosen experts'
-//                    scores (without the correction), or those divided by their sum.
+//                    scores (without the correction), or those divided by their sum.  The last outputs of the router may
+//                    be identity experts, which have no matrices and give back what they read: they are chosen like the
+//                    others, and the sum of a token's weights of them is a number of its own.
 //   li_moe_sort      the (token, slot) pairs ordered by expert, each expert's run cut into tiles of `tile_rows` rows:
-//                    order[], offsets[experts + 1], and per tile its expert and first row (-1: no such tile).
+//                    order[], offsets[experts + 1], and per tile its expert and first row (-1: no such tile).  A pair whose
+//                    expert is none of those (an identity expert) is in no run; its place is -1.
 //   li_moe_grouped   out[pair] = f(W_e x[row of the pair]) for every pair of expert e, tile by tile, so that an
-//                    expert's weights are read once per tile of its rows.  Two modes: gate and up product with the
-//                    activation (x = the token's row; out [pairs, ff]), and the down product times the pair's weight
+//                    expert's weights are read once per tile of its rows.  Three modes: gate and up product with the
+//                    activation (x = the token's row; out [pairs, ff]), the same for experts without a gate (the up product
+//                    through the square of relu), and the down product times the pair's weight
 //                    (x = the pair's activated row; out [pairs, hidden]).  float32 and odd sizes run FFMA tiles whose
 //                    sums over k have a fixed order; bfloat16 runs mma.sync m16n8k16 tiles fed by cp.async.
 //   li_moe_combine   out[token] = sum over its slots of the pairs' rows, in slot order, in 32-bit.
@@ -24,7 +28,7 @@
 
 namespace li {
 
-constexpr int kModeGateUp = 0, kModeDown = 1;
+constexpr int kModeGateUp = 0, kModeDown = 1, kModeUp = 2;
 
 __device__ __forceinline__ float expert_activation(float g, float u, int act, float limit, float alpha) {
   if (act == 1) {
@@ -33,6 +37,11 @@ __device__ __forceinline__ float expert_activation(float g, float u, int act, fl
     return g * (1.0f / (1.0f + expf(-alpha * g))) * (u + 1.0f);
   }
   return g * (1.0f / (1.0f + expf(-g))) * u;
+}
+
+__device__ __forceinline__ float squared_relu(float v) {
+  const float r = fmaxf(v, 0.f);
+  return r * r;
 }
 
 // ------------------------------------------------------------------------------------------ route
@@ -57,12 +66,14 @@ constexpr int kRankedExperts = 64;      // up to this many experts are ranked si
 
 // How a router turns its logits into chosen experts and weights.
 struct RouteRule {
-  int experts, top, groups, keep, renormalise;
+  int experts, top, groups, keep, renormalise;      // experts: all outputs of the router, identity experts included
   int sigmoid;                // scores: 0 softmax over all experts, 1 the sigmoid of each logit
   int pair_rank;              // a group's score: 0 its largest choice score, 1 the sum of its two largest
   int slots;                  // entries of ids and weights a token has (>= top; the first `top` are the chosen experts)
   float floor;                // added to the sum the weights are divided by
   const float* correction;    // [experts] or null
+  int first_identity;         // outputs from this one on are identity experts (= experts: there are none)
+  float* identity;            // [tokens]: the sum of a token's weights of identity experts (null where there are none)
 };
 
 __host__ __device__ __forceinline__ int route_floats(int experts, int groups) { return 3 * experts + 2 * groups; }
@@ -123,6 +134,7 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
   }
   if (experts <= kRankedExperts) {
     // Every lane counts how many experts stand before its own: the place is the rank, with no round after another.
+    float same = 0.f;
     for (int e = lane; e < experts; e += 32) {
       const float mine = choice[e];
       int before = 0;
@@ -130,20 +142,26 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
       if (before < rule.top) {
         ids[(size_t)t * rule.slots + before] = e;
         kept_score[before] = sc[e];
+        if (e >= rule.first_identity) same += sc[e];
       }
     }
     __syncwarp();
     float total = 0.f;
     for (int r = 0; r < rule.top; ++r) total += kept_score[r];
+    if (rule.identity != nullptr) {
+      same = warp_sum(same);
+      if (lane == 0) rule.identity[t] = rule.renormalise ? same / (total + rule.floor) : same;
+    }
     for (int r = lane; r < rule.top; r += 32)
       weights[(size_t)t * rule.slots + r] = rule.renormalise ? kept_score[r] / (total + rule.floor) : kept_score[r];
     return;
   }
-  float total = 0.f;
+  float total = 0.f, same = 0.f;
   for (int r = 0; r < rule.top; ++r) {
     const int e = warp_argmax(choice, experts, lane);
     const float w = sc[e];
     total += w;
+    if (e >= rule.first_identity) same += w;
     __syncwarp();
     if (lane == 0) {
       ids[(size_t)t * rule.slots + r] = e;
@@ -152,6 +170,7 @@ __device__ __forceinline__ void route_token(const float* z, float* scratch, int 
     }
     __syncwarp();
   }
+  if (rule.identity != nullptr && lane == 0) rule.identity[t] = rule.renormalise ? same / (total + rule.floor) : same;
   if (rule.renormalise)
     for (int r = lane; r < rule.top; r += 32) weights[(size_t)t * rule.slots + r] /= total + rule.floor;
 }
@@ -263,7 +282,7 @@ moe_router_kernel(const T* __restrict__ x, size_t x_stride, const float* __restr
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* __restrict__ ids, int pairs, int experts, int tile_rows, int* __restrict__ offsets,
                 int* __restrict__ order, int* __restrict__ tile_expert, int* __restrict__ tile_row0, int max_tiles,
-                int* __restrict__ place) {
+                int* __restrict__ place, int in_pairs) {
   extern __shared__ int sort_smem[];          // counts[experts], cursor[experts]
   int* counts = sort_smem;
   int* cursor = sort_smem + experts;
@@ -297,7 +316,9 @@ moe_sort_kernel(const int* __restrict__ ids, int pairs, int experts, int tile_ro
     if (e >= 0 && e < experts) {
       const int at = atomicAdd(&cursor[e], 1);
       order[at] = i;
-      if (place != nullptr) place[i] = at;
+      if (place != nullptr) place[i] = in_pairs ? i : at;
+    } else if (place != nullptr) {
+      place[i] = -1;
     }
   }
 }
@@ -305,11 +326,11 @@ moe_sort_kernel(const int* __restrict__ ids, int pairs, int experts, int tile_ro
 // out[m] = x[order[m] / top]: every pair's token row, in the order of the experts' runs.
 template <typename T>
 __global__ void moe_gather_kernel(const T* __restrict__ x, size_t x_stride, const int* __restrict__ order, int top,
-                                  T* __restrict__ out, int pairs, int width) {
+                                  T* __restrict__ out, const int* __restrict__ count, int width) {
   constexpr int N = Vec16<T>::N;
   grid_dependency_wait();
   const int per_row = width / N;
-  const size_t total = (size_t)pairs * per_row;
+  const size_t total = (size_t)*count * per_row;       // pairs of identity experts are in no run
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
     const int m = (int)(i / per_row), c = (int)(i - (size_t)m * per_row) * N;
     store16(out + (size_t)m * width + c, load16(x + (size_t)(order[m] / top) * x_stride + c));
@@ -345,7 +366,7 @@ moe_grouped_simt_kernel(const T* __restrict__ a, size_t a_stride, const T* __res
   if (threadIdx.x < kSimtRows) {
     const int pair = threadIdx.x < rows ? order[row0 + threadIdx.x] : -1;
     out_rows[threadIdx.x] = pair;
-    src_rows[threadIdx.x] = pair < 0 ? -1 : (MODE == kModeGateUp ? pair / top : pair);
+    src_rows[threadIdx.x] = pair < 0 ? -1 : (MODE == kModeDown ? pair : pair / top);
   }
   __syncthreads();
   const int n0 = blockIdx.y * (MODE == kModeGateUp ? 32 : 64);
@@ -393,7 +414,7 @@ moe_grouped_simt_kernel(const T* __restrict__ a, size_t a_stride, const T* __res
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int col = n0 + (j < 2 ? 0 : 32) + 2 * tx + (j & 1);
-        if (col < N) orow[col] = from_float<T>(acc[i][j] * scale);
+        if (col < N) orow[col] = from_float<T>(MODE == kModeUp ? squared_relu(acc[i][j]) : acc[i][j] * scale);
       }
     }
   }
@@ -422,7 +443,7 @@ moe_grouped_mma_kernel(const bf16* __restrict__ a, size_t a_stride, const bf16* 
   if (tid < kMmaRows) {
     const int pair = tid < rows ? order[row0 + tid] : -1;
     out_rows[tid] = pair;
-    src_rows[tid] = pair < 0 ? -1 : (MODE == kModeGateUp ? pair / top : pair);
+    src_rows[tid] = pair < 0 ? -1 : (MODE == kModeDown ? pair : pair / top);
   }
   __syncthreads();
   const int n0 = blockIdx.y * (MODE == kModeGateUp ? 32 : 64);
@@ -500,7 +521,9 @@ moe_grouped_mma_kernel(const bf16* __restrict__ a, size_t a_stride, const bf16* 
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         const int col = n0 + j * 8 + 2 * t;
-        if (col < N) *reinterpret_cast<unsigned*>(orow + col) = pack_bf16(acc[j][2 * h] * scale, acc[j][2 * h + 1] * scale);
+        const float lo = MODE == kModeUp ? squared_relu(acc[j][2 * h]) : acc[j][2 * h] * scale;
+        const float hi = MODE == kModeUp ? squared_relu(acc[j][2 * h + 1]) : acc[j][2 * h + 1] * scale;
+        if (col < N) *reinterpret_cast<unsigned*>(orow + col) = pack_bf16(lo, hi);
       }
     }
   }
@@ -569,7 +592,8 @@ using namespace li;
 
 static bool bad_rule(const RouteRule& r) {
   return r.experts < 1 || r.top < 1 || r.top > r.experts || r.groups < 1 || r.experts % r.groups || r.keep < 1 ||
-         r.keep > r.groups || r.keep * (r.experts / r.groups) < r.top || r.slots < r.top;
+         r.keep > r.groups || r.keep * (r.experts / r.groups) < r.top || r.slots < r.top || r.first_identity < 0 ||
+         r.first_identity > r.experts;
 }
 
 // logits [tokens, experts] float; ids [tokens, top] int; weights [tokens, top] float.  sigmoid, pair_rank, floor,
@@ -578,7 +602,7 @@ LI_EXPORT int li_moe_route(const float* logits, int tokens, int experts, int top
                            int renormalise, int sigmoid, int pair_rank, float floor, const float* correction, int* ids,
                            float* weights, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top, floor, correction};
+  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top, floor, correction, experts, nullptr};
   if (bad_rule(rule)) return LI_ERR_UNSUPPORTED;
   const size_t smem = (size_t)kRouteWarps * route_floats(experts, groups) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
@@ -593,27 +617,30 @@ LI_EXPORT int li_moe_tile_rows(int dtype, int N, int K) {
 
 // ids [pairs] int (the expert of every pair); offsets [experts + 1]; order [pairs]; tile_expert, tile_row0 [max_tiles]
 // with max_tiles >= pairs / tile_rows + experts.
-// place [pairs] (optional): where in `order` each pair stands.
+// place [pairs] (optional): where in `order` each pair stands (`in_pairs`: the pair itself), -1 for a pair of no expert.
 LI_EXPORT int li_moe_sort(const int* ids, int pairs, int experts, int tile_rows, int* offsets, int* order,
-                          int* tile_expert, int* tile_row0, int max_tiles, int* place, cudaStream_t stream) {
+                          int* tile_expert, int* tile_row0, int max_tiles, int* place, int in_pairs, cudaStream_t stream) {
   if (experts < 1 || tile_rows < 1 || max_tiles < (pairs + tile_rows - 1) / tile_rows + experts - 1)
     return LI_ERR_UNSUPPORTED;
   const size_t smem = (size_t)2 * experts * sizeof(int);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
   return (int)launch_pdl(pairs, moe_sort_kernel, dim3(1), dim3(1024), smem, stream, ids, pairs, experts, tile_rows,
-                         offsets, order, tile_expert, tile_row0, max_tiles, place);
+                         offsets, order, tile_expert, tile_row0, max_tiles, place, in_pairs);
 }
 
 // x [tokens, K] (rows x_stride apart) in the engine's dtype, w [experts, K] float: the router's product and the routing
 // of li_moe_route in one launch.  gated: w has a row more (see moe_router_kernel); ids and weights are [tokens, top +
-// extra], gate [tokens] float or null.
+// extra], gate [tokens] float or null.  identity_experts: the last so many of `experts` are identity experts; identity
+// [tokens] receives the sum of a token's weights of them.
 LI_EXPORT int li_moe_router(int dtype, const void* x, size_t x_stride, const float* w, int tokens, int K, int experts,
                             int top, int groups, int keep, int renormalise, int sigmoid, int pair_rank, float floor,
                             const float* correction, int gated, int extra, int* ids, float* weights, float* gate,
-                            cudaStream_t stream) {
+                            int identity_experts, float* identity, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top + extra, floor, correction};
+  const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top + extra, floor, correction,
+                       experts - identity_experts, identity};
   if (K < 1 || extra < 0 || (extra > 0 && !gated) || bad_rule(rule)) return LI_ERR_UNSUPPORTED;
+  if (identity_experts < 0 || (identity_experts > 0) != (identity != nullptr) || (identity_experts > 0 && gated)) return LI_ERR_UNSUPPORTED;
   const bool wide = tokens > 128;
   const size_t smem = (size_t)(wide ? 8 : 1) * (route_floats(experts, groups) + 1) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;
@@ -630,9 +657,9 @@ LI_EXPORT int li_moe_router(int dtype, const void* x, size_t x_stride, const flo
 #undef LI_ROUTER
 }
 
-// out [pairs, width] = x[order[m] / top] for every place m of `order`; width a multiple of 16 bytes.
+// out [pairs, width] = x[order[m] / top] for every place m < *count of `order`; width a multiple of 16 bytes.
 LI_EXPORT int li_moe_gather(int dtype, const void* x, size_t x_stride, const int* order, int top, void* out, int pairs,
-                            int width, cudaStream_t stream) {
+                            const int* count, int width, cudaStream_t stream) {
   if (pairs == 0 || width == 0) return 0;
   const int n = dtype == kFloat32 ? 4 : 8;
   if (width % n || x_stride % n || !aligned16(x) || !aligned16(out)) return LI_ERR_ALIGNMENT;
@@ -640,13 +667,14 @@ LI_EXPORT int li_moe_gather(int dtype, const void* x, size_t x_stride, const int
   const dim3 grid((unsigned)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16));
   if (dtype == kFloat32)
     return (int)launch_pdl(pairs, moe_gather_kernel<float>, grid, dim3(256), 0, stream, (const float*)x, x_stride, order,
-                           top, (float*)out, pairs, width);
+                           top, (float*)out, count, width);
   return (int)launch_pdl(pairs, moe_gather_kernel<bf16>, grid, dim3(256), 0, stream, (const bf16*)x, x_stride, order, top,
-                         (bf16*)out, pairs, width);
+                         (bf16*)out, count, width);
 }
 
 // mode 0: out[pair, 0:N] = act(W_gate,e x[pair / top], W_up,e x[pair / top]), w [experts, 2N, K] (gate rows, then up).
 // mode 1: out[pair, 0:N] = (W_down,e a[pair]) * pair_weights[pair] (null: 1), w [experts, N, K].
+// mode 2: out[pair, 0:N] = relu(W_up,e x[pair / top])^2, w [experts, N, K].
 // `tile_rows`: the rows of the tiles li_moe_sort made: 64 runs the tensor-core tiles (only where
 // li_moe_tile_rows(dtype, N, K) says 64), 32 the FFMA tiles.
 LI_EXPORT int li_moe_grouped(int dtype, int mode, const void* a, size_t a_stride, const void* w, void* out,
@@ -657,19 +685,25 @@ LI_EXPORT int li_moe_grouped(int dtype, int mode, const void* a, size_t a_stride
   if (max_tiles <= 0 || N <= 0 || K <= 0) return 0;
   if (tile_rows != kSimtRows && !(tile_rows == kMmaRows && li_moe_tile_rows(dtype, N, K) == kMmaRows))
     return LI_ERR_UNSUPPORTED;
-  if (mode != kModeGateUp && mode != kModeDown) return LI_ERR_UNSUPPORTED;
+  if (mode != kModeGateUp && mode != kModeDown && mode != kModeUp) return LI_ERR_UNSUPPORTED;
   if (eights && mode == kModeGateUp && (N % 8)) return LI_ERR_UNSUPPORTED;
   if (max_tiles > 0x7fffffff / 2 || (N + 31) / 32 > 65535) return LI_ERR_UNSUPPORTED;
 #define LI_MOE_ARGS a, a_stride, w, out, out_stride, order, offsets, tile_expert, tile_row0, pair_weights, top, N, K, act, \
                     limit, alpha, max_tiles, eights, stream
   if (dtype == kFloat32)
-    return mode == kModeGateUp ? launch_simt<float, kModeGateUp>(LI_MOE_ARGS) : launch_simt<float, kModeDown>(LI_MOE_ARGS);
+    return mode == kModeGateUp ? launch_simt<float, kModeGateUp>(LI_MOE_ARGS)
+           : mode == kModeUp   ? launch_simt<float, kModeUp>(LI_MOE_ARGS)
+                               : launch_simt<float, kModeDown>(LI_MOE_ARGS);
   if (tile_rows == kMmaRows) {
     if ((a_stride % 8) || (out_stride % 2) || !aligned16(a) || !aligned16(w) || (reinterpret_cast<uintptr_t>(out) & 3))
       return LI_ERR_ALIGNMENT;
-    return mode == kModeGateUp ? launch_mma<kModeGateUp>(LI_MOE_ARGS) : launch_mma<kModeDown>(LI_MOE_ARGS);
+    return mode == kModeGateUp ? launch_mma<kModeGateUp>(LI_MOE_ARGS)
+           : mode == kModeUp   ? launch_mma<kModeUp>(LI_MOE_ARGS)
+                               : launch_mma<kModeDown>(LI_MOE_ARGS);
   }
-  return mode == kModeGateUp ? launch_simt<bf16, kModeGateUp>(LI_MOE_ARGS) : launch_simt<bf16, kModeDown>(LI_MOE_ARGS);
+  return mode == kModeGateUp ? launch_simt<bf16, kModeGateUp>(LI_MOE_ARGS)
+         : mode == kModeUp   ? launch_simt<bf16, kModeUp>(LI_MOE_ARGS)
+                             : launch_simt<bf16, kModeDown>(LI_MOE_ARGS);
 #undef LI_MOE_ARGS
 }
 

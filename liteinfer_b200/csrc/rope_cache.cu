@@ -27,6 +27,12 @@
 // `norm_flags`: bit 0, q and k are divided by their root mean square also where no weight is given; bit 1, the norm
 // (and its weight) comes behind the rotation instead of in front of it.  `cs_scale` multiplies every cosine and sine.
 //
+// li_projection_norm_rope_kv_write does it for an attention whose q and k pass a root-mean-square norm over their whole
+// projection (all heads at once, one weight per row of the projection), optionally behind a bias, and whose values may be
+// its keys as projected (with the bias, in front of norm and rotation):
+//     q <- rot(w_q * (q + b_q) / sqrt(mean((q + b_q)^2) + eps));  k likewise;  v <- v + b_v, or k + b_k
+// The mean runs over `q_count` and `k_count` numbers: heads that were rounded up with zeros count as what they were.
+//
 // li_sigmoid_gate_heads multiplies head h of every row of x by sigmoid(gate[row, h]) in place; li_sigmoid_gate
 // every element by the sigmoid of its own gate.
 #include "common.cuh"
@@ -238,6 +244,134 @@ head_norm_rope_kv_write_vec_kernel(T* __restrict__ qkv, size_t row_stride, const
     }
     store16(v_pool + (((size_t)page * kv_heads + h) * page_size + slot) * v_dim + j, v);
   }
+}
+
+// A block a token.  The row's q and k (with their biases) wait in shared memory as floats between the sums of squares and
+// the rotation; E neighbouring dimensions a thread (16 bytes, or one).
+template <typename T, int E>
+__global__ void __launch_bounds__(kPrepWarps * 32)
+projection_norm_rope_kv_write_kernel(T* __restrict__ qkv, size_t row_stride, const int* __restrict__ positions,
+                                     const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                                     int table_stride, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                                     const float* __restrict__ inv_freq, int heads, int kv_heads, int head_dim, int rotary_dim,
+                                     int page_size, int num_pages, int v_dim, const float* __restrict__ q_norm,
+                                     const float* __restrict__ k_norm, float q_count, float k_count, float norm_eps,
+                                     const float* __restrict__ bias, int values_are_keys, float cs_scale) {
+  extern __shared__ __align__(16) float shared[];  // q and k as floats, cos [half], sin [half]
+  __shared__ float scratch[33];
+  const int t = blockIdx.x;
+  const int q_width = heads * head_dim, qk_width = q_width + kv_heads * head_dim;
+  const int half = rotary_dim / 2;
+  float* cosv = shared + qk_width;
+  float* sinv = cosv + half;
+  grid_launch_dependents();
+  const int pos = positions[t];
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float angle = __fmul_rn((float)pos, inv_freq[i]);
+    cosv[i] = cosf(angle) * cs_scale;
+    sinv[i] = sinf(angle) * cs_scale;
+  }
+  const int seq = seq_of_token[t];
+  const int page = seq < 0 ? -1 : block_table[(size_t)seq * table_stride + pos / page_size];
+  const bool store = page >= 0 && page < num_pages;
+  const int slot = pos % page_size;
+  grid_dependency_wait();           // q, k and v come from the projection before this kernel
+
+  T* row = qkv + (size_t)t * row_stride;
+  float q_sum = 0.f, k_sum = 0.f;
+  for (int i = threadIdx.x * E; i < qk_width; i += blockDim.x * E) {
+    float x[E];
+    if constexpr (E > 1) unpack16(load16(row + i), x);
+    else x[0] = to_float(row[i]);
+    if (bias != nullptr)
+#pragma unroll
+      for (int e = 0; e < E; ++e) x[e] += bias[i + e];
+    float sum = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      shared[i + e] = x[e];
+      sum = fmaf(x[e], x[e], sum);
+    }
+    if (i < q_width) q_sum += sum;
+    else k_sum += sum;
+    if (store && values_are_keys && i >= q_width) {      // (then v_dim == head_dim)
+      const int h = (i - q_width) / head_dim, j = i - q_width - h * head_dim;
+      T* dst = v_pool + (((size_t)page * kv_heads + h) * page_size + slot) * v_dim + j;
+      if constexpr (E > 1) {
+        Vec16<T> v;
+#pragma unroll
+        for (int e = 0; e < E; ++e) v.set(e, x[e]);
+        store16(dst, v);
+      } else {
+        dst[0] = from_float<T>(x[0]);
+      }
+    }
+  }
+  const float q_inv = 1.0f / sqrtf(block_sum(q_sum, scratch) / q_count + norm_eps);
+  const float k_inv = 1.0f / sqrtf(block_sum(k_sum, scratch) / k_count + norm_eps);   // (its barriers show `shared` to all)
+
+  // Work items: a head's rotated part in pairs of E dimensions half a rotary width apart, then what passes through.
+  const int pairs = half / E, rest = (head_dim - rotary_dim) / E, per_head = pairs + rest;
+  for (int w = threadIdx.x; w < (heads + kv_heads) * per_head; w += blockDim.x) {
+    const int h = w / per_head, i = w - h * per_head;
+    const bool is_q = h < heads;
+    if (!is_q && !store) continue;
+    const int j = i < pairs ? i * E : rotary_dim + (i - pairs) * E;      // the first dimension within the head
+    const int at = h * head_dim + j;
+    const float inv = is_q ? q_inv : k_inv;
+    const float* weight = is_q ? q_norm + at : k_norm + (at - q_width);
+    T* dst = is_q ? row + at : k_pool + (((size_t)page * kv_heads + (h - heads)) * page_size + slot) * head_dim + j;
+    float lo[E], hi[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) lo[e] = shared[at + e] * inv * weight[e];
+    if (i < pairs) {
+#pragma unroll
+      for (int e = 0; e < E; ++e) {
+        const float b = shared[at + half + e] * inv * weight[half + e], c = cosv[j + e], s = sinv[j + e];
+        hi[e] = rotate_hi(lo[e], b, c, s);
+        lo[e] = rotate_lo(lo[e], b, c, s);
+      }
+    }
+    if constexpr (E > 1) {
+      Vec16<T> v;
+#pragma unroll
+      for (int e = 0; e < E; ++e) v.set(e, lo[e]);
+      store16(dst, v);
+      if (i < pairs) {
+#pragma unroll
+        for (int e = 0; e < E; ++e) v.set(e, hi[e]);
+        store16(dst + half, v);
+      }
+    } else {
+      dst[0] = from_float<T>(lo[0]);
+      if (i < pairs) dst[half] = from_float<T>(hi[0]);
+    }
+  }
+  if (!store || values_are_keys) return;
+  for (int i = threadIdx.x; i < kv_heads * v_dim; i += blockDim.x) {
+    const int h = i / v_dim, j = i - h * v_dim;
+    float v = to_float(row[qk_width + i]);
+    if (bias != nullptr) v += bias[qk_width + i];
+    v_pool[(((size_t)page * kv_heads + h) * page_size + slot) * v_dim + j] = from_float<T>(v);
+  }
+}
+
+template <typename T, int E>
+static int launch_projection_norm(cudaStream_t stream, size_t smem, int tokens, void* qkv, size_t row_stride,
+                                  const int* positions, const int* seq_of_token, const int* block_table, int table_stride,
+                                  void* k_pool, void* v_pool, const float* inv_freq, int heads, int kv_heads, int head_dim,
+                                  int rotary_dim, int page_size, int num_pages, int v_dim, const float* q_norm,
+                                  const float* k_norm, float q_count, float k_count, float norm_eps, const float* bias,
+                                  int values_are_keys, float cs_scale) {
+  if (smem > 48 * 1024) {
+    cudaError_t e = cudaFuncSetAttribute(projection_norm_rope_kv_write_kernel<T, E>,
+                                         cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+  }
+  return (int)launch_pdl(tokens, projection_norm_rope_kv_write_kernel<T, E>, dim3(tokens), dim3(kPrepWarps * 32), smem, stream,
+                         (T*)qkv, row_stride, positions, seq_of_token, block_table, table_stride, (T*)k_pool, (T*)v_pool,
+                         inv_freq, heads, kv_heads, head_dim, rotary_dim, page_size, num_pages, v_dim, q_norm, k_norm, q_count,
+                         k_count, norm_eps, bias, values_are_keys, cs_scale);
 }
 
 // x [tokens, heads * size] in 16-byte vectors (size a multiple of the vector's length).
@@ -499,6 +633,38 @@ LI_EXPORT int li_head_norm_rope_kv_write(int dtype, void* qkv, size_t row_stride
                          (bf16*)v_pool, inv_freq, heads, kv_heads, head_dim, rotary_dim, page_size, num_pages, v_dim,
                          (const bf16*)q_norm, (const bf16*)k_norm, norm_eps, (const bf16*)v_other, v_other_stride,
                          lambda, norm_flags, cs_scale);
+}
+
+// q_norm [heads * head_dim], k_norm [kv_heads * head_dim] float32.  bias (optional): one float per column of q, k (and v).
+// values_are_keys: the stored values are k with its bias; the row then holds no v, and v_dim == head_dim.  num_pages 0:
+// nothing is stored.
+LI_EXPORT int li_projection_norm_rope_kv_write(int dtype, void* qkv, size_t row_stride, const int* positions,
+                                               const int* seq_of_token, const int* block_table, int table_stride,
+                                               void* k_pool, void* v_pool, const float* inv_freq, int tokens, int heads,
+                                               int kv_heads, int head_dim, int rotary_dim, int page_size, int num_pages,
+                                               int v_dim, const float* q_norm, const float* k_norm, int q_count, int k_count,
+                                               float norm_eps, const float* bias, int values_are_keys, float cs_scale,
+                                               cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  if (v_dim < 1 || head_dim < 1 || heads < 1 || kv_heads < 1 || q_count < 1 || k_count < 1) return LI_ERR_UNSUPPORTED;
+  if (rotary_dim < 0 || rotary_dim > head_dim || (rotary_dim & 1)) return LI_ERR_UNSUPPORTED;
+  if ((rotary_dim > 0 && inv_freq == nullptr) || q_norm == nullptr || k_norm == nullptr) return LI_ERR_UNSUPPORTED;
+  if (values_are_keys && v_dim != head_dim) return LI_ERR_UNSUPPORTED;
+  const size_t smem = ((size_t)(heads + kv_heads) * head_dim + rotary_dim) * sizeof(float);
+  if (smem > 200 * 1024) return LI_ERR_UNSUPPORTED;
+  // Vectors of 16 bytes where each lies within one head and one side of the rotation.
+  const int n = dtype == kFloat32 ? 4 : 8;
+  const bool fits = (rotary_dim / 2) % n == 0 && head_dim % n == 0 && rotary_dim % n == 0 && row_stride % n == 0 &&
+                    aligned16(qkv) && aligned16(k_pool) && aligned16(v_pool);
+#define LI_PREP(T, E)                                                                                                  \
+  return launch_projection_norm<T, E>(stream, smem, tokens, qkv, row_stride, positions, seq_of_token, block_table,     \
+                                      table_stride, k_pool, v_pool, inv_freq, heads, kv_heads, head_dim, rotary_dim,   \
+                                      page_size, num_pages, v_dim, q_norm, k_norm, (float)q_count, (float)k_count,     \
+                                      norm_eps, bias, values_are_keys, cs_scale)
+  if (dtype == kFloat32) { if (fits) LI_PREP(float, 4); LI_PREP(float, 1); }
+  if (fits) LI_PREP(bf16, 8);
+  LI_PREP(bf16, 1);
+#undef LI_PREP
 }
 
 LI_EXPORT int li_sigmoid_gate_heads(int dtype, void* x, const void* gate, size_t gate_stride, int tokens, int heads,

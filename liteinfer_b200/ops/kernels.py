@@ -22,6 +22,9 @@ from liteinfer_b200.ops.library import KernelLibraryError, load
 
 _DTYPE_CODE = {torch.float32: 0, torch.bfloat16: 1}
 ACTIVATIONS = {"silu": 0, "gelu": 1, "gelu_pytorch_tanh": 2, "gelu_tanh": 2, "relu": 3}
+# Ways to join a gate and an up projection: act(gate) * up, and "capped_swiglu" (with numbers `limit` and `alpha`): with
+# g' = min(g, limit), g' * sigmoid(alpha g') * (clamp(u, -limit, limit) + 1).
+GATED_ACTIVATIONS = {**ACTIVATIONS, "capped_swiglu": 4}
 # Activations of a feed-forward without a gate (`activation`): the above, and the square of relu.
 UNARY_ACTIVATIONS = {**ACTIVATIONS, "relu_squared": 4}
 # A weight-streaming product takes an activation of one argument as this base plus its code (csrc/gemm_skinny.cuh).
@@ -42,8 +45,9 @@ _SIGNATURES = {
                                    c_int, c_void_p]),
     "li_add": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_void_p]),
     "li_add_bias": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_void_p]),
-    "li_act_mul": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_void_p]),
-    "li_act_mul_interleaved": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_void_p]),
+    "li_act_mul": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_float, c_float, c_void_p]),
+    "li_act_mul_interleaved": ("elementwise", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_float, c_float,
+                                               c_void_p]),
     "li_rope_kv_write": ("rope_cache", [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                         c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                         c_void_p]),
@@ -51,15 +55,19 @@ _SIGNATURES = {
                                                   c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                                   c_int, c_int, c_int, c_void_p, c_void_p, c_float, c_void_p,
                                                   c_size_t, c_void_p, c_int, c_float, c_void_p]),
+    "li_projection_norm_rope_kv_write": ("rope_cache", [
+        c_int, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+        c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_float, c_void_p]),
     "li_sigmoid_gate": ("rope_cache", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_void_p]),
     "li_softcap": ("elementwise", [c_int, c_void_p, c_size_t, c_float, c_void_p]),
     "li_moe_route": ("moe", [c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p, c_void_p,
                              c_void_p, c_void_p]),
     "li_moe_tile_rows": ("moe", [c_int, c_int, c_int]),
-    "li_moe_sort": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+    "li_moe_sort": ("moe", [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int,
                             c_void_p]),
     "li_moe_router": ("moe", [c_int, c_void_p, c_size_t, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                              c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]),
+                              c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p,
+                              c_void_p]),
     "li_hgrn2_steps": ("hgrn2", [c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p]),
     "li_hgrn2_token": ("hgrn2", [c_int, c_void_p, c_size_t, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p,
@@ -68,7 +76,7 @@ _SIGNATURES = {
     "li_sum_norms": ("sum_norms", [c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_void_p,
                                    c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                    c_float, c_int, c_void_p]),
-    "li_moe_gather": ("moe", [c_int, c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p]),
+    "li_moe_gather": ("moe", [c_int, c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p]),
     "li_gemm_tcgen05_grouped": ("gemm_tcgen05", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float,
                                                  c_float, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
                                                  c_void_p, c_void_p]),
@@ -89,9 +97,28 @@ _SIGNATURES = {
     "li_projection_rmsnorm": ("layernorm", [c_int, c_void_p, c_size_t, c_int, c_int, c_void_p, c_int, c_void_p,
                                             c_float, c_void_p]),
     "li_gated_rmsnorm": ("layernorm", [c_int, c_void_p, c_void_p, c_size_t, c_void_p, c_void_p, c_size_t, c_int, c_int, c_int,
-                                       c_float, c_int, c_int, c_void_p, c_void_p]),
+                                       c_float, c_int, c_int, c_void_p, c_void_p, c_size_t, c_void_p, c_void_p]),
+    "li_gated_group_norm": ("layernorm", [c_int, c_void_p, c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_size_t, c_void_p,
+                                          c_void_p, c_size_t, c_int, c_int, c_int, c_float, c_void_p]),
+    "li_output_norm": ("output_norm", [c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_float, c_void_p, c_float,
+                                       c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_void_p, c_float, c_void_p,
+                                       c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "li_memory_record_floats": ("linear_memory", [c_int, c_int, c_int, c_void_p]),
+    "li_ssd_steps": ("linear_memory", [c_int, c_void_p, c_size_t, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int,
+                                       c_void_p]),
+    "li_ssd_token": ("linear_memory", [c_int, c_void_p, c_size_t, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p,
+                                       c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "li_wkv_steps": ("linear_memory", [c_int, c_void_p, c_void_p, c_void_p, c_size_t, c_void_p, c_size_t, c_int, c_void_p,
+                                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                       c_int, c_void_p, c_int, c_int, c_void_p]),
+    "li_wkv_token": ("linear_memory", [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_size_t, c_void_p, c_size_t, c_int,
+                                       c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_float,
+                                       c_void_p, c_size_t, c_int, c_int, c_void_p]),
+    "li_token_shift": ("linear_memory", [c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                         c_int, c_int, c_int, c_void_p]),
     "li_short_conv": ("delta_rule", [c_int, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+                                     c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p]),
     "li_short_conv_update": ("delta_rule", [c_int, c_void_p, c_size_t, c_void_p, c_void_p, c_void_p, c_int, c_int,
                                             c_int, c_void_p]),
     "li_gated_delta_rule": ("delta_rule", [c_int, c_void_p, c_void_p, c_size_t, c_int, c_int, c_void_p, c_void_p,
@@ -115,17 +142,17 @@ _SIGNATURES = {
         c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_void_p, c_int,
         c_void_p]),
     "li_paged_attention_tcgen05_supports": ("attention_tcgen05", [c_int, c_int, c_int, c_int]),
-    "li_gemm_skinny": ("gemm_skinny", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+    "li_gemm_skinny": ("gemm_skinny", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
                                        c_void_p, c_size_t, c_void_p, c_int, c_void_p]),
     "li_gemm_skinny_fused": ("gemm_skinny", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                                              c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                              c_float, c_void_p, c_void_p, c_int, c_void_p]),
     "li_gemm_skinny_plan": ("gemm_skinny", [c_int, c_int, c_void_p, c_void_p]),
-    "li_gemm_stream": ("gemm_stream", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
+    "li_gemm_stream": ("gemm_stream", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p,
                                        c_int, c_void_p, c_void_p]),
     "li_gemm_stream_supports": ("gemm_stream", [c_int, c_int, c_int]),
-    "li_gemm_tcgen05": ("gemm_tcgen05", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p,
-                                         c_void_p]),
+    "li_gemm_tcgen05": ("gemm_tcgen05", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                         c_void_p, c_void_p]),
     "li_gemm_simt": ("gemm_simt", [c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "li_gemm_simt_batched": ("gemm_simt", [c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                            c_int, c_long, c_long, c_long, c_void_p]),
@@ -405,15 +432,16 @@ def add_bias_(out: torch.Tensor, bias: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str) -> torch.Tensor:
-    """out = act(gate_up[:, :w]) * gate_up[:, w:], w = out.shape[1]."""
+def act_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str, limit: float = 0.0,
+            alpha: float = 1.0) -> torch.Tensor:
+    """out = act(gate_up[:, :w]) * gate_up[:, w:], w = out.shape[1] (or another of `GATED_ACTIVATIONS`)."""
     _on_gpu(gate_up, out)
     rows, width = out.shape
     assert gate_up.shape == (rows, 2 * width) and gate_up.dtype == out.dtype
-    if activation not in ACTIVATIONS:
-        raise KernelLibraryError(f"activation {activation!r} has no kernel; known: {sorted(ACTIVATIONS)}")
-    _check(_fn("li_act_mul")(_code(out), gate_up.data_ptr(), out.data_ptr(), rows, width, ACTIVATIONS[activation],
-                             _stream()), "act_mul")
+    if activation not in GATED_ACTIVATIONS:
+        raise KernelLibraryError(f"activation {activation!r} has no kernel; known: {sorted(GATED_ACTIVATIONS)}")
+    _check(_fn("li_act_mul")(_code(out), gate_up.data_ptr(), out.data_ptr(), rows, width, GATED_ACTIVATIONS[activation],
+                             float(limit), float(alpha), _stream()), "act_mul")
     return out
 
 
@@ -543,7 +571,8 @@ SKINNY_SMALL_WEIGHT_ROWS = 4096
 NUM_SMS = 148
 
 
-def _skinny(x, weight, out, bias, gated_act: int, residual: torch.Tensor | None = None, rings: bool = True):
+def _skinny(x, weight, out, bias, gated_act: int, residual: torch.Tensor | None = None, rings: bool = True,
+            limit: float = 0.0, alpha: float = 1.0):
     """A weight-streaming kernel, with what `x` (a tensor or a PendingNorm) and `residual` ask to be fused in:
     the persistent kernel with TMA rings where it takes the sizes (and `rings`), else the one that loads through
     registers."""
@@ -557,7 +586,7 @@ def _skinny(x, weight, out, bias, gated_act: int, residual: torch.Tensor | None 
         if residual is not None:
             stats = RowStats(torch.empty((-(-N // 16), M), dtype=torch.float32, device=weight.device))
         code = _fn("li_gemm_stream")(x.data_ptr(), weight.data_ptr(), _ptr(bias),
-                                     (residual if residual is not None else out).data_ptr(), M, N, K, gated_act,
+                                     (residual if residual is not None else out).data_ptr(), M, N, K, gated_act, limit, alpha,
                                      _ptr(stats.sumsq if stats is not None else None), M if stats is not None else 0,
                                      ws.gemm_error.data_ptr(), _stream())
         if code != 100001:          # sizes it refuses go to the kernel below
@@ -565,9 +594,11 @@ def _skinny(x, weight, out, bias, gated_act: int, residual: torch.Tensor | None 
             return stats if stats is not None else out
     if pending is None and residual is None:
         _check(_fn("li_gemm_skinny")(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), M, N, K, gated_act,
-                                     ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
+                                     limit, alpha, ws.gemm.data_ptr(), ws.gemm.numel(), ws.gemm_counters.data_ptr(),
                                      ws.gemm_counters.numel(), _stream()), "gemm_skinny")
         return out
+    if gated_act == GATED_ACTIVATIONS["capped_swiglu"]:
+        raise KernelLibraryError("the capped gate takes x as it is: no pending norm, no residual")
     stats = None
     if residual is not None:
         stats = RowStats(torch.empty((-(-N // 16), M), dtype=torch.float32, device=weight.device))
@@ -610,14 +641,14 @@ def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bias: 
     if residual is not None:
         stats = RowStats(torch.empty((-(-N // 16), M), dtype=torch.float32, device=weight.device))
     _check(_fn("li_gemm_stream")(x.data_ptr(), weight.data_ptr(), _ptr(bias),
-                                 (residual if residual is not None else out).data_ptr(), M, N, K, act,
+                                 (residual if residual is not None else out).data_ptr(), M, N, K, act, 0.0, 1.0,
                                  _ptr(stats.sumsq if stats is not None else None), M if stats is not None else 0,
                                  scratch_for(x.device).gemm_error.data_ptr(), _stream()), "gemm_stream")
     return stats if stats is not None else out
 
 
 def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None,
-                 gated_activation: str | None = None) -> torch.Tensor:
+                 gated_activation: str | None = None, limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """The tcgen05 / TMA / tensor-memory product for bfloat16: out = x @ weight^T (+ bias), or with
     `gated_activation` act(gate) * up on a weight whose rows are interleaved in eights (out is [M, N/2]).
 
@@ -627,9 +658,9 @@ def gemm_tcgen05(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, bias:
     N = weight.shape[0]
     assert weight.shape[1] == K and x.dtype == weight.dtype == out.dtype == torch.bfloat16
     assert out.shape == ((M, N) if gated_activation is None else (M, N // 2))
-    act = -1 if gated_activation is None else ACTIVATIONS[gated_activation]
-    _check(_fn("li_gemm_tcgen05")(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), M, N, K, act,
-                                  scratch_for(x.device).gemm_error.data_ptr(), _stream()), "gemm_tcgen05")
+    act = -1 if gated_activation is None else GATED_ACTIVATIONS[gated_activation]
+    _check(_fn("li_gemm_tcgen05")(x.data_ptr(), weight.data_ptr(), _ptr(bias), out.data_ptr(), M, N, K, act, float(limit),
+                                  float(alpha), scratch_for(x.device).gemm_error.data_ptr(), _stream()), "gemm_tcgen05")
     return out
 
 
@@ -692,28 +723,30 @@ def gated_linear_supported(x: "torch.Tensor | PendingNorm", weight: torch.Tensor
 
 
 def gated_linear(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, activation: str,
-                 bias: torch.Tensor | None = None) -> torch.Tensor:
+                 bias: torch.Tensor | None = None, limit: float = 0.0, alpha: float = 1.0) -> torch.Tensor:
     """out[M, N/2] = act(gate) * up, where `weight` [N, K] holds gate and up rows interleaved in eights
     (rows 16b..16b+7 are gate rows 8b..8b+7, rows 16b+8..16b+15 their up rows): product, activation and
     multiply in one kernel (bfloat16)."""
     M, K = x.shape
     N = weight.shape[0]
-    if isinstance(x, PendingNorm) and M > SKINNY_MAX_ROWS:
+    if isinstance(x, PendingNorm) and (M > SKINNY_MAX_ROWS or activation == "capped_swiglu"):
         x = x.materialise()
     _on_gpu(x.x if isinstance(x, PendingNorm) else x, weight, out, bias)
     assert weight.shape[1] == K and out.shape == (M, N // 2) and gated_linear_supported(x, weight)
     if M <= SKINNY_MAX_ROWS:
-        return _skinny(x, weight, out, bias, ACTIVATIONS[activation])
-    return gemm_tcgen05(x, weight, out, bias, activation)
+        return _skinny(x, weight, out, bias, GATED_ACTIVATIONS[activation], limit=float(limit), alpha=float(alpha))
+    return gemm_tcgen05(x, weight, out, bias, activation, limit, alpha)
 
 
-def act_mul_interleaved(gate_up: torch.Tensor, out: torch.Tensor, activation: str) -> torch.Tensor:
+def act_mul_interleaved(gate_up: torch.Tensor, out: torch.Tensor, activation: str, limit: float = 0.0,
+                        alpha: float = 1.0) -> torch.Tensor:
     """`act_mul` for a gate_up whose columns are interleaved in eights like `gated_linear`'s weight rows."""
     _on_gpu(gate_up, out)
     rows, width = out.shape
     assert gate_up.shape == (rows, 2 * width) and gate_up.dtype == out.dtype and width % 8 == 0
     _check(_fn("li_act_mul_interleaved")(_code(out), gate_up.data_ptr(), out.data_ptr(), rows, width,
-                                         ACTIVATIONS[activation], _stream()), "act_mul_interleaved")
+                                         GATED_ACTIVATIONS[activation], float(limit), float(alpha), _stream()),
+           "act_mul_interleaved")
     return out
 
 
@@ -789,6 +822,41 @@ def head_norm_rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, seq_of_t
         _ptr(q_norm), _ptr(k_norm), float(norm_eps), _ptr(v_other), v_other.stride(0) if v_other is not None else 0,
         _ptr(blend), int(unit_norm) | (2 if norm_after_rotation else 0), float(cos_sin_scale), _stream()),
         "head_norm_rope_kv_write")
+
+
+def projection_norm_rope_kv_write(qkv: torch.Tensor, positions: torch.Tensor, seq_of_token: torch.Tensor,
+                                  block_table: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
+                                  inv_freq: torch.Tensor | None, heads: int, kv_heads: int, head_dim: int, rotary_dim: int,
+                                  q_norm: torch.Tensor, k_norm: torch.Tensor, q_count: int, k_count: int, norm_eps: float,
+                                  bias: torch.Tensor | None = None, values_are_keys: bool = False, store: bool = True,
+                                  cos_sin_scale: float = 1.0) -> None:
+    """`rope_kv_write` for an attention whose q and k pass a root-mean-square norm over their whole projection first:
+    q becomes rot(q_norm * q' / sqrt(mean(q'^2) + eps)) in place, q' = q + bias, k likewise on its way into its page.  The
+    means run over `q_count` and `k_count` numbers (heads rounded up with zeros count as what they were).  The stored
+    values are v + bias, or with `values_are_keys` k + bias, in front of norm and rotation.
+
+    qkv [tokens, >= columns]: q, k and (unless `values_are_keys`) v side by side at the start of each row; bias: one float32
+    per column of those, or None.  q_norm [heads * head_dim], k_norm [kv_heads * head_dim] float32.  Statistics, norm and
+    rotation are 32-bit; every result is rounded once."""
+    _rows2d(qkv, "qkv")
+    _on_gpu(positions, seq_of_token, block_table, k_pool, v_pool, inv_freq, q_norm, k_norm, bias)
+    _int32(positions, "positions"); _int32(seq_of_token, "seq_of_token"); _int32(block_table, "block_table")
+    tokens = qkv.shape[0]
+    pages, kvh, page_size, hd = k_pool.shape
+    vd = v_pool.shape[-1]
+    columns = (heads + kv_heads) * head_dim + (0 if values_are_keys else kv_heads * vd)
+    assert (kvh, hd) == (kv_heads, head_dim) and v_pool.shape == (pages, kv_heads, page_size, vd)
+    assert qkv.shape[1] >= columns and k_pool.dtype == qkv.dtype == v_pool.dtype
+    assert inv_freq is None or (inv_freq.dtype == torch.float32 and inv_freq.numel() * 2 == rotary_dim)
+    assert q_norm.dtype == k_norm.dtype == torch.float32
+    assert q_norm.numel() == heads * head_dim and k_norm.numel() == kv_heads * head_dim
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() >= columns)
+    _check(_fn("li_projection_norm_rope_kv_write")(
+        _code(qkv), qkv.data_ptr(), qkv.stride(0), positions.data_ptr(), seq_of_token.data_ptr(), block_table.data_ptr(),
+        block_table.stride(0), k_pool.data_ptr(), v_pool.data_ptr(), _ptr(inv_freq), tokens, heads, kv_heads, head_dim,
+        rotary_dim if inv_freq is not None else 0, page_size, pages if store else 0, vd, q_norm.data_ptr(),
+        k_norm.data_ptr(), int(q_count), int(k_count), float(norm_eps), _ptr(bias), int(values_are_keys),
+        float(cos_sin_scale), _stream()), "projection_norm_rope_kv_write")
 
 
 def sigmoid_gate_(x: torch.Tensor, gate: torch.Tensor) -> torch.Tensor:
@@ -1176,12 +1244,14 @@ def qk_projection_rmsnorm_(q: torch.Tensor, q_weight: torch.Tensor, k: torch.Ten
 
 
 def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tensor, eps: float, out: torch.Tensor,
-                  heads: int, gate_activation: str = "silu", den: torch.Tensor | None = None) -> torch.Tensor:
+                  heads: int, gate_activation: str = "silu", den: torch.Tensor | None = None,
+                  add: torch.Tensor | None = None, add_scale: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, h] = weight * x[t, h] / sqrt(mean(x[t, h]^2) + eps) * act(gate[t, h]) per head.  x: float32
     [tokens, heads * size]; weight: float32, `size` entries shared by the heads or `heads * size`, one vector
     per head; gate and out in the engine's dtype (column slices are fine).  `gate_activation`: "silu" or
     "sigmoid"; without a gate (None) the norm alone.  `den` [tokens, heads] float32: x[t, h] is divided by den[t, h]
-    first."""
+    first.  `add` [tokens, heads * size] (a column slice is fine) with `add_scale` [tokens, heads] float32: add_scale[t, h] *
+    add[t, h] is added to it first."""
     _on_gpu(x, weight, den)
     _rows2d(out, "out")
     tokens, width = out.shape
@@ -1192,34 +1262,63 @@ def gated_rmsnorm(x: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tens
         _rows2d(gate, "gate")
         assert gate.shape == out.shape and gate.dtype == out.dtype
     assert den is None or (den.dtype == torch.float32 and den.numel() == tokens * heads)
+    assert (add is None) == (add_scale is None)
+    if add is not None:
+        _rows2d(add, "add")
+        _on_gpu(add_scale)
+        assert add.shape == out.shape and add.dtype == out.dtype
+        assert add_scale.dtype == torch.float32 and add_scale.numel() == tokens * heads
     if gate_activation not in ("silu", "sigmoid"):
         raise KernelLibraryError(f"gated_rmsnorm knows the gates 'silu' and 'sigmoid', not {gate_activation!r}")
     act = 2 if gate is None else int(gate_activation == "sigmoid")
     _check(_fn("li_gated_rmsnorm")(_code(out), x.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0,
                                    weight.data_ptr(), out.data_ptr(), out.stride(0), tokens, heads, size, float(eps),
-                                   int(weight.numel() == width and heads > 1), act, _ptr(den), _stream()),
+                                   int(weight.numel() == width and heads > 1), act, _ptr(den), _ptr(add),
+                                   add.stride(0) if add is not None else 0, _ptr(add_scale), _stream()),
            "gated_rmsnorm")
+    return out
+
+
+def gated_group_norm(x: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, groups: int,
+                     add: torch.Tensor | None = None, skip: torch.Tensor | None = None) -> torch.Tensor:
+    """y = (x + skip[head] * add) * silu(gate), then out = weight * y / its root mean square within each of `groups` equal
+    parts of the row.  x [tokens, width] and weight [width] float32; add [tokens, width] with skip [heads] float32 (the row is
+    that many heads), or neither; add, gate and out in the engine's dtype (column slices are fine)."""
+    _on_gpu(x, weight, skip)
+    _rows2d(out, "out"); _rows2d(gate, "gate")
+    tokens, width = out.shape
+    assert x.dtype == weight.dtype == torch.float32 and x.shape == out.shape == gate.shape and gate.dtype == out.dtype
+    assert weight.numel() == width and width % groups == 0 and (add is None) == (skip is None)
+    if add is not None:
+        _rows2d(add, "add")
+        assert add.shape == out.shape and add.dtype == out.dtype
+        assert skip.dtype == torch.float32 and width % skip.numel() == 0
+    _check(_fn("li_gated_group_norm")(
+        _code(out), x.data_ptr(), _ptr(add), add.stride(0) if add is not None else 0, _ptr(skip),
+        width // skip.numel() if skip is not None else width, gate.data_ptr(), gate.stride(0), weight.data_ptr(),
+        out.data_ptr(), out.stride(0), tokens, width, groups, float(eps), _stream()), "gated_group_norm")
     return out
 
 
 def short_conv_step(x: torch.Tensor, taps: torch.Tensor, tail: torch.Tensor, seq_of_token: torch.Tensor,
                     query_start_loc: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, out: torch.Tensor,
-                    activation: str = "silu", single_tokens: bool = False) -> torch.Tensor:
+                    activation: str = "silu", single_tokens: bool = False, bias: torch.Tensor | None = None) -> torch.Tensor:
     """`short_conv`, then `short_conv_update`: a step's convolution and the tails moved on by it.  With
     `single_tokens` (every sequence of the step brings exactly one token) one launch does both where the kernel
     can."""
     if single_tokens and short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation,
-                                    move_tail=True) is not None:
+                                    move_tail=True, bias=bias) is not None:
         return out
-    short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation)
+    short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation, bias=bias)
     short_conv_update(x, tail, query_start_loc, state_slots, num_seqs)
     return out
 
 
 def short_conv(x: torch.Tensor, taps: torch.Tensor, tail: torch.Tensor, seq_of_token: torch.Tensor,
                query_start_loc: torch.Tensor, state_slots: torch.Tensor, out: torch.Tensor,
-               activation: str = "silu", move_tail: bool = False) -> "torch.Tensor | None":
-    """A short causal convolution over time per channel, then the activation.
+               activation: str = "silu", move_tail: bool = False,
+               bias: torch.Tensor | None = None) -> "torch.Tensor | None":
+    """A short causal convolution over time per channel (plus `bias`, float32 [channels], if given), then the activation.
 
     x [tokens, channels] (a column slice is fine): this step's inputs, every sequence's end to end.  taps
     [K, channels] (tap by tap): row K-1 multiplies the current token, K-2 the one before.  tail [slots, K-1, channels]: the
@@ -1228,7 +1327,8 @@ def short_conv(x: torch.Tensor, taps: torch.Tensor, tail: torch.Tensor, seq_of_t
     which every sequence brings exactly one token): the launch also moves the tails on; None is returned, and
     nothing done, where the kernel cannot (sizes that its vector form does not take)."""
     _rows2d(x, "x")
-    _on_gpu(taps, tail, seq_of_token, query_start_loc, state_slots, out)
+    _on_gpu(taps, tail, seq_of_token, query_start_loc, state_slots, out, bias)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == x.shape[1])
     _int32(seq_of_token, "seq_of_token"); _int32(query_start_loc, "query_start_loc"); _int32(state_slots, "state_slots")
     tokens, channels = x.shape
     K = taps.shape[0]
@@ -1239,7 +1339,7 @@ def short_conv(x: torch.Tensor, taps: torch.Tensor, tail: torch.Tensor, seq_of_t
     code = _fn("li_short_conv")(_code(x), x.data_ptr(), x.stride(0), taps.data_ptr(), tail.data_ptr() if K > 1 else None,
                                 seq_of_token.data_ptr(), query_start_loc.data_ptr(), state_slots.data_ptr(),
                                 out.data_ptr(), tokens, channels, K, 1 if activation == "silu" else 0,
-                                int(move_tail and K > 1), _stream())
+                                int(move_tail and K > 1), _ptr(bias), _stream())
     if move_tail and code == 100001:
         return None
     _check(code, "short_conv")
@@ -1369,7 +1469,7 @@ def hgrn2(proj: torch.Tensor, offsets: tuple[int, int, int], f_bias: torch.Tenso
 @dataclass
 class RoutedRows:
     """The rows of the experts that every token runs, already multiplied by their weights and not yet added up: those of
-    token t are value[place[t * top + s]] for s < top (place None: value[t * top + s])."""
+    token t are value[place[t * top + s]] for s < top (place None: value[t * top + s]; a negative place: no row)."""
 
     value: torch.Tensor                 # [tokens * top, width]
     top: int
@@ -1378,11 +1478,15 @@ class RoutedRows:
 
 @dataclass
 class SumTerm:
-    """factor * value, each row also times row_factor[row] (float32 [tokens]) where that is given."""
+    """factor * value, each row also times row_factor[row] (float32 [tokens]) where that is given.  With `norm_weight`
+    (float32 [width]) the row is first divided by its root mean square (`norm_eps`) and multiplied by it (only of a sum that
+    is itself normalised, `output_norm`)."""
 
     value: torch.Tensor
     factor: float = 1.0
     row_factor: torch.Tensor | None = None
+    norm_weight: torch.Tensor | None = None
+    norm_eps: float = 0.0
 
 
 @dataclass
@@ -1421,7 +1525,7 @@ def sum_norms(x: torch.Tensor | None, delta: SumDelta, weights: tuple[torch.Tens
     assert x is None or (x.dtype == torch.float32 and len(weights) == len(outs) and (outs or write_stream))
     assert not (write_stream and rows is not None) and (n == tokens if rows is None else rows.numel() == n)
     for t in terms:
-        assert t.value.shape == (tokens, width) and t.value.dtype == dtype
+        assert t.value.shape == (tokens, width) and t.value.dtype == dtype and t.norm_weight is None
         assert t.row_factor is None or (t.row_factor.dtype == torch.float32 and t.row_factor.numel() == tokens)
     if routed is not None:
         assert routed.value.shape == (tokens * routed.top, width) and routed.value.dtype == dtype
@@ -1439,6 +1543,146 @@ def sum_norms(x: torch.Tensor | None, delta: SumDelta, weights: tuple[torch.Tens
         routed.top if routed else 0, _ptr(weights[0] if weights else None), _ptr(weights[1] if len(weights) > 1 else None),
         _ptr(outs[0] if outs else None), _ptr(outs[1] if len(outs) > 1 else None), _ptr(rows), n, width, float(eps),
         int(write_stream), _stream()), "sum_norms")
+
+
+def output_norm(x: torch.Tensor, delta: "NormedDelta", out: torch.Tensor | None = None,
+                weight: torch.Tensor | None = None, eps: float = 0.0, rows: torch.Tensor | None = None,
+                write_stream: bool = True) -> torch.Tensor:
+    """v = x[row] + delta.weight * y / sqrt(mean(y^2) + delta.eps), y the sum of `delta.value` (a `SumDelta`), row = rows[r]
+    if given else r; `out` (the terms' dtype, or None) receives v, or with `weight` (float32) v / sqrt(mean(v^2) + eps) *
+    weight.  With `write_stream` v is stored back.  x [tokens, width] float32; everything in between is 32-bit."""
+    total = delta.value
+    routed, terms = total.routed, list(total.terms)
+    values = [t.value for t in terms] + ([routed.value] if routed is not None else [])
+    _on_gpu(x, out, weight, rows, delta.weight, *values, *(t.row_factor for t in terms), *(t.norm_weight for t in terms),
+            routed.place if routed is not None else None)
+    _int32(rows, "rows")
+    dtype, (tokens, width) = values[0].dtype, x.shape
+    n = tokens if rows is None else rows.numel()
+    assert len(terms) <= 2 and x.dtype == delta.weight.dtype == torch.float32 and delta.weight.numel() == width
+    assert not delta.centred and not (write_stream and rows is not None)
+    assert out is None or (out.shape == (n, width) and out.dtype == dtype)
+    assert weight is None or (weight.dtype == torch.float32 and weight.numel() == width and out is not None)
+    for t in terms:
+        assert t.value.shape == (tokens, width) and t.value.dtype == dtype
+        assert t.row_factor is None or (t.row_factor.dtype == torch.float32 and t.row_factor.numel() == tokens)
+        assert t.norm_weight is None or (t.norm_weight.dtype == torch.float32 and t.norm_weight.numel() == width)
+    if routed is not None:
+        assert routed.value.shape == (tokens * routed.top, width) and routed.value.dtype == dtype
+        _int32(routed.place, "place")
+    dense = []
+    for t in terms + [None] * (2 - len(terms)):
+        dense += ([None, 0.0, None, None, 0.0] if t is None else
+                  [t.value.data_ptr(), float(t.factor), _ptr(t.row_factor), _ptr(t.norm_weight), float(t.norm_eps)])
+    _check(_fn("li_output_norm")(
+        _DTYPE_CODE[dtype], x.data_ptr(), *dense, _ptr(routed.value if routed else None),
+        _ptr(routed.place if routed else None), routed.top if routed else 0, delta.weight.data_ptr(), float(delta.eps),
+        _ptr(weight), float(eps), _ptr(out), _ptr(rows), n, width, int(write_stream), _stream()), "output_norm")
+    return x
+
+
+# ------------------------------------------- memories that are linear in what they hold
+def _memory_records(scalar: bool, dim: int, vdim: int, rows_of_groups: int, rows_of_heads: int, device):
+    head = ctypes.c_int(0)
+    group = int(_fn("li_memory_record_floats")(int(scalar), dim, vdim, ctypes.byref(head)))
+    return (torch.empty(max(rows_of_groups, 1) * group, dtype=torch.float32, device=device),
+            torch.empty(max(rows_of_heads, 1) * head.value, dtype=torch.float32, device=device))
+
+
+def state_space(conved: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor,
+                query_start_loc: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, heads: int, groups: int, dim: int,
+                vdim: int, out: torch.Tensor, max_query_len: int = 0) -> torch.Tensor:
+    """The recurrence of a Mamba-2 layer, token by token, on a 32-bit state per request and head.
+
+    conved [tokens, heads * vdim + 2 * groups * dim]: x (heads of vdim), B and C (groups of dim; head h reads group
+    h // (heads / groups)); dt [tokens, heads] raw (column slices are fine).  With d = softplus(dt + dt_bias):
+    S <- exp(-exp(a_log) d) S + d B x^T;  out[t, h] = S^T C.  out [tokens, heads * vdim] float32.  dt_bias, a_log float32
+    [heads].  state [slots, heads, vdim, dim] float32 (S kept column by column) is read and written.  `max_query_len`: the
+    most tokens a sequence brings, if known (1: one kernel)."""
+    global launch_count
+    _rows2d(conved, "conved"); _rows2d(dt, "dt")
+    _on_gpu(dt_bias, a_log, state, query_start_loc, state_slots, out)
+    _int32(query_start_loc, "query_start_loc"); _int32(state_slots, "state_slots")
+    tokens = conved.shape[0]
+    assert conved.shape[1] == heads * vdim + 2 * groups * dim and dt.shape == (tokens, heads) and dt.dtype == conved.dtype
+    assert dt_bias.dtype == a_log.dtype == state.dtype == out.dtype == torch.float32
+    assert dt_bias.numel() == a_log.numel() == heads and heads % groups == 0
+    assert state.shape[1:] == (heads, vdim, dim) and out.shape == (tokens, heads * vdim)
+    common = (_code(conved), conved.data_ptr(), conved.stride(0), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(),
+              a_log.data_ptr())
+    if max_query_len == 1:
+        _check(_fn("li_ssd_token")(*common, state.data_ptr(), query_start_loc.data_ptr(), state_slots.data_ptr(), num_seqs,
+                                   out.data_ptr(), heads, groups, dim, vdim, _stream()), "ssd_token")
+        return out
+    records = _memory_records(True, dim, vdim, tokens * groups, tokens * heads, conved.device)
+    _check(_fn("li_ssd_steps")(*common, records[0].data_ptr(), records[1].data_ptr(), state.data_ptr(),
+                               query_start_loc.data_ptr(), state_slots.data_ptr(), tokens, num_seqs, out.data_ptr(), heads,
+                               groups, dim, vdim, _stream()), "ssd_steps")
+    launch_count += 1       # two kernels
+    return out
+
+
+def wkv_memory(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gate: torch.Tensor, low: torch.Tensor, w2: torch.Tensor,
+               w2t: torch.Tensor, w0: torch.Tensor, bonus: torch.Tensor, state: torch.Tensor, query_start_loc: torch.Tensor,
+               state_slots: torch.Tensor, num_seqs: int, heads: int, dim: int, norm_weight: torch.Tensor, eps: float,
+               out: torch.Tensor, max_query_len: int = 0) -> torch.Tensor:
+    """The memory of an RWKV-style layer, token by token, on a 32-bit state per request and head, its norm and its gate.
+
+    r, k, v, gate [tokens, heads * dim] (rows equally far apart); low [tokens, rank].  Per head and channel the decay is
+    w = exp(-exp(w2 tanh(low) + w0));  o = (S + diag(bonus) k v^T)^T r, then S <- diag(w) S + k v^T;
+    out[t, h] = o / sqrt(mean(o^2) + eps) * norm_weight[h] * silu(gate).  w2 [heads * dim, rank] and its transpose w2t in the
+    engine's dtype; w0, bonus, norm_weight float32 [heads * dim]; out [tokens, heads * dim] in the engine's dtype.  state
+    [slots, heads, dim, dim] float32 (S kept column by column) is read and written."""
+    global launch_count
+    for t, what in ((r, "r"), (k, "k"), (v, "v"), (gate, "gate"), (low, "low"), (out, "out")):
+        _rows2d(t, what)
+    _on_gpu(w2, w2t, w0, bonus, state, query_start_loc, state_slots, norm_weight)
+    _int32(query_start_loc, "query_start_loc"); _int32(state_slots, "state_slots")
+    tokens, width = r.shape
+    rank = low.shape[1]
+    assert width == heads * dim and k.shape == v.shape == gate.shape == out.shape == r.shape and low.shape[0] == tokens
+    assert k.stride(0) == v.stride(0) == gate.stride(0) == r.stride(0)
+    assert r.dtype == k.dtype == v.dtype == gate.dtype == low.dtype == w2.dtype == w2t.dtype == out.dtype
+    assert w2.shape == (width, rank) and w2t.shape == (rank, width)
+    assert w0.dtype == bonus.dtype == norm_weight.dtype == state.dtype == torch.float32
+    assert w0.numel() == bonus.numel() == norm_weight.numel() == width and state.shape[1:] == (heads, dim, dim)
+    if max_query_len == 1:
+        _check(_fn("li_wkv_token")(_code(r), r.data_ptr(), k.data_ptr(), v.data_ptr(), gate.data_ptr(), r.stride(0),
+                                   low.data_ptr(), low.stride(0), rank, w2.data_ptr(), w0.data_ptr(), bonus.data_ptr(),
+                                   state.data_ptr(), query_start_loc.data_ptr(), state_slots.data_ptr(), num_seqs,
+                                   norm_weight.data_ptr(), float(eps), out.data_ptr(), out.stride(0), heads, dim,
+                                   _stream()), "wkv_token")
+        return out
+    records = _memory_records(False, dim, dim, tokens * heads, tokens * heads, r.device)
+    read = torch.empty((tokens, width), dtype=torch.float32, device=r.device)
+    share = torch.empty((tokens, heads), dtype=torch.float32, device=r.device)
+    _check(_fn("li_wkv_steps")(_code(r), r.data_ptr(), k.data_ptr(), v.data_ptr(), r.stride(0), low.data_ptr(),
+                               low.stride(0), rank, w2t.data_ptr(), w0.data_ptr(), bonus.data_ptr(), records[0].data_ptr(),
+                               records[1].data_ptr(), share.data_ptr(), state.data_ptr(), query_start_loc.data_ptr(),
+                               state_slots.data_ptr(), tokens, num_seqs, read.data_ptr(), heads, dim, _stream()), "wkv_steps")
+    launch_count += 1       # two kernels
+    return gated_rmsnorm(read, gate, norm_weight, eps, out, heads, add=v, add_scale=share)
+
+
+def token_shift_step(x: torch.Tensor, mu: torch.Tensor, before: torch.Tensor, seq_of_token: torch.Tensor,
+                     query_start_loc: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, out: torch.Tensor,
+                     single_tokens: bool = False) -> torch.Tensor:
+    """out[i, t] = x[t] + (x[t - 1] - x[t]) * mu[i] for every i; in front of a sequence's first token of the step stands
+    before[slot], which afterwards is the sequence's last token of it.  x [tokens, width], before [slots, 1, width] and out
+    [count, tokens, width] in the engine's dtype, mu [count, width] float32; 32-bit inside.  Tokens whose sequence is -1
+    give zeros.  `single_tokens`: every sequence brings exactly one token, and one launch does both."""
+    _on_gpu(x, mu, before, seq_of_token, query_start_loc, state_slots, out)
+    _int32(seq_of_token, "seq_of_token"); _int32(query_start_loc, "query_start_loc"); _int32(state_slots, "state_slots")
+    tokens, width = x.shape
+    count = mu.shape[0]
+    assert mu.shape == (count, width) and mu.dtype == torch.float32 and before.shape[1:] == (1, width)
+    assert out.shape == (count, tokens, width) and x.dtype == before.dtype == out.dtype
+    _check(_fn("li_token_shift")(_code(x), x.data_ptr(), mu.data_ptr(), count, before.data_ptr(), seq_of_token.data_ptr(),
+                                 query_start_loc.data_ptr(), state_slots.data_ptr(), out.data_ptr(), tokens, width,
+                                 int(single_tokens), _stream()), "token_shift")
+    if not single_tokens:
+        short_conv_update(x, before, query_start_loc, state_slots, num_seqs)
+    return out
 
 
 # ------------------------------------------- several residual streams, latent attention
@@ -1661,6 +1905,7 @@ def gate_heads(v: torch.Tensor, gate: torch.Tensor | None, out: torch.Tensor) ->
 
 # ------------------------------------------------------------- mixture of experts
 EXPERT_ACTIVATIONS = {"swiglu": 0, "capped_swiglu": 1}
+UNGATED_EXPERT_ACTIVATIONS = ("relu_squared",)       # of experts that have no gate: down_e(act(up_e x))
 
 
 @dataclass
@@ -1700,13 +1945,18 @@ def moe_route(logits: torch.Tensor, top: int, groups: int, keep: int, renormalis
 
 def moe_router(x: torch.Tensor, weight: torch.Tensor, top: int, groups: int, keep: int, renormalise: bool,
                ids: torch.Tensor, weights: torch.Tensor, scores: str = "softmax", correction: torch.Tensor | None = None,
-               rank_by: int = 1, floor: float = 0.0, gated: bool = False, gate: torch.Tensor | None = None) -> None:
+               rank_by: int = 1, floor: float = 0.0, gated: bool = False, gate: torch.Tensor | None = None,
+               identity: torch.Tensor | None = None, identity_experts: int = 0) -> None:
     """`moe_route` of the logits x @ weight^T, product and routing in one launch: x [tokens, hidden] in the engine's
     dtype (a column slice is fine), weight [experts, hidden] float32; the product is 32-bit, its sums in an order that
     depends on nothing but the sizes.  `gated`: weight has one more row, and the sigmoid of its logit, one number per
     token, goes to `gate` [tokens] float32 (None: nowhere) and is the weight of the slots that ids and weights have
-    behind the first `top`; those hold the experts number `experts`, `experts` + 1, ... (experts that every token runs)."""
-    _on_gpu(weight, ids, weights, correction, gate)
+    behind the first `top`; those hold the experts number `experts`, `experts` + 1, ... (experts that every token runs).
+    `identity_experts`: the last so many rows of weight are of experts that give back what they read; they are scored and
+    chosen like the others, and `identity` [tokens] float32 receives the sum of a token's weights of them."""
+    _on_gpu(weight, ids, weights, correction, gate, identity)
+    assert (identity_experts > 0) == (identity is not None)
+    assert identity is None or (identity.dtype == torch.float32 and identity.numel() == x.shape[0])
     _rows2d(x, "x")
     _int32(ids, "ids")
     tokens, hidden = x.shape
@@ -1720,7 +1970,7 @@ def moe_router(x: torch.Tensor, weight: torch.Tensor, top: int, groups: int, kee
     _check(_fn("li_moe_router")(_code(x), x.data_ptr(), x.stride(0), weight.data_ptr(), tokens, hidden, experts, top,
                                 groups, keep, int(renormalise), ROUTER_SCORES[scores], rank_by - 1, float(floor),
                                 _ptr(correction), int(gated), extra, ids.data_ptr(), weights.data_ptr(), _ptr(gate),
-                                _stream()), "moe_router")
+                                int(identity_experts), _ptr(identity), _stream()), "moe_router")
 
 
 # LITEINFER_MOE_TCGEN05: 1 (default) = bfloat16 experts of steps with at least LITEINFER_MOE_TCGEN05_MIN_PAIRS (1) pairs of
@@ -1743,8 +1993,10 @@ def moe_tile_rows(dtype: torch.dtype, hidden: int, ff: int, pairs: int | None = 
     return 64 if both else 32
 
 
-def moe_sort(ids: torch.Tensor, experts: int, tile_rows: int, with_place: bool = False) -> ExpertPlan:
-    """The plan of a step whose pair p = token * top + slot goes to expert ids.flatten()[p]."""
+def moe_sort(ids: torch.Tensor, experts: int, tile_rows: int, with_place: bool = False, in_pairs: bool = False) -> ExpertPlan:
+    """The plan of a step whose pair p = token * top + slot goes to expert ids.flatten()[p]; a pair whose number is none of
+    the experts' is in no run, and its place is -1.  `in_pairs`: the place of the others is the pair itself (their rows are
+    to lie in the order of the pairs)."""
     _on_gpu(ids)
     _int32(ids, "ids")
     pairs = ids.numel()
@@ -1756,19 +2008,19 @@ def moe_sort(ids: torch.Tensor, experts: int, tile_rows: int, with_place: bool =
     tile_row0 = scratch[pairs + experts + 1 + max_tiles:pairs + experts + 1 + 2 * max_tiles]
     place = scratch[pairs + experts + 1 + 2 * max_tiles:] if with_place else None
     _check(_fn("li_moe_sort")(ids.data_ptr(), pairs, experts, tile_rows, offsets.data_ptr(), order.data_ptr(),
-                              tile_expert.data_ptr(), tile_row0.data_ptr(), max_tiles, _ptr(place), _stream()),
+                              tile_expert.data_ptr(), tile_row0.data_ptr(), max_tiles, _ptr(place), int(in_pairs), _stream()),
            "moe_sort")
     return ExpertPlan(order, offsets, tile_expert, tile_row0, tile_rows, max_tiles, place)
 
 
 def moe_gather(x: torch.Tensor, plan: ExpertPlan, top: int, out: torch.Tensor) -> torch.Tensor:
-    """out[m] = x[plan.order[m] // top]: every pair's token row, in the order of the experts' runs."""
+    """out[m] = x[plan.order[m] // top]: the token row of every pair that has an expert, in the order of their runs."""
     _on_gpu(out)
     _rows2d(x, "x")
     pairs = plan.order.numel()
     assert out.shape == (pairs, x.shape[1]) and out.dtype == x.dtype and out.is_contiguous()
     _check(_fn("li_moe_gather")(_code(x), x.data_ptr(), x.stride(0), plan.order.data_ptr(), top, out.data_ptr(), pairs,
-                                x.shape[1], _stream()), "moe_gather")
+                               plan.offsets[-1:].data_ptr(), x.shape[1], _stream()), "moe_gather")
     return out
 
 
@@ -1777,13 +2029,15 @@ def moe_grouped_tcgen05(mode: str, a: torch.Tensor, weight: torch.Tensor, out: t
                         pair_weights: torch.Tensor | None = None) -> torch.Tensor:
     """`moe_grouped` on the tcgen05 kernel (bfloat16): `a` [pairs, K] and `out` hold their rows in the order of the
     experts' runs (`plan.order`), the plan's tiles are 128 rows, and in mode "gate_up" an expert's gate and up rows lie
-    interleaved in eights.  mode "down" multiplies row m by pair_weights[plan.order[m]]."""
+    interleaved in eights.  mode "down" multiplies row m by pair_weights[plan.order[m]]; mode "up": experts without a gate."""
     _on_gpu(a, weight, out, pair_weights)
     experts, rows, K = weight.shape
     pairs = plan.order.numel()
-    assert plan.tile_rows == 128 and mode in ("gate_up", "down") and a.dtype == weight.dtype == out.dtype == torch.bfloat16
+    assert plan.tile_rows == 128 and mode in ("gate_up", "down", "up") and a.dtype == weight.dtype == out.dtype == torch.bfloat16
     assert a.shape == (pairs, K) and out.shape == (pairs, rows // 2 if mode == "gate_up" else rows)
-    act = -1 if mode == "down" else {"swiglu": 0, "capped_swiglu": 4}[activation]
+    act = {"down": -1, "up": -2}.get(mode)
+    if act is None:
+        act = {"swiglu": 0, "capped_swiglu": 4}[activation]
     scale = pair_weights if mode == "down" else None
     _check(_fn("li_gemm_tcgen05_grouped")(
         a.data_ptr(), weight.data_ptr(), out.data_ptr(), pairs, rows, K, experts, act, float(limit), float(alpha),
@@ -1800,19 +2054,20 @@ def moe_grouped(mode: str, a: torch.Tensor, weight: torch.Tensor, out: torch.Ten
     for pair p of expert e; a [tokens, hidden], weight [experts, 2 * ff, hidden] (an expert's gate rows, then its up
     rows), out [pairs, ff]; `activation` of `EXPERT_ACTIVATIONS` ("capped_swiglu": g' = min(g, limit), u' = clamp(u,
     -limit, limit), g' * sigmoid(alpha * g') * (u' + 1)).  mode "down": out[p] = (W_down,e a[p]) * pair_weights[p];
-    a [pairs, ff], weight [experts, hidden, ff], out [pairs, hidden].  `eights` (mode "gate_up"): an expert's gate and
+    a [pairs, ff], weight [experts, hidden, ff], out [pairs, hidden].  mode "up" (experts without a gate): out[p] = relu(W_up,e
+    a[p // top])^2, weight [experts, ff, hidden].  `eights` (mode "gate_up"): an expert's gate and
     up rows lie interleaved in eights (eight gate rows, then their eight up rows) instead of one half after the other."""
     _on_gpu(a, weight, out, pair_weights)
     _rows2d(a, "a")
-    assert mode in ("gate_up", "down") and a.dtype == weight.dtype == out.dtype and out.is_contiguous()
+    assert mode in ("gate_up", "down", "up") and a.dtype == weight.dtype == out.dtype and out.is_contiguous()
     experts, rows, K = weight.shape
     N = rows // 2 if mode == "gate_up" else rows
     assert weight.is_contiguous() and a.shape[1] == K and out.shape == (plan.order.numel(), N)
     assert pair_weights is None or (pair_weights.dtype == torch.float32 and pair_weights.numel() == plan.order.numel())
-    _check(_fn("li_moe_grouped")(_code(a), 0 if mode == "gate_up" else 1, a.data_ptr(), a.stride(0), weight.data_ptr(),
+    _check(_fn("li_moe_grouped")(_code(a), {"gate_up": 0, "down": 1, "up": 2}[mode], a.data_ptr(), a.stride(0), weight.data_ptr(),
                                  out.data_ptr(), out.stride(0), plan.order.data_ptr(), plan.offsets.data_ptr(),
                                  plan.tile_expert.data_ptr(), plan.tile_row0.data_ptr(), _ptr(pair_weights), top, N, K,
-                                 EXPERT_ACTIVATIONS[activation], float(limit), float(alpha), plan.max_tiles,
+                                 EXPERT_ACTIVATIONS[activation] if mode == "gate_up" else 0, float(limit), float(alpha), plan.max_tiles,
                                  plan.tile_rows, int(eights), _stream()), "moe_grouped")
     return out
 
@@ -1829,27 +2084,31 @@ def moe_combine(y: torch.Tensor, out: torch.Tensor, top: int, place: torch.Tenso
 
 
 def moe_expert_rows(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,
-                    activation: str, limit: float, alpha: float, eights: bool) -> RoutedRows:
+                    activation: str, limit: float, alpha: float, eights: bool, partial: bool = False) -> RoutedRows:
     """weights[t, s] * down_e(act(gate_e x[t], up_e x[t])), e = ids[t, s], for every pair (t, s): the chosen experts'
     rows, their products grouped by expert, not yet added up.  gate_up [experts, 2 * ff, hidden] (`eights`: gate and up
     rows interleaved in eights), down [experts, hidden, ff].  Steps of many pairs in bfloat16 run the tcgen05 kernel
-    over the pairs' rows gathered expert by expert; the others the mma.sync or FFMA tiles, which gather as they load."""
+    over the pairs' rows gathered expert by expert; the others the mma.sync or FFMA tiles, which gather as they load.  `activation` of
+    `UNGATED_EXPERT_ACTIVATIONS`: gate_up is [experts, ff, hidden], the up rows alone.  `partial`: some pairs have no expert
+    (ids beyond theirs), and no row."""
     tokens, top = ids.shape
     experts, hidden, ff = down.shape
     pairs = tokens * top
-    tile = moe_tile_rows(x.dtype, hidden, ff, pairs if eights else None)
-    plan = moe_sort(ids, experts, tile, with_place=tile == 128)
+    gated = activation not in UNGATED_EXPERT_ACTIVATIONS
+    first = "gate_up" if gated else "up"
+    tile = moe_tile_rows(x.dtype, hidden, ff, pairs if eights or not gated else None)
+    plan = moe_sort(ids, experts, tile, with_place=tile == 128 or partial, in_pairs=tile != 128)
     act = torch.empty((pairs, ff), dtype=x.dtype, device=x.device)
     each = torch.empty((pairs, hidden), dtype=x.dtype, device=x.device)
     scale = weights.view(-1)
     if tile == 128:
         rows = moe_gather(x, plan, top, torch.empty((pairs, hidden), dtype=x.dtype, device=x.device))
-        moe_grouped_tcgen05("gate_up", rows, gate_up, act, plan, activation, limit, alpha)
+        moe_grouped_tcgen05(first, rows, gate_up, act, plan, activation, limit, alpha)
         moe_grouped_tcgen05("down", act, down, each, plan, pair_weights=scale)
         return RoutedRows(each, top, plan.place)
-    moe_grouped("gate_up", x, gate_up, act, plan, top, activation, limit, alpha, eights=eights)
+    moe_grouped(first, x, gate_up, act, plan, top, activation, limit, alpha, eights=eights)
     moe_grouped("down", act, down, each, plan, top, pair_weights=scale)
-    return RoutedRows(each, top)
+    return RoutedRows(each, top, plan.place)
 
 
 def moe_experts(x: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor,

@@ -35,8 +35,8 @@ NVCC_FLAGS = [
 ]
 
 # Source file (without .cu) of every library.
-SOURCES = ("elementwise", "layernorm", "stream_mix", "delta_rule", "hgrn2", "mlstm", "rope_cache", "attention_generic", "attention_latent", "attention_latent_mma", "attention_mma", "attention_stream", "attention_tcgen05",
-           "gemm_simt", "gemm_skinny", "gemm_skinny_static", "gemm_stream", "gemm_tcgen05", "moe", "sampling", "sum_norms")
+SOURCES = ("elementwise", "layernorm", "stream_mix", "delta_rule", "hgrn2", "linear_memory", "mlstm", "rope_cache", "attention_generic", "attention_latent", "attention_latent_mma", "attention_mma", "attention_stream", "attention_tcgen05",
+           "gemm_simt", "gemm_skinny", "gemm_skinny_static", "gemm_stream", "gemm_tcgen05", "moe", "output_norm", "sampling", "sum_norms")
 
 
 class KernelLibraryError(RuntimeError):

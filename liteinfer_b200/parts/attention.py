@@ -44,11 +44,16 @@ class Attention:
     in `ctx.extras[value_mix_key]` for later layers; "mixed" stores (1 - l) v + l v_source instead of v, l the
     scalar tensor `value_mix` and v_source what the source layer left for the same tokens.  `chunk` (instead of a
     window): positions form chunks of that many from the sequence's start, and a query reads the keys of its own chunk
-    only.  Everything that reads x is one product against the concatenated weights.
+    only.  `values_are_keys`: there is no value projection; what is stored as a token's value is its key as projected (with
+    its bias, before norm and rotation).  `fixed_sink`: a sink as above whose number is a constant for all heads (0: the
+    softmax's denominator is 1 larger than the sum of the exponentials).  Everything that reads x is one product against the
+    concatenated weights; where q and k are normalised over the projection and there are biases or no values of their own,
+    biases, norm, rotation and the cache write are one kernel behind it (`joint_norm`).
 
     `pad_heads`: in bfloat16 on a GPU, keys and values whose sizes no tensor-core kernel takes are rounded up to sizes
     that one does (`tensor_core_sizes`): the added rows of the projections and columns of `o_proj.weight` are zeros, so
-    every score and every output is the same sum.  (Not with q/k norms, biases, mixed values or an output gate.)
+    every score and every output is the same sum.  (Not with mixed values or an output gate; with q/k norms or biases only
+    where they are those of `joint_norm`.)
 
     A mixer that runs several side by side (parts/side_by_side.py) makes one product of their projections and one of
     their output projections; it uses `in_weight`, `out_weight` and `mix`.
@@ -61,7 +66,14 @@ class Attention:
                  qk_norm: str | None = None, qk_norm_eps: float = 1e-6, head_gate: bool = False,
                  value_mix: str | None = None, value_mix_key: str = "value_mix", qk_norm_weight: bool = True,
                  qk_norm_after_rotation: bool = False, sink: bool = False, output_gate: bool = False,
-                 chunk: int | None = None, pad_heads: bool = False) -> None:
+                 chunk: int | None = None, pad_heads: bool = False, values_are_keys: bool = False,
+                 fixed_sink: float | None = None) -> None:
+        if values_are_keys and (qk_norm != "projection" or v_head_dim not in (None, head_dim) or value_mix or head_gate
+                                or output_gate):
+            raise ValueError("values that are the keys as projected go with qk_norm='projection', heads of one size, and "
+                             "neither gates nor mixed values")
+        if sink and fixed_sink is not None:
+            raise ValueError("an attention has learned sinks or a fixed one")
         if window is not None and chunk is not None:
             raise ValueError("an attention has a window or chunks, not both")
         if heads % kv_heads:
@@ -77,6 +89,8 @@ class Attention:
         self.qk_norm_weight, self.qk_norm_after_rotation = bool(qk_norm_weight), bool(qk_norm_after_rotation)
         self.has_sink, self.output_gate = bool(sink), bool(output_gate)
         self.sink: torch.Tensor | None = None
+        self.values_are_keys = bool(values_are_keys)
+        self.fixed_sink = None if fixed_sink is None else float(fixed_sink)
         self.head_gate, self.value_mix, self.value_mix_key = bool(head_gate), value_mix, value_mix_key
         self.blend: torch.Tensor | None = None
         self.hidden_size, self.heads, self.kv_heads, self.head_dim = hidden_size, heads, kv_heads, head_dim
@@ -94,8 +108,11 @@ class Attention:
         self.position = build_part("position", position, dtype=dtype, device=device)
         # The sizes of the checkpoint's heads; head_dim and v_head_dim are those of the rows that are computed and kept.
         self.key_size, self.value_size = self.head_dim, self.v_head_dim
+        self.joint_norm = (qk_norm == "projection" and (values_are_keys or self.bias or pad_heads)
+                           and not (self.head_gate or self.output_gate or value_mix))
+        self.prep_bias: torch.Tensor | None = None      # float32, of the kernel behind the projection (joint_norm)
         if (pad_heads and dtype == torch.bfloat16 and torch.device(device).type == "cuda"
-                and not (qk_norm or bias or value_mix or output_gate)):
+                and (self.joint_norm or not (qk_norm or bias)) and not (value_mix or output_gate)):
             sizes = ops.tensor_core_sizes(self.head_dim, self.v_head_dim, heads, kv_heads)
             if sizes is not None:
                 self.head_dim, self.v_head_dim = sizes
@@ -112,13 +129,16 @@ class Attention:
             "v_proj.weight": TensorSpec((v, self.hidden_size)),
             "o_proj.weight": TensorSpec((self.hidden_size, self.heads * self.value_size)),
         }
+        if self.values_are_keys:
+            del specs["v_proj.weight"]
         if self.qk_norm == "head":
             if self.qk_norm_weight:
                 specs.update({"q_norm.weight": TensorSpec((self.head_dim,), init="ones_normal"),
                               "k_norm.weight": TensorSpec((self.head_dim,), init="ones_normal")})
         elif self.qk_norm:
-            specs.update({"q_norm.weight": TensorSpec((q,), init="ones_normal"),
-                          "k_norm.weight": TensorSpec((kv,), init="ones_normal")})
+            kind = "f32" if self.joint_norm else "weight"
+            specs.update({"q_norm.weight": TensorSpec((q,), kind, init="ones_normal"),
+                          "k_norm.weight": TensorSpec((kv,), kind, init="ones_normal")})
         if self.head_gate:
             specs["g_proj.weight"] = TensorSpec((self.heads, self.hidden_size))
         if self.output_gate:
@@ -130,6 +150,8 @@ class Attention:
         if self.bias:
             specs.update({"q_proj.bias": TensorSpec((q,), init="zeros"), "k_proj.bias": TensorSpec((kv,), init="zeros"),
                           "v_proj.bias": TensorSpec((v,), init="zeros")})
+            if self.values_are_keys:
+                del specs["v_proj.bias"]
         if self.out_bias:
             specs["o_proj.bias"] = TensorSpec((self.hidden_size,), init="zeros")
         for name, spec in self.position.tensor_specs().items():
@@ -137,8 +159,9 @@ class Attention:
         return specs
 
     def bind(self, tensors: dict[str, torch.Tensor]) -> None:
-        weights = [tensors["q_proj.weight"], tensors["k_proj.weight"], tensors["v_proj.weight"]]
-        biases = [tensors[n] for n in ("q_proj.bias", "k_proj.bias", "v_proj.bias")] if self.bias else []
+        names = ("q_proj", "k_proj") if self.values_are_keys else ("q_proj", "k_proj", "v_proj")
+        weights = [tensors[n + ".weight"] for n in names]
+        biases = [tensors[n + ".bias"] for n in names] if self.bias else []
         order = self.position.pair_order() if hasattr(self.position, "pair_order") else None
         if order is not None:
             # The checkpoint pairs neighbouring dimensions: every head's rows of q and k (and what belongs to those
@@ -150,9 +173,9 @@ class Attention:
                 biases[0], biases[1] = per_head(biases[0]), per_head(biases[1])
         o_weight = tensors["o_proj.weight"]
         if (self.head_dim, self.v_head_dim) != (self.key_size, self.value_size):
-            weights = [_padded_heads(w, old, new) for w, old, new in
-                       zip(weights, (self.key_size, self.key_size, self.value_size),
-                           (self.head_dim, self.head_dim, self.v_head_dim))]
+            sizes = ((self.key_size, self.head_dim), (self.key_size, self.head_dim), (self.value_size, self.v_head_dim))
+            weights = [_padded_heads(w, *size) for w, size in zip(weights, sizes)]
+            biases = [_padded_heads(b[:, None], *size)[:, 0] for b, size in zip(biases, sizes)]
             o_weight = _padded_heads(o_weight.t(), self.value_size, self.v_head_dim).t().contiguous()
         if self.head_gate or self.output_gate:
             # The gate's rows ride behind v, filled up to a multiple of 16 rows (what the products' tiles like).
@@ -162,7 +185,9 @@ class Attention:
             if self.bias:
                 biases.append(biases[0].new_zeros(gate.shape[0] + pad))
         self.qkv_weight = torch.cat(weights).contiguous()
-        if self.bias:
+        if self.bias and self.joint_norm:
+            self.prep_bias = torch.cat(biases).to(torch.float32).contiguous()
+        elif self.bias:
             self.qkv_bias = torch.cat(biases).contiguous()
         if self.value_mix == "mixed":
             self.blend = tensors["value_mix"].to(torch.float32).reshape(1).contiguous()
@@ -173,8 +198,13 @@ class Attention:
                 self.q_norm_weight, self.k_norm_weight = self.q_norm_weight[at].contiguous(), self.k_norm_weight[at].contiguous()
             elif order is not None:
                 self.q_norm_weight, self.k_norm_weight = per_head(self.q_norm_weight), per_head(self.k_norm_weight)
+        if self.joint_norm and self.head_dim != self.key_size:
+            self.q_norm_weight, self.k_norm_weight = (_padded_heads(w[:, None], self.key_size, self.head_dim)[:, 0].contiguous()
+                                                      for w in (self.q_norm_weight, self.k_norm_weight))
         if self.has_sink:
             self.sink = tensors["sink"].to(torch.float32).contiguous()
+        elif self.fixed_sink is not None:
+            self.sink = torch.full((self.heads,), self.fixed_sink, dtype=torch.float32, device=self.qkv_weight.device)
         self.o_bias = tensors.get("o_proj.bias") if self.out_bias else None
         self.position.bind({n[len("position."):]: t for n, t in tensors.items() if n.startswith("position.")})
 
@@ -198,7 +228,7 @@ class Attention:
 
     @property
     def has_biases(self) -> bool:
-        return self.bias or self.out_bias
+        return (self.bias and not self.joint_norm) or self.out_bias
 
     takes_pending_norm = True       # x may be an ops.PendingNorm: the qkv product folds the norm in
     adds_to_residual = True         # the output projection adds into the residual stream where its kernel can
@@ -221,10 +251,10 @@ class Attention:
         if self.sink is not None:
             masked["sink"] = self.sink
         prepared = self.qk_norm == "head" or self.head_gate or self.output_gate or self.value_mix
-        if self.qk_norm and not prepared:
+        if self.qk_norm and not prepared and not self.joint_norm:
             ops.qk_projection_rmsnorm_(qkv[:, :q_width], self.q_norm_weight, qkv[:, q_width:q_width + kv_width],
                                        self.k_norm_weight, self.qk_norm_eps)
-        plain = (not masked and not prepared and self.v_head_dim % self.head_dim == 0
+        plain = (not masked and not prepared and not self.joint_norm and self.v_head_dim % self.head_dim == 0
                  and (rotary is None or rotary.attention_scaling == 1.0))
         newest = {}
         if plain and rotary is not None and ops.fused_decode_supports(qkv.dtype, self.heads, self.kv_heads, self.head_dim,
@@ -254,6 +284,14 @@ class Attention:
         if rotary is None:
             self.position.apply(qkv[:, :q_width].unflatten(1, (self.heads, self.head_dim)),
                                 qkv[:, q_width:q_width + kv_width].unflatten(1, (self.kv_heads, self.head_dim)), ctx)
+        if self.joint_norm:
+            ops.projection_norm_rope_kv_write(
+                qkv, ctx.positions, ctx.seq_of_token, table, kv.k_pool, kv.v_pool, rotary.inv_freq if rotary else None,
+                self.heads, self.kv_heads, self.head_dim, rotary.rotary_dim if rotary else 0, self.q_norm_weight,
+                self.k_norm_weight, self.heads * self.key_size, self.kv_heads * self.key_size, self.qk_norm_eps,
+                bias=self.prep_bias, values_are_keys=self.values_are_keys, store=not cache.read_only,
+                cos_sin_scale=rotary.attention_scaling if rotary else 1.0)
+            return
         if not prepared and qkv.is_contiguous() and qkv.shape[1] == q_width + kv_width + v_width:
             plain = self.v_head_dim == self.head_dim and (rotary is None or rotary.attention_scaling == 1.0)
             wide = {} if plain else dict(v_head_dim=self.v_head_dim,

@@ -156,7 +156,9 @@ class OutputNormBlock:
     """h = h + norm(mixer(h)); h = h + norm'(feed_forward(h)): the sublayers read the stream as it is, and only
     what they give back is normalised.  The normalised output travels as an `ops.NormedDelta`; whoever reads the
     stream next adds it: this block's `_read` (one kernel: the outgoing norm, the 32-bit sum, and the sum rounded
-    to the engine's dtype for the sublayer's products) or the model's final norm."""
+    to the engine's dtype for the sublayer's products) or the model's final norm.  A sublayer may leave its output as a sum
+    still to be made (`ops.SumDelta`: experts' rows, mixers side by side that are each normalised first); the same kernel
+    then makes it."""
 
     roles = {"mixer": "mixer", "mixer_out_norm": "norm", "feed_forward": "feed_forward",
              "feed_forward_out_norm": "norm"}
@@ -171,6 +173,9 @@ class OutputNormBlock:
         """Adds the pending delta into the stream and returns the stream in the engine's dtype."""
         narrow = hidden.dtype != self.dtype
         out = torch.empty(hidden.shape, dtype=self.dtype, device=hidden.device) if narrow else None
+        if isinstance(delta, ops.NormedDelta) and isinstance(delta.value, ops.SumDelta):
+            ops.output_norm(hidden, delta, out)
+            return out if narrow else hidden
         if isinstance(delta, ops.NormedDelta):
             ops.layernorm_add(hidden, delta.value, delta.weight, delta.eps, centred=delta.centred, out=out)
             return out if narrow else hidden

@@ -18,13 +18,17 @@ class GatedMLP:
     """down(act(gate(x)) * up(x)) — liteinfer/models/llama.py:105-114.
 
     gate and up are one product against the concatenated weights; the activation
-    and the multiply are one kernel.
+    and the multiply are one kernel.  `activation` "capped_swiglu" joins them with caps instead: with g' = min(g, limit),
+    g' * sigmoid(alpha g') * (clamp(u, -limit, limit) + 1).
     """
 
     def __init__(self, hidden_size: int, intermediate_size: int, activation: str, dtype: torch.dtype,
-                 device: torch.device, bias: bool = False) -> None:
-        if activation not in ops.ACTIVATIONS:
-            raise ValueError(f"activation {activation!r} has no kernel; known: {sorted(ops.ACTIVATIONS)}")
+                 device: torch.device, bias: bool = False, limit: float = 0.0, alpha: float = 1.0) -> None:
+        if activation not in ops.GATED_ACTIVATIONS:
+            raise ValueError(f"activation {activation!r} has no kernel; known: {sorted(ops.GATED_ACTIVATIONS)}")
+        if activation == "capped_swiglu" and not limit > 0:
+            raise ValueError("the caps of 'capped_swiglu' must be > 0")
+        self.caps = dict(limit=float(limit), alpha=float(alpha)) if activation == "capped_swiglu" else {}
         self.hidden_size, self.intermediate_size, self.activation, self.bias = (
             hidden_size, intermediate_size, activation, bias)
         self.gate_up_weight = self.gate_up_bias = self.down_weight = self.down_bias = None
@@ -64,14 +68,14 @@ class GatedMLP:
         tokens = x.shape[0]
         hidden = torch.empty((tokens, self.intermediate_size), dtype=x.dtype, device=x.device)
         if self.interleaved and ops.gated_linear_supported(x, self.gate_up_weight):
-            ops.gated_linear(x, self.gate_up_weight, hidden, self.activation, self.gate_up_bias)
+            ops.gated_linear(x, self.gate_up_weight, hidden, self.activation, self.gate_up_bias, **self.caps)
         else:
             gate_up = torch.empty((tokens, 2 * self.intermediate_size), dtype=x.dtype, device=x.device)
             ops.linear(x, self.gate_up_weight, gate_up, self.gate_up_bias)
             if self.interleaved:
-                ops.act_mul_interleaved(gate_up, hidden, self.activation)
+                ops.act_mul_interleaved(gate_up, hidden, self.activation, **self.caps)
             else:
-                ops.act_mul(gate_up, hidden, self.activation)
+                ops.act_mul(gate_up, hidden, self.activation, **self.caps)
         return ops.linear(hidden, self.down_weight, None, self.down_bias, residual=residual)
 
 
@@ -119,6 +123,11 @@ class RoutedExperts:
     their weight: a down projection adds up over its columns, so the sum is the same and the grouped products do it all.
     Otherwise it runs as a gated feed-forward of its own.
 
+    `activation` of `ops.UNGATED_EXPERT_ACTIVATIONS`: the experts have no gate, down_e(act(up_e x)).
+
+    `identity` > 0: the router has that many more outputs, the last ones, which stand for experts without tensors that give
+    back what they read; they are scored and chosen like the others.
+
     `gives_sum`: `forward` returns the rows and terms not yet added up (`ops.SumDelta`).
     """
 
@@ -126,17 +135,21 @@ class RoutedExperts:
                  device: torch.device, groups: int = 1, groups_keep: int = 1, activation: str = "swiglu",
                  limit: float = 0.0, alpha: float = 1.0, renormalise: bool = False, scores: str = "softmax",
                  correction: bool = False, group_rank: int = 1, floor: float = 0.0, shared_size: int = 0,
-                 gives_sum: bool = False) -> None:
-        if activation not in ops.EXPERT_ACTIVATIONS:
-            raise ValueError(f"activation {activation!r} has no kernel; known: {sorted(ops.EXPERT_ACTIVATIONS)}")
+                 gives_sum: bool = False, identity: int = 0) -> None:
+        known = sorted((*ops.EXPERT_ACTIVATIONS, *ops.UNGATED_EXPERT_ACTIVATIONS))
+        if activation not in known:
+            raise ValueError(f"activation {activation!r} has no kernel; known: {known}")
+        if identity < 0 or (identity and (not gives_sum or groups != 1 or shared_size)):
+            raise ValueError("identity experts go with an output left to the stream's sum (gives_sum), without groups and "
+                             "without a shared expert")
         if scores not in ops.ROUTER_SCORES:
             raise ValueError(f"scores {scores!r} are not supported; known: {sorted(ops.ROUTER_SCORES)}")
         if group_rank not in (1, 2):
             raise ValueError("a group ranks by its largest choice score (1) or by the sum of its two largest (2)")
-        if not 1 <= top <= experts or groups < 1 or experts % groups or not 1 <= groups_keep <= groups:
+        if not 1 <= top <= experts + identity or groups < 1 or experts % groups or not 1 <= groups_keep <= groups:
             raise ValueError("a mixture of experts needs 1 <= top <= experts, groups that divide experts, and "
                              "1 <= groups_keep <= groups")
-        if groups_keep * (experts // groups) < top:
+        if groups_keep * (experts // groups) + identity < top:
             raise ValueError("the kept groups hold fewer experts than `top`")
         if shared_size and (not gives_sum or activation != "swiglu"):
             raise ValueError("a shared expert is a plain gated silu one, and its output is left to the stream's sum "
@@ -146,6 +159,7 @@ class RoutedExperts:
         self.limit, self.alpha, self.renormalise = float(limit), float(alpha), bool(renormalise)
         self.scores, self.has_correction, self.group_rank, self.floor = scores, bool(correction), group_rank, float(floor)
         self.shared_size, self.gives_sum = int(shared_size), bool(gives_sum)
+        self.identity, self.gated = int(identity), activation in ops.EXPERT_ACTIVATIONS
         # The shared expert as so many experts that every token runs (0: it has a feed-forward of its own).
         self.shared_slots = shared_size // intermediate_size if shared_size % intermediate_size == 0 else 0
         self.shared = (GatedMLP(hidden_size, shared_size, "silu", dtype, device)
@@ -156,11 +170,12 @@ class RoutedExperts:
 
     def tensor_specs(self) -> dict[str, TensorSpec]:
         f, h = self.intermediate_size, self.hidden_size
-        specs = {"router.weight": TensorSpec((self.experts, h), kind="f32")}
+        outputs = self.experts + self.identity
+        specs = {"router.weight": TensorSpec((outputs, h), kind="f32")}
         if self.has_correction:
-            specs["correction"] = TensorSpec((self.experts,), kind="f32", init=_correction_init)
+            specs["correction"] = TensorSpec((outputs,), kind="f32", init=_correction_init)
         for e in range(self.experts):
-            specs.update(_expert_specs(f"experts.{e}.", h, f))
+            specs.update(_expert_specs(f"experts.{e}.", h, f, self.gated))
         if self.shared_size:
             specs.update(_expert_specs("shared.", h, self.shared_size))
             specs["shared.sg.weight"] = TensorSpec((1, h), kind="f32")
@@ -172,6 +187,10 @@ class RoutedExperts:
             router = torch.cat([router, tensors["shared.sg.weight"].to(torch.float32)])
         self.router = router.contiguous()
         self.correction = tensors["correction"].to(torch.float32).contiguous() if self.has_correction else None
+        if not self.gated:
+            stack = lambda n: torch.stack([tensors[f"experts.{e}.{n}_proj.weight"] for e in range(self.experts)]).contiguous()
+            self.gate_up, self.down = stack("up"), stack("down")        # [experts, ff, hidden]: the up rows alone
+            return
         # [experts, 2 * ff, hidden]: an expert's gate rows, then its up rows; in bfloat16 with a width in eights both
         # interleaved in eights (eight gate rows, then their eight up rows), the layout whose product and activation
         # the tensor-core kernels do together.  [experts, hidden, ff].
@@ -192,9 +211,10 @@ class RoutedExperts:
         self.gate_up = torch.stack([pair(g, u) for g, u in zip(gates, ups)]).contiguous()
         self.down = torch.stack(downs).contiguous()
 
-    def route(self, x: torch.Tensor, gate: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
+    def route(self, x: torch.Tensor, gate: torch.Tensor | None = None,
+              identity: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor]:
         """(chosen experts [tokens, top + shared slots] int32, their weights, float32); `gate` [tokens] float32 receives
-        the shared expert's weight."""
+        the shared expert's weight, `identity` [tokens] float32 the sum of the identity experts' weights."""
         tokens, slots = x.shape[0], self.top + self.shared_slots
         ids = torch.empty((tokens, slots), dtype=torch.int32, device=x.device)
         weights = torch.empty((tokens, slots), dtype=torch.float32, device=x.device)
@@ -202,6 +222,8 @@ class RoutedExperts:
         if self.scores != "softmax" or self.has_correction or self.group_rank != 1 or self.floor or self.shared_size:
             options = dict(scores=self.scores, correction=self.correction, rank_by=self.group_rank, floor=self.floor,
                            gated=bool(self.shared_size), gate=gate)
+        if self.identity:
+            options.update(identity=identity, identity_experts=self.identity)
         ops.moe_router(x, self.router, self.top, self.groups, self.groups_keep, self.renormalise, ids, weights, **options)
         return ids, weights
 
@@ -212,6 +234,12 @@ class RoutedExperts:
             return ops.moe_experts(x, self.gate_up, self.down, ids, weights, self.activation, self.limit, self.alpha,
                                    self.eights, out)
         gate = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device) if self.shared is not None else None
+        if self.identity:
+            same = torch.empty((x.shape[0],), dtype=torch.float32, device=x.device)
+            ids, weights = self.route(x, None, same)
+            rows = ops.moe_expert_rows(x, self.gate_up, self.down, ids, weights, self.activation, self.limit, self.alpha,
+                                       self.eights, partial=True)
+            return ops.SumDelta((ops.SumTerm(x, 1.0, same),), rows)
         ids, weights = self.route(x, gate)
         rows = ops.moe_expert_rows(x, self.gate_up, self.down, ids, weights, self.activation, self.limit, self.alpha,
                                    self.eights)
@@ -219,7 +247,9 @@ class RoutedExperts:
         return ops.SumDelta(terms, rows)
 
 
-def _expert_specs(prefix: str, hidden: int, width: int) -> dict[str, TensorSpec]:
+def _expert_specs(prefix: str, hidden: int, width: int, gated: bool = True) -> dict[str, TensorSpec]:
+    if not gated:
+        return {prefix + "up_proj.weight": TensorSpec((width, hidden)), prefix + "down_proj.weight": TensorSpec((hidden, width))}
     return {prefix + "gate_proj.weight": TensorSpec((width, hidden)), prefix + "up_proj.weight": TensorSpec((width, hidden)),
             prefix + "down_proj.weight": TensorSpec((hidden, width))}
 

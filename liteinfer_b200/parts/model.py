@@ -19,11 +19,13 @@ import liteinfer_b200.parts.embedding  # noqa: F401
 import liteinfer_b200.parts.feed_forward  # noqa: F401
 import liteinfer_b200.parts.hgrn2  # noqa: F401
 import liteinfer_b200.parts.latent_attention  # noqa: F401
+import liteinfer_b200.parts.mamba2  # noqa: F401
 import liteinfer_b200.parts.mlstm  # noqa: F401
 import liteinfer_b200.parts.norm  # noqa: F401
 import liteinfer_b200.parts.position  # noqa: F401
 import liteinfer_b200.parts.reentry  # noqa: F401
 import liteinfer_b200.parts.side_by_side  # noqa: F401
+import liteinfer_b200.parts.wkv  # noqa: F401
 from liteinfer_b200 import ops
 from liteinfer_b200.parts.block import apply_norm
 from liteinfer_b200.parts.context import LayerCache, StepContext
@@ -38,7 +40,9 @@ def _settled(hidden: torch.Tensor, delta, copies: int | None = None) -> torch.Te
         if isinstance(delta, ops.StreamUpdate):
             ops.stream_rmsnorm(out, None, 0.0, None, update=delta)
         return out.view(out.shape[0], copies, -1).sum(1)
-    if isinstance(delta, ops.NormedDelta):
+    if isinstance(delta, ops.NormedDelta) and isinstance(delta.value, ops.SumDelta):
+        ops.output_norm(out, delta)
+    elif isinstance(delta, ops.NormedDelta):
         ops.layernorm_add(out, delta.value, delta.weight, delta.eps, centred=delta.centred)
     elif isinstance(delta, ops.SumDelta):
         ops.sum_norms(out, delta, (), 0.0, (), write_stream=True)

@@ -140,11 +140,15 @@ class AffineRMSNorm:
         if isinstance(delta, ops.SumDelta):
             ops.sum_norms(x, delta, (self.weight,), self.eps, (out,), rows=rows, write_stream=rows is None)
             return out
+        if isinstance(delta, ops.NormedDelta) and isinstance(delta.value, ops.SumDelta):
+            ops.output_norm(x, delta, out, self.weight, self.eps, rows=rows, write_stream=rows is None)
+            return out
         return ops.layernorm(x, self.weight, self.eps, out, delta=delta, rows=rows,
                              write_stream=delta is not None and rows is None, centre=False)
 
-    def normed_delta(self, value: torch.Tensor) -> "ops.NormedDelta":
-        """What a sublayer's output becomes when this norm stands between it and the stream."""
+    def normed_delta(self, value: "torch.Tensor | ops.SumDelta") -> "ops.NormedDelta":
+        """What a sublayer's output becomes when this norm stands between it and the stream; the output may be a sum still
+        to be made (`ops.SumDelta`), over a 32-bit stream."""
         return ops.NormedDelta(value, self.weight, self.eps, centred=False)
 
 

@@ -25,11 +25,20 @@ class TensorSpec:
     "ones_normal" (1 + N(0, 0.01)), "zeros", or a function `(shape, generator) ->
     float32 tensor` for a part whose parameters need a distribution of their own
     (a decay kept in log space, a gate that must be positive).
+    A size that only the checkpoint knows is None in `shape` (the part reads it off the tensor it is bound to); the
+    random-weights mode draws it as `free` wide.
     """
 
-    shape: tuple[int, ...]
+    shape: tuple[int | None, ...]
     kind: str = "weight"
     init: str | Callable[[tuple[int, ...], Any], Any] = "normal"
+    free: int = 0
+
+    def accepts(self, shape: tuple[int, ...]) -> bool:
+        return len(shape) == len(self.shape) and all(want in (None, got) for got, want in zip(shape, self.shape))
+
+    def drawn_shape(self) -> tuple[int, ...]:
+        return tuple(self.free if n is None else n for n in self.shape)
 
 
 @dataclass(frozen=True)

@@ -76,7 +76,7 @@ def load_model(model_dir: str | Path, dtype: torch.dtype, device: torch.device |
                         unexpected.append(name)
                     continue
                 got = tuple(f.get_slice(name).get_shape())
-                if got != tuple(want.shape):
+                if not want.accepts(got):
                     wrong_shape.append((name, got, tuple(want.shape)))
                     continue
                 tensors[name] = f.get_tensor(name).to(device=device, dtype=_target_dtype(want.kind, dtype))

@@ -31,19 +31,20 @@ def random_tensors(raw_config: dict[str, Any], seed: int, dtype: torch.dtype = t
     for name, want in model.tensor_specs().items():
         if name in spec.tied:
             continue
+        shape = want.drawn_shape()
         if want.kind == "int":
-            tensors[name] = torch.randint(0, 2 ** 15, want.shape, generator=generator, dtype=torch.int32)
+            tensors[name] = torch.randint(0, 2 ** 15, shape, generator=generator, dtype=torch.int32)
             continue
         if callable(want.init):
-            value = torch.as_tensor(want.init(tuple(want.shape), generator), dtype=torch.float32)
-            if tuple(value.shape) != tuple(want.shape):
-                raise ValueError(f"the init function of {name!r} returned shape {tuple(value.shape)}, not {tuple(want.shape)}")
+            value = torch.as_tensor(want.init(shape, generator), dtype=torch.float32)
+            if tuple(value.shape) != shape:
+                raise ValueError(f"the init function of {name!r} returned shape {tuple(value.shape)}, not {shape}")
         elif want.init == "zeros":
-            value = torch.zeros(want.shape, dtype=torch.float32)
+            value = torch.zeros(shape, dtype=torch.float32)
         elif want.init == "ones_normal":
-            value = 1.0 + 0.01 * torch.randn(want.shape, generator=generator, dtype=torch.float32)
+            value = 1.0 + 0.01 * torch.randn(shape, generator=generator, dtype=torch.float32)
         else:
-            value = 0.02 * torch.randn(want.shape, generator=generator, dtype=torch.float32)
+            value = 0.02 * torch.randn(shape, generator=generator, dtype=torch.float32)
         tensors[name] = value if want.kind == "f32" else value.to(dtype)
     return tensors
 

@@ -72,18 +72,25 @@ def _activate(x, activation):
     raise ValueError(activation)
 
 
-def act_mul(gate_up, out, activation):
+def _gated(g, u, activation, dtype, limit, alpha):
+    if activation == "capped_swiglu":
+        g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
+        return g * torch.sigmoid(alpha * g) * (u + 1.0)
+    return _r(_activate(g, activation), dtype) * u
+
+
+def act_mul(gate_up, out, activation, limit=0.0, alpha=1.0):
     w = out.shape[1]
     g, u = gate_up[:, :w].float(), gate_up[:, w:].float()
-    out.copy_((_r(_activate(g, activation), out.dtype) * u).to(out.dtype))
+    out.copy_(_gated(g, u, activation, out.dtype, limit, alpha).to(out.dtype))
     return out
 
 
-def act_mul_interleaved(gate_up, out, activation):
+def act_mul_interleaved(gate_up, out, activation, limit=0.0, alpha=1.0):
     rows, w = out.shape
     pairs = gate_up.float().view(rows, w // 8, 2, 8)
     g, u = pairs[:, :, 0].reshape(rows, w), pairs[:, :, 1].reshape(rows, w)
-    out.copy_((_r(_activate(g, activation), out.dtype) * u).to(out.dtype))
+    out.copy_(_gated(g, u, activation, out.dtype, limit, alpha).to(out.dtype))
     return out
 
 
@@ -91,10 +98,10 @@ def gated_linear_supported(x, weight):
     return False
 
 
-def gated_linear(x, weight, out, activation, bias=None):
+def gated_linear(x, weight, out, activation, bias=None, limit=0.0, alpha=1.0):
     gate_up = torch.empty(x.shape[0], weight.shape[0], dtype=x.dtype, device=x.device)
     linear(x, weight, gate_up, bias)
-    return act_mul_interleaved(gate_up, out, activation)
+    return act_mul_interleaved(gate_up, out, activation, limit, alpha)
 
 
 def linear(x, weight, out, bias=None, residual=None, activation=None):
@@ -269,12 +276,14 @@ def qk_projection_rmsnorm_(q, q_weight, k, k_weight, eps):
     projection_rmsnorm_(k, k_weight, eps)
 
 
-def gated_rmsnorm(x, gate, weight, eps, out, heads, gate_activation="silu", den=None):
+def gated_rmsnorm(x, gate, weight, eps, out, heads, gate_activation="silu", den=None, add=None, add_scale=None):
     tokens, width = out.shape
     size = width // heads
     v = x.view(tokens, heads, size)
     if den is not None:
         v = v / den.view(tokens, heads, 1)
+    if add is not None:
+        v = v + add_scale.view(tokens, heads, 1) * add.float().reshape(tokens, heads, size)
     y = _norm(v, eps, centre=False) * weight.float().view(-1, size)
     if gate is None:
         out.copy_(y.reshape(tokens, width).to(out.dtype))
@@ -283,6 +292,41 @@ def gated_rmsnorm(x, gate, weight, eps, out, heads, gate_activation="silu", den=
     act = torch.sigmoid(g) if gate_activation == "sigmoid" else g / (1.0 + torch.exp(-g))
     out.copy_((y.reshape(tokens, width) * act).to(out.dtype))
     return out
+
+
+def gated_group_norm(x, gate, weight, eps, out, groups, add=None, skip=None):
+    y = x.float()
+    if add is not None:
+        y = y + skip.repeat_interleave(x.shape[1] // skip.numel()) * add.float()
+    g = gate.float()
+    y = y * (g / (1.0 + torch.exp(-g)))
+    out.copy_((_norm(y.unflatten(1, (groups, -1)), eps, centre=False).flatten(1) * weight).to(out.dtype))
+    return out
+
+
+def projection_norm_rope_kv_write(qkv, positions, seq_of_token, block_table, k_pool, v_pool, inv_freq, heads, kv_heads,
+                                  head_dim, rotary_dim, q_norm, k_norm, q_count, k_count, norm_eps, bias=None,
+                                  values_are_keys=False, store=True, cos_sin_scale=1.0):
+    """Norms over the whole projection (divided by the numbers that count), then what `rope_kv_write` does, on a compact
+    32-bit copy of the row."""
+    T, dtype = qkv.shape[0], qkv.dtype
+    vd = v_pool.shape[-1]
+    qw, kw = heads * head_dim, kv_heads * head_dim
+    columns = qw + kw + (0 if values_are_keys else kv_heads * vd)
+    row = qkv[:, :columns].float()
+    if bias is not None:
+        row = row + bias[:columns]
+    q, k = row[:, :qw], row[:, qw:qw + kw]
+    v = k if values_are_keys else row[:, qw + kw:]
+    q = q / torch.sqrt(q.pow(2).sum(-1, keepdim=True) / q_count + norm_eps) * q_norm
+    k = k / torch.sqrt(k.pow(2).sum(-1, keepdim=True) / k_count + norm_eps) * k_norm
+    compact = torch.cat([q, k, v], dim=1)
+    wide_k, wide_v = k_pool.float(), v_pool.float()         # (copies, or the pools themselves in 32-bit)
+    rope_kv_write(compact, positions, seq_of_token, block_table, wide_k, wide_v, inv_freq, heads, kv_heads, head_dim,
+                  rotary_dim, store=store, v_head_dim=vd, cos_sin_scale=cos_sin_scale)
+    if dtype != torch.float32:
+        k_pool.copy_(wide_k); v_pool.copy_(wide_v)
+    qkv[:, :qw] = compact[:, :qw].to(dtype)
 
 
 def head_norm_rope_kv_write(qkv, positions, seq_of_token, block_table, k_pool, v_pool, inv_freq, heads, kv_heads,
@@ -401,14 +445,91 @@ def sum_norms(x, delta, weights, eps, outs, rows=None, write_stream=False):
         out.copy_((_norm(v, eps, centre=False) * w).to(out.dtype))
 
 
+def output_norm(x, delta, out=None, weight=None, eps=0.0, rows=None, write_stream=True):
+    total = torch.zeros_like(x)
+    for term in delta.value.terms:
+        v = term.value.float()
+        if term.norm_weight is not None:
+            v = _norm(v, term.norm_eps, centre=False) * term.norm_weight
+        v = v * term.factor
+        total = total + (v if term.row_factor is None else v * term.row_factor[:, None])
+    routed = delta.value.routed
+    if routed is not None:
+        each = routed.value.float()
+        if routed.place is not None:
+            at = routed.place.long()
+            each = torch.where((at >= 0)[:, None], each[at.clamp(min=0)], torch.zeros(()))
+        total = total + each.view(x.shape[0], routed.top, -1).sum(1)
+    v = x + _norm(total, delta.eps, centre=False) * delta.weight
+    if write_stream:
+        x.copy_(v)
+    if rows is not None:
+        v = v[rows.long()]
+    if out is not None:
+        out.copy_((v if weight is None else _norm(v, eps, centre=False) * weight).to(out.dtype))
+    return x
+
+
+def state_space(conved, dt, dt_bias, a_log, state, query_start_loc, state_slots, num_seqs, heads, groups, dim, vdim, out,
+                max_query_len=0):
+    """state: [slots, heads, vdim, dim], the transpose of S [dim, vdim] per head."""
+    qsl, slots = query_start_loc.tolist(), state_slots.tolist()
+    T = conved.shape[0]
+    x, b, c = torch.split(conved.float(), [heads * vdim, groups * dim, groups * dim], dim=1)
+    per = heads // groups
+    x = x.reshape(T, heads, vdim)
+    b, c = (v.reshape(T, groups, dim).repeat_interleave(per, dim=1) for v in (b, c))
+    d = torch.nn.functional.softplus(dt.float() + dt_bias)
+    for s in range(num_seqs):
+        for t in range(qsl[s], qsl[s + 1]):
+            S = state[slots[s]]
+            S.mul_(torch.exp(-torch.exp(a_log) * d[t])[:, None, None])
+            S.add_((d[t][:, None] * x[t])[:, :, None] * b[t][:, None, :])
+            out[t] = torch.einsum("hvd,hd->hv", S, c[t]).reshape(-1)
+    return out
+
+
+def wkv_memory(r, k, v, gate, low, w2, w2t, w0, bonus, state, query_start_loc, state_slots, num_seqs, heads, dim, norm_weight,
+               eps, out, max_query_len=0):
+    """state: [slots, heads, dim, dim], the transpose of S per head."""
+    qsl, slots = query_start_loc.tolist(), state_slots.tolist()
+    R, K, V = (x.float().unflatten(1, (heads, dim)) for x in (r, k, v))
+    w = torch.exp(-torch.exp(torch.tanh(low.float()) @ w2.float().t() + w0)).unflatten(1, (heads, dim))
+    u = bonus.view(heads, dim)
+    g = gate.float()
+    g = g / (1.0 + torch.exp(-g))
+    for s in range(num_seqs):
+        for t in range(qsl[s], qsl[s + 1]):
+            S = state[slots[s]]
+            o = torch.einsum("hvd,hd->hv", S, R[t]) + (R[t] * u * K[t]).sum(-1, keepdim=True) * V[t]
+            S.mul_(w[t][:, None, :])
+            S.add_(V[t][:, :, None] * K[t][:, None, :])
+            out[t] = (_norm(o, eps, centre=False).reshape(-1) * norm_weight * g[t]).to(out.dtype)
+    return out
+
+
+def token_shift_step(x, mu, before, seq_of_token, query_start_loc, state_slots, num_seqs, out, single_tokens=False):
+    qsl, slots = query_start_loc.tolist(), state_slots.tolist()
+    out.zero_()
+    for s in range(num_seqs):
+        a, b = qsl[s], qsl[s + 1]
+        if b <= a:
+            continue
+        now = x[a:b].float()
+        last = torch.cat([before[slots[s]].float(), now[:-1]])
+        out[:, a:b] = (now + (last - now) * mu[:, None, :]).to(out.dtype)
+        before[slots[s], 0] = x[b - 1]
+    return out
+
+
 def short_conv_step(x, taps, tail, seq_of_token, query_start_loc, state_slots, num_seqs, out, activation="silu",
-                    single_tokens=False):
-    short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation)
+                    single_tokens=False, bias=None):
+    short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation, bias=bias)
     short_conv_update(x, tail, query_start_loc, state_slots, num_seqs)
     return out
 
 
-def short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation="silu", move_tail=False):
+def short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, activation="silu", move_tail=False, bias=None):
     K = taps.shape[0]                  # taps: [K, channels]
     qsl, slots = query_start_loc.tolist(), state_slots.tolist()
     out.zero_()
@@ -417,7 +538,7 @@ def short_conv(x, taps, tail, seq_of_token, query_start_loc, state_slots, out, a
         if b <= a:
             continue
         padded = torch.cat([tail[slots[s]].float(), x[a:b].float()])
-        acc = torch.zeros(b - a, x.shape[1], device=x.device)
+        acc = torch.zeros(b - a, x.shape[1], device=x.device) + (bias if bias is not None else 0.0)
         for j in range(K):
             acc = acc + padded[j:j + b - a] * taps[j].float()
         out[a:b] = (acc / (1.0 + torch.exp(-acc)) if activation == "silu" else acc).to(out.dtype)
@@ -656,11 +777,13 @@ def moe_route(logits, top, groups, keep, renormalise, ids, weights, scores="soft
 
 
 def moe_router(x, weight, top, groups, keep, renormalise, ids, weights, scores="softmax", correction=None, rank_by=1,
-               floor=0.0, gated=False, gate=None):
+               floor=0.0, gated=False, gate=None, identity=None, identity_experts=0):
     logits = x.float() @ weight.float().t()
     experts = logits.shape[1] - int(gated)
     moe_route(logits[:, :experts], top, groups, keep, renormalise, ids[:, :top], weights[:, :top], scores, correction,
               rank_by, floor)
+    if identity is not None:
+        identity.copy_((weights[:, :top] * (ids[:, :top] >= experts - identity_experts)).sum(-1))
     if gated:
         g = torch.sigmoid(logits[:, experts])
         if gate is not None:
@@ -681,7 +804,7 @@ class _Plan:
         self.place = torch.argsort(self.order)
 
 
-def moe_sort(ids, experts, tile_rows, with_place=False):
+def moe_sort(ids, experts, tile_rows, with_place=False, in_pairs=False):
     return _Plan(ids, experts)
 
 
@@ -698,21 +821,26 @@ def moe_experts(x, gate_up, down, ids, weights, activation, limit, alpha, eights
     return moe_combine(rows.value, out, rows.top)
 
 
-def moe_expert_rows(x, gate_up, down, ids, weights, activation, limit, alpha, eights):
+def moe_expert_rows(x, gate_up, down, ids, weights, activation, limit, alpha, eights, partial=False):
     from liteinfer_b200.ops import RoutedRows
 
     tokens, top = ids.shape
     plan = moe_sort(ids, gate_up.shape[0], 32)
     act = torch.empty(tokens * top, down.shape[2], dtype=x.dtype, device=x.device)
     each = torch.empty(tokens * top, down.shape[1], dtype=x.dtype, device=x.device)
-    moe_grouped("gate_up", x, gate_up, act, plan, top, activation, limit, alpha, eights=eights)
+    moe_grouped("up" if activation == "relu_squared" else "gate_up", x, gate_up, act, plan, top, activation, limit, alpha,
+                eights=eights)
     moe_grouped("down", act, down, each, plan, top, pair_weights=weights.view(-1))
-    return RoutedRows(each, top)
+    place = torch.arange(tokens * top, dtype=torch.int32)
+    return RoutedRows(each, top, torch.where(plan.ids < plan.experts, place, -1).to(torch.int32) if partial else None)
 
 
 def moe_grouped(mode, a, weight, out, plan, top, activation="swiglu", limit=0.0, alpha=1.0, pair_weights=None,
                 eights=False):
     for pair, e in enumerate(plan.ids.tolist()):
+        if e >= plan.experts:
+            out[pair] = float("nan")        # no expert: nobody reads this row
+            continue
         w = weight[e].float()
         if mode == "gate_up":
             x = a[pair // top].float()
@@ -723,6 +851,8 @@ def moe_grouped(mode, a, weight, out, plan, top, activation="swiglu", limit=0.0,
                 y = g * torch.sigmoid(alpha * g) * (u + 1.0)
             else:
                 y = g * torch.sigmoid(g) * u
+        elif mode == "up":
+            y = torch.relu(w @ a[pair // top].float()) ** 2
         else:
             y = (w @ a[pair].float()) * (1.0 if pair_weights is None else pair_weights[pair])
         out[pair] = y.to(out.dtype)
@@ -739,7 +869,7 @@ def fused_decode_supports(*args) -> bool:
     return False      # the stand-ins rotate and store in `rope_kv_write`, never inside the attention
 
 
-ALL = ("hgrn2", "sum_norms", "moe_expert_rows", "moe_router", "moe_experts", "moe_route", "moe_tile_rows", "moe_sort", "moe_grouped", "moe_combine", "sigmoid_gate_", "softcap_",
+ALL = ("gated_group_norm", "output_norm", "projection_norm_rope_kv_write", "state_space", "token_shift_step", "wkv_memory", "hgrn2", "sum_norms", "moe_expert_rows", "moe_router", "moe_experts", "moe_route", "moe_tile_rows", "moe_sort", "moe_grouped", "moe_combine", "sigmoid_gate_", "softcap_",
        "head_norm_rope_kv_write", "sigmoid_gate_heads_", "mlstm", "embedding_streams", "stream_rmsnorm", "activation", "batched_linear", "latent_prep", "latent_attention",
        "gate_heads", "convert", "layernorm", "layernorm_add", "projection_rmsnorm_", "qk_projection_rmsnorm_", "gated_rmsnorm",
        "short_conv", "short_conv_step", "short_conv_update", "gated_delta_rule", "fused_decode_supports", "scatter_tokens", "embedding", "rmsnorm", "add_", "add_bias_", "act_mul", "act_mul_interleaved", "gated_linear_supported",
