@@ -19,6 +19,8 @@ decoder beside the Llama decoder at equal layer sizes, and the Kegizen kernels o
 the same sizes, its closest relative, and its kernels beside their like.
 `--compare lulisun` sets the Lulisun decoder (chunked attention and an HGRN2 memory side by side, experts in parallel)
 beside a Kutolix decoder of the same sizes.
+`--compare sogazen` sets the Sogazen decoder (attention and a Mamba-2 state space side by side, RWKV-style time mixers, experts
+without gates and identity experts) beside a Lulisun decoder of the same sizes, and its kernels beside their like.
 `--compare kutolix` sets the Kutolix decoder (windowed gated attention with a sink, windowed latent attention, dense
 and routed feed-forwards) beside a Gifudra decoder of the same sizes, and its kernels beside their like.
 """
@@ -380,6 +382,25 @@ def _lulisun_config(width: int, ff: int, layers: int, heads: int, kv_heads: int,
              "mlp": {"kind": "moe", "expert": {"ff": ff // 4}, "shared": {"ff": ff // 4},
                      "router": {"experts": 32, "top": 3, "groups": {"count": 8, "keep": 4}}}}
     return {"architecture": "Lulisun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": [layer] * layers}
+
+
+def _sogazen_config(width: int, ff: int, layers: int, heads: int, kv_heads: int, head_dim: int, vocab: int) -> dict:
+    """Three layers with two mixers side by side, then one with a time mixer, over and over: the attention with the heads of
+    the Lulisun attention (all of each head rotated, capped scores), a state space with as large a state as the Lulisun
+    memory (heads of 64 x 128), a time mixer with heads of 64 x 64 as wide as the model.  The first of four layers has a dense
+    feed-forward; the others 32 experts with as many weights as a Lulisun expert (two matrices instead of three), of which,
+    and of eight identity experts, each token runs four."""
+    h = heads * head_dim // 128
+    moe = {"kind": "moe", "expert": {"ff": ff * 3 // 8}, "router": {"experts": 32, "identity": 8, "top": 4}}
+    pair = {"left": {"heads": h, "kv_heads": max(1, h // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 50.0,
+                     "rot": {"dims": 128, "base": 100000.0}},
+            "right": {"heads": width // 64, "vdim": 64, "state": 128, "groups": 2, "conv": 4, "norm_groups": 2}}
+    time_mixer = {"heads": width // 64, "dim": 64, "decay_rank": 64}
+    order = [{"type": "parallel", "mixer": pair, "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}},
+             {"type": "parallel", "mixer": pair, "mlp": moe}, {"type": "wkv", "mixer": time_mixer, "mlp": moe},
+             {"type": "parallel", "mixer": pair, "mlp": moe}]
+    return {"architecture": "Sogazen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "logit_softcap": 30.0,
+            "layers": [order[i % 4] for i in range(layers)]}
 
 
 def _timed(fn, repeats: int = 20, warmup: int = 5, inner: int = 1) -> float:
@@ -999,6 +1020,197 @@ def _lulisun_kernels(peaks: dict) -> dict:
     return {k: round(v, 4) for k, v in out.items()}
 
 
+def _sogazen_kernels(peaks: dict) -> dict:
+    """Each kernel that the Sogazen design brought or changed, alone beside its like, as fractions of the measured copy
+    bandwidth (kernels that stream) or product throughput (products, attention over prompts); inputs larger than L2 where a
+    kernel streams."""
+    import torch
+
+    from liteinfer_b200 import ops
+    from liteinfer_b200.parts.context import AttentionPlan
+
+    dev, bf = "cuda:0", torch.bfloat16
+    hbm, tflops = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops_burst"] * 1e12
+    out: dict = {}
+
+    def ints(v):
+        return torch.tensor(v, dtype=torch.int32, device=dev)
+
+    def rand(*shape, dtype=bf):
+        return torch.randn(*shape, device=dev).to(dtype)
+
+    def in_graph(fn, inner: int = 10) -> float:
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(inner):
+                fn()
+        return _timed(graph.replay, repeats=10, warmup=2) / inner
+
+    # -- attention (16 / 4 heads of 128), every earlier key visible: capped scores and a fixed sink beside neither
+    H, kv_heads, page, n, hd = 16, 4, 16, 2048, 128
+    pages = n // page
+    k_pool, v_pool = rand(pages * 64, kv_heads, page, hd), rand(pages * 64, kv_heads, page, hd)
+    for name, extra in (("attention", dict(softcap=50.0, sink=torch.zeros(H, device=dev))), ("lulisun_attention", {})):
+        table = torch.arange(pages, dtype=torch.int32, device=dev).view(1, pages)
+        q, o = rand(n, H * hd), torch.empty(n, H * hd, dtype=bf, device=dev)
+        plan = AttentionPlan(num_prefill=1, prefill_seqs=ints([0]), max_prefill_query_len=n)
+        args = (q, q.shape[1], o, k_pool, v_pool, table, ints([0, n]), ints([n]), 1, n, H, kv_heads, hd, hd ** -0.5)
+        ms = _timed(lambda: ops.paged_attention(*args, plan=plan, **extra))
+        out[f"{name}_prompt_us"] = ms * 1e3
+        out[f"{name}_prompt_tflops_frac"] = 4 * H * hd * n * (n + 1) / 2 / (ms * 1e-3) / tflops
+        for B in (64, 8):
+            table = torch.arange(B * pages, dtype=torch.int32, device=dev).view(B, pages)
+            plan = AttentionPlan(num_decode=B, decode_seqs=ints(list(range(B))), decode_tokens=ints(list(range(B))),
+                                 max_decode_context_len=n)
+            q, o = rand(B, H * hd), torch.empty(B, H * hd, dtype=bf, device=dev)
+            args = (q, q.shape[1], o, k_pool, v_pool, table, ints(list(range(B + 1))), ints([n] * B), B, 1, H, kv_heads, hd,
+                    hd ** -0.5)
+            ms = in_graph(lambda: ops.paged_attention(*args, plan=plan, **extra))
+            out[f"{name}_decode_b{B}_us"] = ms * 1e3
+            out[f"{name}_decode_b{B}_hbm_frac"] = B * n * kv_heads * hd * 2 * 2 / (ms * 1e-3) / hbm
+
+    # -- in front of it: biases, norms over the projection, rotation and cache write, beside the per-head form without norms
+    inv_freq = (10000.0 ** (-torch.arange(hd // 2, device=dev) * 2 / hd)).float()
+    T = 16384
+    big_k, big_v = rand(T // page, kv_heads, page, hd), rand(T // page, kv_heads, page, hd)
+    table = torch.arange(T // page, dtype=torch.int32, device=dev).view(1, -1)
+    pos, seq_of = torch.arange(T, dtype=torch.int32, device=dev), torch.zeros(T, dtype=torch.int32, device=dev)
+    qk, ones = (H + kv_heads) * hd, torch.ones(H * hd, device=dev)
+    row, bias = rand(T, qk + kv_heads * hd), torch.zeros(qk, device=dev)
+    for rows, key in ((T, "16384"), (64, "b64"), (8, "b8")):
+        timer = _timed if rows > 64 else in_graph
+        ms = timer(lambda: ops.projection_norm_rope_kv_write(
+            row[:rows], pos[:rows], seq_of[:rows], table, big_k, big_v, inv_freq, H, kv_heads, hd, hd, ones,
+            ones[:kv_heads * hd], H * hd, kv_heads * hd, 1e-5, bias=bias, values_are_keys=True))
+        out[f"projection_norm_rope_{key}_us"] = ms * 1e3
+        out[f"projection_norm_rope_{key}_hbm_frac"] = rows * (2 * H + 3 * kv_heads) * hd * 2 / (ms * 1e-3) / hbm
+        ms = timer(lambda: ops.head_norm_rope_kv_write(row[:rows], pos[:rows], seq_of[:rows], table, big_k, big_v, inv_freq, H,
+                                                       kv_heads, hd, hd, None, None, 1e-5))
+        out[f"lulisun_rope_{key}_us"] = ms * 1e3
+        out[f"lulisun_rope_{key}_hbm_frac"] = rows * (2 * H + 4 * kv_heads) * hd * 2 / (ms * 1e-3) / hbm
+    del big_k, big_v, row
+
+    # -- the memories beside the HGRN2 memory (16 heads of 128 x 128), each with the norm (and gate) behind it: the state space
+    #    (32 heads of 64 x 128 in two groups, its convolution too), time mixing (32 heads of 64 x 64, decays of rank 64)
+    W = 2048
+    for batch, each, key in ((64, 1, "decode_b64"), (8, 1, "decode_b8"), (1, 2048, "prompt_2048"), (8, 2048, "prompts_8x2048")):
+        m = batch * each
+        at = (ints([i * each for i in range(batch + 1)]), ints(list(range(batch))), batch)
+        seqs = torch.arange(batch, dtype=torch.int32, device=dev).repeat_interleave(each)
+        heads, vdim, dim, groups = 32, 64, 128, 2
+        proj = rand(m, 2 * W + 2 * groups * dim + heads)
+        channels = W + 2 * groups * dim
+        taps, tail = rand(4, channels), torch.zeros(batch, 3, channels, dtype=bf, device=dev)
+        conved, conv_bias = torch.empty(m, channels, dtype=bf, device=dev), torch.zeros(channels, device=dev)
+        per_head, read, gated = torch.zeros(heads, device=dev), torch.empty(m, W, device=dev), torch.empty(m, W, dtype=bf, device=dev)
+        space, weight = torch.zeros(batch, heads, vdim, dim, device=dev), torch.ones(W, device=dev)
+
+        def convolve():
+            ops.short_conv_step(proj[:, W:W + channels], taps, tail, seqs, *at[:2], batch, conved, single_tokens=each == 1,
+                                bias=conv_bias)
+
+        def space_step():
+            ops.state_space(conved, proj[:, W + channels:], per_head, per_head, space, *at, heads, groups, dim, vdim, read, each)
+            ops.gated_group_norm(read, proj[:, :W], weight, 1e-5, gated, 2, add=conved[:, :W], skip=per_head)
+
+        r, k, v, g = rand(4, m, W)
+        low, w2 = rand(m, 64), rand(W, 64)
+        w2t, w0, memory = w2.t().contiguous(), torch.full((W,), -3.0, device=dev), torch.zeros(batch, 32, 64, 64, device=dev)
+
+        def time_step():
+            ops.wkv_memory(r, k, v, g, low, w2, w2t, w0, w0, memory, *at, 32, 64, weight, 1e-5, gated, each)
+
+        p3, s3 = rand(m, 3 * W), torch.zeros(batch, 16, 128, 128, device=dev)
+        lower = torch.full((W,), 0.5, device=dev)
+
+        def hgrn2():
+            ops.hgrn2(p3, (0, W, 2 * W), torch.zeros_like(lower), lower, s3, *at, 16, 128, 128, weight[:128], 1e-5, gated, each)
+
+        timer = in_graph if each == 1 else _timed
+        ms = timer(convolve)
+        out[f"short_conv_step_{key}_us"] = ms * 1e3
+        if m > 8192:
+            out[f"short_conv_step_{key}_hbm_frac"] = m * channels * 4 / (ms * 1e-3) / hbm
+        for name, run, state in (("state_space", space_step, space), ("time_mixing", time_step, memory), ("lulisun_hgrn2", hgrn2, s3)):
+            ms = timer(run)
+            out[f"{name}_{key}_us"] = ms * 1e3
+            entries = state[0].numel()
+            if each == 1:
+                out[f"{name}_{key}_hbm_frac"] = batch * entries * 4 * 2 / (ms * 1e-3) / hbm
+            else:       # three multiply-adds an entry and token, against 75 TFLOP/s of FFMA
+                out[f"{name}_{key}_ffma_frac"] = m * entries * 6 / (ms * 1e-3) / 75e12
+        # the token shift and the four products behind it, beside one product of the same size against one input
+        x, mu, last = rand(m, W), torch.rand(5, W, device=dev), torch.zeros(batch, 1, W, dtype=bf, device=dev)
+        mixed, weights4, four = torch.empty(5, m, W, dtype=bf, device=dev), rand(4, W, W), torch.empty(4, m, W, dtype=bf, device=dev)
+        ms = timer(lambda: ops.token_shift_step(x, mu, last, seqs, *at, mixed, single_tokens=each == 1))
+        out[f"token_shift_{key}_us"] = ms * 1e3
+        if m > 8192:
+            out[f"token_shift_{key}_hbm_frac"] = m * W * 6 * 2 / (ms * 1e-3) / hbm
+        joined, wide = weights4.view(4 * W, W), torch.empty(m, 4 * W, dtype=bf, device=dev)
+        for name, run in (("shifted_products", lambda: ops.batched_linear(mixed[:4], weights4, four)),
+                          ("one_product", lambda: ops.linear(x, joined, wide))):
+            ms = timer(run)
+            out[f"{name}_{key}_us"] = ms * 1e3
+            if m >= 2048:
+                out[f"{name}_{key}_tflops_frac"] = 2 * m * 4 * W * W / (ms * 1e-3) / tflops
+
+    # -- what a sublayer gives back on its way into the stream: two normed mixers, four experts' rows and an identity, beside
+    #    the sum and two norms of the Lulisun layer
+    top = 4
+    for T, key in ((8192, "8192"), (64, "b64"), (8, "b8")):
+        x, a, b = torch.randn(T, W, device=dev), rand(T, W), rand(T, W)
+        rows, w32, share = rand(T * top, W), torch.ones(W, device=dev), torch.rand(T, device=dev)
+        place = torch.randperm(T * top, device=dev).to(torch.int32)
+        o1, o2 = torch.empty(T, W, dtype=bf, device=dev), torch.empty(T, W, dtype=bf, device=dev)
+        pair = ops.NormedDelta(ops.SumDelta((ops.SumTerm(a, 0.5, None, w32, 1e-5), ops.SumTerm(b, 0.5, None, w32, 1e-5))), w32, 1e-5, False)
+        experts = ops.NormedDelta(ops.SumDelta((ops.SumTerm(a, 1.0, share),), ops.RoutedRows(rows, top, place)), w32, 1e-5, False)
+        both = ops.SumDelta((ops.SumTerm(a, 0.8),), ops.RoutedRows(rows, top, place))
+        timer = _timed if T > 64 else in_graph
+        for name, run, nbytes in (("output_norm_pair", lambda: ops.output_norm(x, pair, o1), 8 + 4 + 2),
+                                  ("output_norm_experts", lambda: ops.output_norm(x, experts, o1), 8 + 2 + 2 * top + 2),
+                                  ("lulisun_sum_norms", lambda: ops.sum_norms(x, both, (w32, w32), 1e-5, (o1, o2), write_stream=True),
+                                   8 + 2 + 2 * top + 4)):
+            ms = timer(run)
+            out[f"{name}_{key}_us"] = ms * 1e3
+            if T > 64:
+                out[f"{name}_{key}_hbm_frac"] = T * W * nbytes / (ms * 1e-3) / hbm
+
+    # -- router and experts: four of 32 without gates and eight identity experts (router only, and all pairs with experts),
+    #    beside Lulisun's three and the shared one; the capped gated product beside the silu one
+    F, FU, E = 2048, 3072, 32
+    gate_up, down = (rand(E + 1, 2 * F, W) * 0.02).to(bf), (rand(E + 1, W, F) * 0.02).to(bf)
+    up, down_u = (rand(E, FU, W) * 0.02).to(bf), (rand(E, W, FU) * 0.02).to(bf)
+    router, shared, correction = torch.randn(E + 8, W, device=dev) * 0.02, torch.randn(E + 1, W, device=dev) * 0.02, torch.zeros(E + 8, device=dev)
+    wide, caps = (rand(2 * 8192, W) * 0.02).to(bf), dict(limit=7.0, alpha=1.702)
+    for tokens, key in ((2048, "prompt_2048"), (64, "decode_b64"), (8, "decode_b8")):
+        x = rand(tokens, W)
+        timer = _timed if tokens > 64 else in_graph
+        ids, weights, same = torch.empty(tokens, top, dtype=torch.int32, device=dev), torch.empty(tokens, top, device=dev), torch.empty(tokens, device=dev)
+        forms = (("sogazen", lambda: ops.moe_router(x, router, top, 1, 1, False, ids, weights, correction=correction, identity=same,
+                                                    identity_experts=8),
+                  lambda: ops.moe_expert_rows(x, up, down_u, ids, weights, "relu_squared", 0.0, 1.0, False, partial=True)),
+                 ("lulisun", lambda: ops.moe_router(x, shared, 3, 8, 4, True, ids, weights, scores="sigmoid",
+                                                    correction=correction[:E], rank_by=2, floor=1e-20, gated=True),
+                  lambda: ops.moe_expert_rows(x, gate_up, down, ids, weights, "swiglu", 0.0, 1.0, True)))
+        for name, route, run in forms:
+            out[f"{name}_router_{key}_us"] = timer(route) * 1e3
+            ms = timer(run)
+            out[f"{name}_experts_{key}_us"] = ms * 1e3
+            live = ids[ids < (E if name == "sogazen" else E + 1)]
+            if tokens > 64:
+                out[f"{name}_experts_{key}_tflops_frac"] = 2 * live.numel() * 3 * F * W / (ms * 1e-3) / tflops
+            else:
+                out[f"{name}_experts_{key}_hbm_frac"] = int(torch.unique(live).numel()) * 3 * F * W * 2 / (ms * 1e-3) / hbm
+        if tokens != 64:
+            h = torch.empty(tokens, 8192, dtype=bf, device=dev)
+            for name, activation, options in (("capped", "capped_swiglu", caps), ("silu", "silu", {})):
+                ms = timer(lambda: ops.gated_linear(x, wide, h, activation, **options))
+                out[f"{name}_gated_product_{key}_us"] = ms * 1e3
+    return {k: round(v, 4) for k, v in out.items()}
+
+
 def run_kegizen(args, which: str = "kegizen") -> dict:
     """Prefill (one prompt of 2,048 tokens) and decode (batch 8 and 64 near a context of 2,048) of a Kegizen (or
     Gifudra) model and of a Llama model with the same width, depth, head sizes and feed-forward, random weights,
@@ -1019,11 +1231,11 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
     if which == "gifudra":      # heads of 128 in both sizes: the latent attention's heads are 128 + 64 wide
         sizes = {"w2048": dict(width=2048, ff=8192, layers=8, heads=16, kv_heads=4, head_dim=128),
                  "w4096": dict(width=4096, ff=14336, layers=4, heads=32, kv_heads=8, head_dim=128)}
-    if which in ("kutolix", "lulisun"):
+    if which in ("kutolix", "lulisun", "sogazen"):
         sizes = {"w2048": dict(width=2048, ff=8192, layers=8, heads=16, kv_heads=4, head_dim=128),
                  "w4096": dict(width=4096, ff=14336, layers=4, heads=32, kv_heads=8, head_dim=128)}
     design = {"gifudra": _gifudra_config, "karupel": _karupel_config, "kutolix": _kutolix_config,
-              "lulisun": _lulisun_config}.get(which, _kegizen_config)
+              "lulisun": _lulisun_config, "sogazen": _sogazen_config}.get(which, _kegizen_config)
     result: dict = {"impl": "ours", "compare": which, "dtype": "bf16", "data": "synthetic ids, random weights",
                     "peaks": peaks, "models": {}}
     for name, size in sizes.items():
@@ -1037,6 +1249,8 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
             beside = ("gifudra", _gifudra_config(vocab=vocab, **size))
         if which == "lulisun":      # its closest relative: windowed attention, experts in every other layer
             beside = ("kutolix", _kutolix_config(vocab=vocab, **size))
+        if which == "sogazen":      # its closest relative: attention and a memory side by side, experts in every layer
+            beside = ("lulisun", _lulisun_config(vocab=vocab, **size))
         for arch, cfg in ((which, design(vocab=vocab, **size)), beside):
             with tempfile.TemporaryDirectory() as tmp:
                 model_dir = write_random_model(cfg, Path(tmp) / arch, seed=0)
@@ -1065,7 +1279,7 @@ def run_kegizen(args, which: str = "kegizen") -> dict:
                 llm.close()
                 result["models"][f"{name}_{arch}"] = numbers
     kernels = {"gifudra": _gifudra_kernels, "karupel": _karupel_kernels, "kutolix": _kutolix_kernels,
-               "lulisun": _lulisun_kernels}.get(which, _kegizen_kernels)
+               "lulisun": _lulisun_kernels, "sogazen": _sogazen_kernels}.get(which, _kegizen_kernels)
     result["kernels"] = kernels(peaks)
     return result
 
@@ -1207,7 +1421,7 @@ def main() -> int:
     parser.add_argument("--workload", default="none", choices=["none", "3b", "8b", "all"],
                         help="run the reference's larger configurations instead (64 requests under continuous batching "
                              "at the 3B sizes; decode at a context of 8,192 at the 8B sizes) and print their line")
-    parser.add_argument("--compare", default="none", choices=["none", "kegizen", "gifudra", "karupel", "kutolix", "lulisun"],
+    parser.add_argument("--compare", default="none", choices=["none", "kegizen", "gifudra", "karupel", "kutolix", "lulisun", "sogazen"],
                         help="instead of the default run: the Kegizen (or Gifudra) decoder beside the Llama decoder, "
                              "the Karupel decoder beside the Kegizen decoder, or the Kutolix decoder beside the Gifudra "
                              "decoder, at equal layer sizes (prefill, decode, and the design's kernels one by one)")

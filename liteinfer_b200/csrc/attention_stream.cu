@@ -142,7 +142,8 @@ __device__ __noinline__ void merge_in_cluster(const AttnParams& p, const float* 
 }
 
 // kRing: slots per warp; up to kRing - 1 groups are on their way while one is multiplied.
-template <int D, int kRing, bool kCluster>
+// kCapped: scores are capped (p.cap_in, p.cap_out); a form of its own, so that the plain one stays what it was.
+template <int D, int kRing, bool kCluster, bool kCapped = false>
 __global__ void __launch_bounds__(kWarps * 32, D == 64 ? 5 : 2)   // blocks per SM that the rings leave room for
 attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                         const AttnParams p) {
@@ -354,6 +355,12 @@ attention_stream_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         // Scale and mask (only a group at the end of the context or at the window's start needs the mask; values
         // of keys that are not visible become zero there, since an unwritten slot of a page may hold anything).
         float group_max[2] = {-INFINITY, -INFINITY};
+        if constexpr (kCapped) {
+#pragma unroll
+          for (int half = 0; half < 2; ++half)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s[half][j] = p.cap_out * fast_tanh(s[half][j] * p.cap_in);   // scaled below like any score
+        }
         if (kpos0 >= lo && kpos0 + kGroupKeys <= hi) {
 #pragma unroll
           for (int half = 0; half < 2; ++half)
@@ -512,6 +519,17 @@ int launch_stream(const CUtensorMap& mk, const CUtensorMap& mv, const AttnParams
     configured = true;
   }
   const dim3 grid(p.num_splits, p.kv_heads * p.v_parts, num_seqs);
+  if (p.cap_out > 0.f) {
+    static bool ready = false;
+    if (!ready) {
+      cudaError_t e = cudaFuncSetAttribute(attention_stream_kernel<D, kRing, false, true>,
+                                           cudaFuncAttributeMaxDynamicSharedMemorySize, (int)stream_smem<D, kRing>());
+      if (e != cudaSuccess) return (int)e;
+      ready = true;
+    }
+    return (int)launch_pdl(num_seqs, attention_stream_kernel<D, kRing, false, true>, grid, dim3(kWarps * 32),
+                           stream_smem<D, kRing>(), stream, mk, mv, p);
+  }
   if (!p.cluster_merge)
     return (int)launch_pdl(num_seqs, attention_stream_kernel<D, kRing, false>, grid, dim3(kWarps * 32), stream_smem<D, kRing>(), stream, mk, mv, p);
   cudaLaunchConfig_t config = {};
@@ -607,7 +625,7 @@ LI_EXPORT int li_paged_attention_stream_capacity(int head_dim) {
 // says how many counters a split launch needs); sizes as li_paged_attention_stream_supports allows.
 // error_flag (device int, zero; may be null): set to 21 if a wait for a group of keys ever gave up.
 // sink (optional, [heads] float32): exp(sink[h]) is one more term of head h's denominator.  v_dim: the size of a value,
-// a multiple of head_dim.
+// a multiple of head_dim.  softcap > 0: a scaled score s becomes softcap * tanh(s / softcap).
 LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* out, int out_row_stride,
                                         const void* k_pool, const void* v_pool, const int* block_table,
                                         int table_stride, const int* query_start_loc, const int* context_lens,
@@ -615,7 +633,7 @@ LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* o
                                         int page_size, int num_pages, float scale, int window, int num_splits,
                                         float* partial_out, float* partial_lse, unsigned* counters,
                                         const float* rope_inv_freq, const void* k_new, const void* v_new,
-                                        int store_new, int* error_flag, const float* sink, int v_dim,
+                                        int store_new, int* error_flag, const float* sink, int v_dim, float softcap,
                                         cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   if (!li_paged_attention_stream_supports(heads, kv_heads, head_dim, page_size)) return LI_ERR_UNSUPPORTED;
@@ -644,7 +662,11 @@ LI_EXPORT int li_paged_attention_stream(const void* q, int q_row_stride, void* o
   const char* cluster_env = getenv("LITEINFER_ATTN_CLUSTER_MERGE");
   p.v_parts = v_parts;
   p.sink = sink;      // added by the merges of attention_mma.cuh; the merge inside a cluster does not know it
-  if (cluster_env && atoi(cluster_env) == 1 && sink == nullptr && num_splits >= 2 && num_splits <= 16 &&
+  if (softcap > 0.f) {
+    p.cap_in = scale / softcap;
+    p.cap_out = softcap / scale;
+  }
+  if (cluster_env && atoi(cluster_env) == 1 && sink == nullptr && softcap <= 0.f && num_splits >= 2 && num_splits <= 16 &&
       li_paged_attention_stream_cluster_capacity(head_dim, num_splits) >= kv_heads * v_parts * num_seqs)
     p.cluster_merge = 1;
   if ((page_size & (page_size - 1)) == 0)

@@ -267,17 +267,17 @@ __global__ void gated_rmsnorm_kernel(const float* __restrict__ x, const T* __res
 }
 
 // The same with 16-byte accesses: a lane keeps NV groups of four of its head's row in registers between the sum
-// of squares and the scaling.  size a multiple of four and at most 128 NV; every row 16-byte (gate: 8-byte in
+// of squares and the scaling; LANES of a warp share a head.  size a multiple of four and at most 4 LANES NV; every row 16-byte (gate: 8-byte in
 // bfloat16) aligned.
-template <typename T, int NV>
+template <typename T, int NV, int LANES>
 __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* __restrict__ gate, size_t gate_stride,
                                          const float* __restrict__ weight, T* __restrict__ out, size_t out_stride, int tokens,
                                          int heads, int size, float eps, int weight_stride, int act,
                                          const float* __restrict__ den, const T* __restrict__ add, size_t add_stride,
                                          const float* __restrict__ add_scale) {
-  const int lane = threadIdx.x & 31;
-  const size_t item = (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);   // (token, head)
-  if (item >= (size_t)tokens * heads) return;
+  const int lane = threadIdx.x % LANES;
+  const size_t item = (size_t)blockIdx.x * (blockDim.x / LANES) + threadIdx.x / LANES;   // (token, head)
+  if (item >= (size_t)tokens * heads) return;            // (by all lanes of an item)
   const size_t t = item / heads;
   const int h = (int)(item - t * heads);
   const int quads = size >> 2;
@@ -285,7 +285,7 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
   float4 wv[NV];
 #pragma unroll
   for (int j = 0; j < NV; ++j)
-    if (lane + 32 * j < quads) wv[j] = *reinterpret_cast<const float4*>(w + 4 * (lane + 32 * j));
+    if (lane + LANES * j < quads) wv[j] = *reinterpret_cast<const float4*>(w + 4 * (lane + LANES * j));
   grid_dependency_wait();
   const float* xr = x + (t * heads + h) * size;
   const T* g = gate + t * gate_stride + (size_t)h * size;
@@ -294,9 +294,9 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
     v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (lane + 32 * j < quads) {
-      v[j] = *reinterpret_cast<const float4*>(xr + 4 * (lane + 32 * j));
-      if (act != 2) load4(g + 4 * (lane + 32 * j), z[j]);
+    if (lane + LANES * j < quads) {
+      v[j] = *reinterpret_cast<const float4*>(xr + 4 * (lane + LANES * j));
+      if (act != 2) load4(g + 4 * (lane + LANES * j), z[j]);
     }
   }
   if (den != nullptr) {
@@ -309,9 +309,9 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
     const T* ar = add + t * add_stride + (size_t)h * size;
 #pragma unroll
     for (int j = 0; j < NV; ++j)
-      if (lane + 32 * j < quads) {
+      if (lane + LANES * j < quads) {
         float a[4];
-        load4(ar + 4 * (lane + 32 * j), a);
+        load4(ar + 4 * (lane + LANES * j), a);
         v[j].x = fmaf(share, a[0], v[j].x);
         v[j].y = fmaf(share, a[1], v[j].y);
         v[j].z = fmaf(share, a[2], v[j].z);
@@ -321,11 +321,14 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
   float q = 0.f;
 #pragma unroll
   for (int j = 0; j < NV; ++j) q += v[j].x * v[j].x + v[j].y * v[j].y + v[j].z * v[j].z + v[j].w * v[j].w;
-  const float inv = 1.0f / sqrtf(warp_sum(q) / (float)size + eps);
+    const unsigned mine = LANES == 32 ? 0xffffffffu : ((1u << (LANES % 32)) - 1u) << (threadIdx.x & 31 & ~(LANES - 1));
+#pragma unroll
+  for (int o = LANES / 2; o > 0; o >>= 1) q += __shfl_xor_sync(mine, q, o);
+  const float inv = 1.0f / sqrtf(q / (float)size + eps);
   T* o = out + t * out_stride + (size_t)h * size;
 #pragma unroll
   for (int j = 0; j < NV; ++j) {
-    if (lane + 32 * j >= quads) continue;
+    if (lane + LANES * j >= quads) continue;
     const float xs[4] = {v[j].x, v[j].y, v[j].z, v[j].w}, ws[4] = {wv[j].x, wv[j].y, wv[j].z, wv[j].w};
     float r[4];
 #pragma unroll
@@ -337,7 +340,7 @@ __global__ void gated_rmsnorm_vec_kernel(const float* __restrict__ x, const T* _
       }
       r[e] = xs[e] * inv * ws[e] * by;
     }
-    store4(o + 4 * (lane + 32 * j), r);
+    store4(o + 4 * (lane + LANES * j), r);
   }
 }
 
@@ -524,8 +527,11 @@ LI_EXPORT int li_gated_rmsnorm(int dtype, const float* x, const void* gate, size
                     (uintptr_t)add % (4 * gate_unit) == 0 && add_stride % 4 == 0;
   if (wide) {
     const int nv = size <= 128 ? 1 : size <= 256 ? 2 : 4;
+    // Heads of up to 64: half a warp each, so that every lane has work.
+    const dim3 half_grid((unsigned)((items + 2 * warps - 1) / (2 * warps)));
 #define LI_GATED(T, NV)                                                                                                \
-  return (int)launch_pdl(tokens, gated_rmsnorm_vec_kernel<T, NV>, grid, dim3(warps * 32), 0, stream, x,               \
+  return (int)launch_pdl(tokens, size <= 64 ? gated_rmsnorm_vec_kernel<T, NV, 16> : gated_rmsnorm_vec_kernel<T, NV, 32>, \
+                         size <= 64 ? half_grid : grid, dim3(warps * 32), 0, stream, x,                              \
                          (const T*)gate, gate_stride, weight, (T*)out, out_stride, tokens, heads, size, eps, weight_stride, act, \
                          den, (const T*)add, add_stride, add_scale)
     if (dtype == kFloat32) {

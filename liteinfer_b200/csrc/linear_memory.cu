@@ -299,67 +299,107 @@ ssd_record_kernel(const T* __restrict__ conved, size_t conved_stride, const T* _
 
 // Time mixing.  r, k, v [tokens, heads * dim] (rows row_stride apart), low [tokens, rank] the decay's inner product
 // (before its tanh), w2t [rank, heads * dim] (transposed), w0, u [heads * dim].  A block: 16 tokens x a few heads.
-constexpr int kRecordTokens = 16;
-template <typename T>
-__global__ void __launch_bounds__(256)
+constexpr int kRecordTokens = 16, kRecordThreads = 128;
+template <typename T> __device__ __forceinline__ float2 two(const T* p);
+template <> __device__ __forceinline__ float2 two<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> __device__ __forceinline__ float2 two<bf16>(const bf16* p) {
+  const unsigned v = *reinterpret_cast<const unsigned*>(p);
+  return make_float2(__uint_as_float(v << 16), __uint_as_float(v & 0xffff0000u));
+}
+
+// kPairs: two neighbouring channels a thread and access (dim even, rows aligned for it), else one.
+template <typename T, bool kPairs>
+__global__ void __launch_bounds__(kRecordThreads)
 wkv_record_kernel(const T* __restrict__ r, const T* __restrict__ k, const T* __restrict__ v, size_t row_stride,
                   const T* __restrict__ low, size_t low_stride, int rank, const T* __restrict__ w2t,
                   const float* __restrict__ w0, const float* __restrict__ u, float* __restrict__ group_records,
                   float* __restrict__ head_records, float* __restrict__ bonus, int tokens, int heads, int heads_per_block,
                   int dim, int dimp, int vdimp) {
-  extern __shared__ float tanhs[];                       // [rank][kRecordTokens]
+  constexpr int C = kPairs ? 2 : 1;
+  extern __shared__ __align__(16) float tanhs[];         // [rank][kRecordTokens]
   grid_dependency_wait();
   const int t0 = blockIdx.x * kRecordTokens, n = min(kRecordTokens, tokens - t0);
   const int h0 = blockIdx.y * heads_per_block, h1 = min(heads, h0 + heads_per_block);
   const int width = heads * dim, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int i = threadIdx.x; i < rank * kRecordTokens; i += 256) {
+  for (int i = threadIdx.x; i < rank * kRecordTokens; i += kRecordThreads) {
     const int t = i / rank, c = i - t * rank;
     tanhs[c * kRecordTokens + t] = t < n ? tanhf(to_float(low[(size_t)(t0 + t) * low_stride + c])) : 0.f;
   }
   __syncthreads();
-  for (int c = h0 * dim + threadIdx.x; c < h1 * dim; c += 256) {
-    float acc[kRecordTokens];
-    const float base = w0[c];
+  for (int c = h0 * dim + threadIdx.x * C; c < h1 * dim; c += kRecordThreads * C) {
+    float acc[C][kRecordTokens];
 #pragma unroll
-    for (int t = 0; t < kRecordTokens; ++t) acc[t] = 0.f;
-#pragma unroll 4
+    for (int e = 0; e < C; ++e)
+#pragma unroll
+      for (int t = 0; t < kRecordTokens; ++t) acc[e][t] = 0.f;
+#pragma unroll 8
     for (int i = 0; i < rank; ++i) {
-      const float w = widen(w2t[(size_t)i * width + c]);
+      float w[2];
+      if constexpr (kPairs) {
+        const float2 p = two<T>(w2t + (size_t)i * width + c);
+        w[0] = p.x; w[1] = p.y;
+      } else {
+        w[0] = widen(w2t[(size_t)i * width + c]);
+      }
       const float4* th = reinterpret_cast<const float4*>(tanhs + i * kRecordTokens);
 #pragma unroll
       for (int t = 0; t < kRecordTokens / 4; ++t) {
         const float4 x = th[t];
-        acc[4 * t] = fmaf(w, x.x, acc[4 * t]);
-        acc[4 * t + 1] = fmaf(w, x.y, acc[4 * t + 1]);
-        acc[4 * t + 2] = fmaf(w, x.z, acc[4 * t + 2]);
-        acc[4 * t + 3] = fmaf(w, x.w, acc[4 * t + 3]);
+#pragma unroll
+        for (int e = 0; e < C; ++e) {
+          acc[e][4 * t] = fmaf(w[e], x.x, acc[e][4 * t]);
+          acc[e][4 * t + 1] = fmaf(w[e], x.y, acc[e][4 * t + 1]);
+          acc[e][4 * t + 2] = fmaf(w[e], x.z, acc[e][4 * t + 2]);
+          acc[e][4 * t + 3] = fmaf(w[e], x.w, acc[e][4 * t + 3]);
+        }
       }
     }
-    const int h = c / dim, d = c - h * dim;
+    const int h = c / dim, d = c - h * dim;              // (a pair lies within one head: dim is even)
+    float* out = group_records + ((size_t)t0 * heads + h) * 3 * dimp + 2 * dimp + d;
+    float base[2] = {w0[c], kPairs ? w0[c + C - 1] : 0.f};
 #pragma unroll
     for (int t = 0; t < kRecordTokens; ++t)
-      if (t < n) group_records[((size_t)(t0 + t) * heads + h) * 3 * dimp + 2 * dimp + d] = expf(-expf(acc[t] + base));
+      if (t < n) {
+        float* o = out + (size_t)t * heads * 3 * dimp;
+        if constexpr (kPairs)
+          *reinterpret_cast<float2*>(o) = make_float2(expf(-expf(acc[0][t] + base[0])), expf(-expf(acc[C - 1][t] + base[1])));
+        else
+          o[0] = expf(-expf(acc[0][t] + base[0]));
+      }
   }
   // r, k and v as floats, zeros in the places past dim, and the bonus r . (u k): a warp a (token, head).
-  for (int item = warp; item < n * (h1 - h0); item += 8) {
+#pragma unroll 4
+  for (int item = warp; item < n * (h1 - h0); item += kRecordThreads / 32) {
     const int t = item / (h1 - h0), h = h0 + item - t * (h1 - h0);
     const size_t row = (size_t)(t0 + t) * row_stride + (size_t)h * dim, rec = (size_t)(t0 + t) * heads + h;
     float* group_out = group_records + rec * 3 * dimp;
     float* head_out = head_records + rec * vdimp;
     float sum = 0.f;
-    for (int d = lane; d < dimp; d += 32) {
-      float rv = 0.f, kv = 0.f, vv = 0.f;
+    for (int d = lane * C; d < dimp; d += 32 * C) {
+      float rv[2] = {0.f, 0.f}, kv[2] = {0.f, 0.f}, vv[2] = {0.f, 0.f};
       if (d < dim) {
-        rv = widen(r[row + d]);
-        kv = widen(k[row + d]);
-        vv = widen(v[row + d]);
-        sum = fmaf(rv * u[h * dim + d], kv, sum);
-      } else {
-        group_out[2 * dimp + d] = 0.f;
+        if constexpr (kPairs) {
+          const float2 a = two<T>(r + row + d), b = two<T>(k + row + d), c = two<T>(v + row + d);
+          rv[0] = a.x; rv[1] = a.y; kv[0] = b.x; kv[1] = b.y; vv[0] = c.x; vv[1] = c.y;
+        } else {
+          rv[0] = widen(r[row + d]);
+          kv[0] = widen(k[row + d]);
+          vv[0] = widen(v[row + d]);
+        }
+#pragma unroll
+        for (int e = 0; e < C; ++e) sum = fmaf(rv[e] * u[h * dim + d + e], kv[e], sum);
       }
-      group_out[d] = rv;
-      group_out[dimp + d] = kv;
-      if (d < vdimp) head_out[d] = vv;
+      if constexpr (kPairs) {
+        *reinterpret_cast<float2*>(group_out + d) = make_float2(rv[0], rv[1]);
+        *reinterpret_cast<float2*>(group_out + dimp + d) = make_float2(kv[0], kv[1]);
+        if (d >= dim) *reinterpret_cast<float2*>(group_out + 2 * dimp + d) = make_float2(0.f, 0.f);
+        if (d < vdimp) *reinterpret_cast<float2*>(head_out + d) = make_float2(vv[0], vv[1]);
+      } else {
+        group_out[d] = rv[0];
+        group_out[dimp + d] = kv[0];
+        if (d >= dim) group_out[2 * dimp + d] = 0.f;
+        if (d < vdimp) head_out[d] = vv[0];
+      }
     }
     sum = warp_sum(sum);
     if (lane == 0) bonus[rec] = sum;
@@ -525,6 +565,23 @@ wkv_token_kernel(const T* __restrict__ r, const T* __restrict__ k, const T* __re
   float* th = os + dim;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, sub = lane & 15, group = warp * 2 + (lane >> 4);
   float* base = state + ((size_t)slot * heads + head) * (size_t)dim * dim;
+  // The decay's second product, a group of lanes a channel (channels group, group + 16, ...), four of the rank a lane: up to
+  // a rank of 64 its weights are on their way to registers before the wait.
+  constexpr bool kEarly = NPL <= 8;
+  const bool early = kEarly && rank <= 64 && rank % 4 == 0 && reinterpret_cast<uintptr_t>(w2) % (4 * sizeof(T)) == 0;
+  float wr[kEarly ? NPL : 1][4];
+  if (early) {
+#pragma unroll
+    for (int i = 0; i < (kEarly ? NPL : 1); ++i) {
+      const int d = i * kRowGroups + group;
+      wr[i][0] = wr[i][1] = wr[i][2] = wr[i][3] = 0.f;
+      if (d < dim && 4 * sub < rank) {
+        const T* p = w2 + ((size_t)head * dim + d) * rank + 4 * sub;
+        const float2 a = two<T>(p), b = two<T>(p + 2);
+        wr[i][0] = a.x; wr[i][1] = a.y; wr[i][2] = b.x; wr[i][3] = b.y;
+      }
+    }
+  }
   grid_dependency_wait();
   float4 s[kAhead][NPL / 4];
   first_columns<NPL>(base, dim, dim, s, sub, group);
@@ -544,15 +601,24 @@ wkv_token_kernel(const T* __restrict__ r, const T* __restrict__ k, const T* __re
     }
   }
   const float bonus = block_sum(mine, scratch);         // (its barriers also show the tanhs to everybody)
-  // A row of W2 is `rank` numbers: two warps' halves a channel each, sixteen lanes over the rank.
-  for (int d0 = 0; d0 < dim; d0 += kRowGroups) {
+  auto finish = [&](int d, float z) {
+#pragma unroll
+    for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
+    if (sub == 0 && d < dim) ws[d] = expf(-expf(z + w0[head * dim + d]));
+  };
+  if (early) {
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (4 * sub < rank) x = make_float4(th[4 * sub], th[4 * sub + 1], th[4 * sub + 2], th[4 * sub + 3]);
+#pragma unroll
+    for (int i = 0; i < (kEarly ? NPL : 1); ++i)
+      finish(i * kRowGroups + group, fmaf(wr[i][3], x.w, fmaf(wr[i][2], x.z, fmaf(wr[i][1], x.y, wr[i][0] * x.x))));
+  }
+  for (int d0 = early ? dim : 0; d0 < dim; d0 += kRowGroups) {
     const int d = d0 + group;
     float z = 0.f;
     if (d < dim)
       for (int i = sub; i < rank; i += 16) z = fmaf(to_float(w2[((size_t)head * dim + d) * rank + i]), th[i], z);
-#pragma unroll
-    for (int o = 8; o > 0; o >>= 1) z += __shfl_xor_sync(0xffffffffu, z, o);
-    if (sub == 0 && d < dim) ws[d] = expf(-expf(z + w0[head * dim + d]));
+    finish(d, z);
   }
   __syncthreads();
   walk_columns<NPL, true>(base, dim, dim, rs, ks, ws, 0.f, vs, s, sub, group,
@@ -727,16 +793,18 @@ LI_EXPORT int li_wkv_steps(int dtype, const void* r, const void* k, const void* 
   const int dimp = rounded_dim(dim), vdimp = rounded_columns(dim);
   const int per_block = dim >= 256 ? 1 : 256 / dim;
   const dim3 grid((tokens + kRecordTokens - 1) / kRecordTokens, (heads + per_block - 1) / per_block);
-  const size_t smem = (size_t)rank * kRecordTokens * sizeof(float);
+  const size_t smem = (size_t)rank * kRecordTokens * sizeof(float), pair = dtype == kFloat32 ? 8 : 4;
+  const bool pairs = dim % 2 == 0 && row_stride % 2 == 0 && (uintptr_t)r % pair == 0 && (uintptr_t)k % pair == 0 &&
+                     (uintptr_t)v % pair == 0 && (uintptr_t)w2t % pair == 0;
   cudaError_t e;
-  if (dtype == kFloat32)
-    e = launch_pdl(tokens, wkv_record_kernel<float>, grid, dim3(256), smem, stream, (const float*)r, (const float*)k,
-                   (const float*)v, row_stride, (const float*)low, low_stride, rank, (const float*)w2t, w0, u, group_records,
-                   head_records, bonus, tokens, heads, per_block, dim, dimp, vdimp);
-  else
-    e = launch_pdl(tokens, wkv_record_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)r, (const bf16*)k,
-                   (const bf16*)v, row_stride, (const bf16*)low, low_stride, rank, (const bf16*)w2t, w0, u, group_records,
-                   head_records, bonus, tokens, heads, per_block, dim, dimp, vdimp);
+#define LI_RECORD(T, P)                                                                                               \
+  e = launch_pdl(tokens, wkv_record_kernel<T, P>, grid, dim3(kRecordThreads), smem, stream, (const T*)r, (const T*)k, \
+                 (const T*)v, row_stride, (const T*)low, low_stride, rank, (const T*)w2t, w0, u, group_records,       \
+                 head_records, bonus, tokens, heads, per_block, dim, dimp, vdimp)
+  if (dtype == kFloat32) { if (pairs) LI_RECORD(float, true); else LI_RECORD(float, false); }
+  else if (pairs) LI_RECORD(bf16, true);
+  else LI_RECORD(bf16, false);
+#undef LI_RECORD
   if (e != cudaSuccess) return (int)e;
 #define LI_STEPS(N, CHUNK)                                                                                            \
   return launch_memory<N, CHUNK, false>(tokens, num_seqs, stream, group_records, head_records, state, query_start_loc, \

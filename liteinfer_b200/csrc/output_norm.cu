@@ -42,23 +42,6 @@ __device__ __forceinline__ void put_four(bf16* p, const float (&v)[4]) {
   *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const unsigned*>(&a), *reinterpret_cast<const unsigned*>(&b));
 }
 
-// Two sums over a block at once (see block_sum); scratch of 66 floats.
-__device__ __forceinline__ float2 block_sum2(float2 v, float* scratch) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int nwarps = (blockDim.x + 31) >> 5;
-  v.x = warp_sum(v.x);
-  v.y = warp_sum(v.y);
-  __syncthreads();
-  if (lane == 0) { scratch[warp] = v.x; scratch[33 + warp] = v.y; }
-  __syncthreads();
-  if (warp == 0) {
-    const float a = warp_sum(lane < nwarps ? scratch[lane] : 0.f), b = warp_sum(lane < nwarps ? scratch[33 + lane] : 0.f);
-    if (lane == 0) { scratch[32] = a; scratch[65] = b; }
-  }
-  __syncthreads();
-  return make_float2(scratch[32], scratch[65]);
-}
-
 // NV: groups of four columns a thread keeps.  (x and a dense term may be the same rows: a thread reads its columns of all
 // terms before it stores any of x.)
 template <typename T, int NV>

@@ -356,6 +356,130 @@ projection_norm_rope_kv_write_kernel(T* __restrict__ qkv, size_t row_stride, con
   }
 }
 
+// The same with everything a thread works on in registers, for rows of at most 512 work items of 16-byte vectors (a head's
+// rotated part in pairs half a rotary width apart, then what passes through): a block takes TOK tokens one after the other,
+// so that norm weights and biases, in 32-bit several times a row's bytes, are fetched once for all of them.
+template <typename T, int TOK>
+__global__ void __launch_bounds__(512)
+projection_norm_rope_kv_write_reg_kernel(T* __restrict__ qkv, size_t row_stride, const int* __restrict__ positions,
+                                         const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                                         int table_stride, T* __restrict__ k_pool, T* __restrict__ v_pool,
+                                         const float* __restrict__ inv_freq, int heads, int kv_heads, int head_dim,
+                                         int rotary_dim, int page_size, int num_pages, int v_dim,
+                                         const float* __restrict__ q_norm, const float* __restrict__ k_norm, float q_count,
+                                         float k_count, float norm_eps, const float* __restrict__ bias, int values_are_keys,
+                                         float cs_scale, int tokens) {
+  constexpr int E = Vec16<T>::N;
+  extern __shared__ __align__(16) float shared[];   // cos [half], sin [half]
+  __shared__ float scratch[66];
+  const int q_width = heads * head_dim, qk_width = q_width + kv_heads * head_dim, half = rotary_dim / 2;
+  const int pairs = half / E, per_head = pairs + (head_dim - rotary_dim) / E;
+  const bool active = threadIdx.x < (heads + kv_heads) * per_head;
+  const int h = active ? threadIdx.x / per_head : 0, i = active ? threadIdx.x - h * per_head : 0;
+  const bool is_q = h < heads, paired = active && i < pairs;
+  const int j = i < pairs ? i * E : rotary_dim + (i - pairs) * E, at = h * head_dim + j;
+  float wlo[E], whi[E], blo[E], bhi[E];
+#pragma unroll
+  for (int e = 0; e < E; ++e) { wlo[e] = whi[e] = blo[e] = bhi[e] = 0.f; }
+  if (active) {                       // inputs of the model, not of a kernel: on their way before the wait
+    const float* w = is_q ? q_norm + at : k_norm + (at - q_width);
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      wlo[e] = w[e];
+      if (paired) whi[e] = w[half + e];
+      if (bias != nullptr) {
+        blo[e] = bias[at + e];
+        if (paired) bhi[e] = bias[at + half + e];
+      }
+    }
+  }
+  grid_launch_dependents();
+  grid_dependency_wait();
+  for (int n = 0; n < TOK; ++n) {
+    const int t = blockIdx.x * TOK + n;
+    if (t >= tokens) return;
+    T* row = qkv + (size_t)t * row_stride;
+    float lo[E], hi[E];
+#pragma unroll
+    for (int e = 0; e < E; ++e) lo[e] = hi[e] = 0.f;
+    if (active) unpack16(load16(row + at), lo);
+    if (paired) unpack16(load16(row + at + half), hi);
+    const int pos = positions[t], seq = seq_of_token[t];
+    if (n > 0) __syncthreads();       // the table of the token before has been read
+    for (int k = threadIdx.x; k < half; k += blockDim.x) {
+      const float angle = __fmul_rn((float)pos, inv_freq[k]);
+      shared[k] = cosf(angle) * cs_scale;
+      shared[half + k] = sinf(angle) * cs_scale;
+    }
+    const int page = seq < 0 ? -1 : block_table[(size_t)seq * table_stride + pos / page_size];
+    const bool store = page >= 0 && page < num_pages;
+    const int slot = pos % page_size;
+    float sum = 0.f;
+#pragma unroll
+    for (int e = 0; e < E; ++e) {
+      lo[e] += blo[e];
+      hi[e] += bhi[e];
+      sum = fmaf(lo[e], lo[e], fmaf(hi[e], hi[e], sum));
+    }
+    const size_t kv_row = ((size_t)page * kv_heads + (h - heads)) * page_size + slot;      // (of a key's head that is stored)
+    Vec16<T> v;
+    if (active && !is_q && store && values_are_keys) {                                    // (then v_dim == head_dim)
+#pragma unroll
+      for (int e = 0; e < E; ++e) v.set(e, lo[e]);
+      store16(v_pool + kv_row * v_dim + j, v);
+      if (paired) {
+#pragma unroll
+        for (int e = 0; e < E; ++e) v.set(e, hi[e]);
+        store16(v_pool + kv_row * v_dim + j + half, v);
+      }
+    }
+    const float2 sums = block_sum2(make_float2(is_q ? sum : 0.f, is_q ? 0.f : sum), scratch);
+    if (active && (is_q || store)) {
+      const float inv = 1.0f / sqrtf(is_q ? sums.x / q_count + norm_eps : sums.y / k_count + norm_eps);
+#pragma unroll
+      for (int e = 0; e < E; ++e) lo[e] = lo[e] * inv * wlo[e];
+      if (paired) {
+#pragma unroll
+        for (int e = 0; e < E; ++e) {
+          const float a = lo[e], b = hi[e] * inv * whi[e], c = shared[j + e], s = shared[half + j + e];
+          lo[e] = rotate_lo(a, b, c, s);
+          hi[e] = rotate_hi(a, b, c, s);
+        }
+      }
+      T* dst = is_q ? row + at : k_pool + kv_row * head_dim + j;
+#pragma unroll
+      for (int e = 0; e < E; ++e) v.set(e, lo[e]);
+      store16(dst, v);
+      if (paired) {
+#pragma unroll
+        for (int e = 0; e < E; ++e) v.set(e, hi[e]);
+        store16(dst + half, v);
+      }
+    }
+    if (!store || values_are_keys) continue;
+    for (int k = threadIdx.x; k < kv_heads * v_dim; k += blockDim.x) {
+      const int hv = k / v_dim, d = k - hv * v_dim;
+      float x = to_float(row[qk_width + k]);
+      if (bias != nullptr) x += bias[qk_width + k];
+      v_pool[(((size_t)page * kv_heads + hv) * page_size + slot) * v_dim + d] = from_float<T>(x);
+    }
+  }
+}
+
+template <typename T, int TOK>
+static int launch_projection_norm_reg(cudaStream_t stream, int items, int tokens, void* qkv, size_t row_stride,
+                                      const int* positions, const int* seq_of_token, const int* block_table, int table_stride,
+                                      void* k_pool, void* v_pool, const float* inv_freq, int heads, int kv_heads, int head_dim,
+                                      int rotary_dim, int page_size, int num_pages, int v_dim, const float* q_norm,
+                                      const float* k_norm, float q_count, float k_count, float norm_eps, const float* bias,
+                                      int values_are_keys, float cs_scale) {
+  return (int)launch_pdl(tokens, projection_norm_rope_kv_write_reg_kernel<T, TOK>, dim3((tokens + TOK - 1) / TOK),
+                         dim3((items + 31) / 32 * 32), (size_t)rotary_dim * sizeof(float), stream, (T*)qkv, row_stride,
+                         positions, seq_of_token, block_table, table_stride, (T*)k_pool, (T*)v_pool, inv_freq, heads, kv_heads,
+                         head_dim, rotary_dim, page_size, num_pages, v_dim, q_norm, k_norm, q_count, k_count, norm_eps, bias,
+                         values_are_keys, cs_scale, tokens);
+}
+
 template <typename T, int E>
 static int launch_projection_norm(cudaStream_t stream, size_t smem, int tokens, void* qkv, size_t row_stride,
                                   const int* positions, const int* seq_of_token, const int* block_table, int table_stride,
@@ -656,6 +780,19 @@ LI_EXPORT int li_projection_norm_rope_kv_write(int dtype, void* qkv, size_t row_
   const int n = dtype == kFloat32 ? 4 : 8;
   const bool fits = (rotary_dim / 2) % n == 0 && head_dim % n == 0 && rotary_dim % n == 0 && row_stride % n == 0 &&
                     aligned16(qkv) && aligned16(k_pool) && aligned16(v_pool);
+  const int items = fits ? (heads + kv_heads) * (rotary_dim / 2 / n + (head_dim - rotary_dim) / n) : 0;
+  if (fits && items <= 512 && rotary_dim <= 8192) {
+    // Wide steps: four tokens a block (weights and biases are read a quarter as often); narrow ones: one.
+#define LI_PREP_REG(T, TOK)                                                                                            \
+  return launch_projection_norm_reg<T, TOK>(stream, items, tokens, qkv, row_stride, positions, seq_of_token, block_table, \
+                                            table_stride, k_pool, v_pool, inv_freq, heads, kv_heads, head_dim, rotary_dim, \
+                                            page_size, num_pages, v_dim, q_norm, k_norm, (float)q_count, (float)k_count, \
+                                            norm_eps, bias, values_are_keys, cs_scale)
+    if (dtype == kFloat32) { if (tokens >= 1024) LI_PREP_REG(float, 4); LI_PREP_REG(float, 1); }
+    if (tokens >= 1024) LI_PREP_REG(bf16, 4);
+    LI_PREP_REG(bf16, 1);
+#undef LI_PREP_REG
+  }
 #define LI_PREP(T, E)                                                                                                  \
   return launch_projection_norm<T, E>(stream, smem, tokens, qkv, row_stride, positions, seq_of_token, block_table,     \
                                       table_stride, k_pool, v_pool, inv_freq, heads, kv_heads, head_dim, rotary_dim,   \

@@ -131,7 +131,7 @@ _SIGNATURES = {
     "li_paged_attention_stream": ("attention_stream", [
         c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
         c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p,
-        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p]),
+        c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int, c_float, c_void_p]),
     "li_paged_attention_stream_supports": ("attention_stream", [c_int, c_int, c_int, c_int]),
     "li_paged_attention_stream_capacity": ("attention_stream", [c_int]),
     "li_paged_attention_stream_cluster_capacity": ("attention_stream", [c_int, c_int]),
@@ -972,7 +972,7 @@ def paged_attention_mma(q, q_row_stride, out, k_pool, v_pool, block_table, query
     sequences only): q is unrotated and the newest key and value are not in their pages yet; the kernel
     rotates q and the key and stores key and value itself.  `streaming` (single-token sequences, sizes that
     `stream_attention_supports` allows): the kernel that passes K and V through registers only.  `keep_first`
-    (with a window) and `softcap`: as in `paged_attention`; not with `newest` or `streaming`.  `sink`: as in
+    (with a window) and `softcap`: as in `paged_attention`; not with `newest`, and `keep_first` not with `streaming`.  `sink`: as in
     `paged_attention`; every form takes it.  `window` < 0: chunks of -window positions.  Values may be a multiple of
     the head size wide."""
     _rows2d(q, "q"); _rows2d(out, "out")
@@ -992,13 +992,13 @@ def paged_attention_mma(q, q_row_stride, out, k_pool, v_pool, block_table, query
     tail = (_ptr(newest.inv_freq if newest else None), _ptr(newest.k if newest else None),
             _ptr(newest.v if newest else None), int(newest.store) if newest else 0)
     if streaming:
-        assert max_q_len == 1 and keep_first <= 0 and softcap <= 0
+        assert max_q_len == 1 and keep_first <= 0 and (softcap <= 0 or newest is None)
         _check(_fn("li_paged_attention_stream")(
             q.data_ptr(), q_row_stride, out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(),
             block_table.data_ptr(), block_table.stride(0), query_start_loc.data_ptr(), context_lens.data_ptr(),
             _ptr(seq_index), num_seqs, heads, kv_heads, head_dim, page_size, pages, float(scale), int(window),
             int(num_splits), _ptr(partial_out), _ptr(partial_lse), _ptr(counters), *tail,
-            scratch_for(q.device).gemm_error.data_ptr(), _ptr(sink), v_dim, _stream()), "paged_attention_stream")
+            scratch_for(q.device).gemm_error.data_ptr(), _ptr(sink), v_dim, float(softcap), _stream()), "paged_attention_stream")
         return out
     _check(_fn("li_paged_attention_mma")(
         q.data_ptr(), q_row_stride, out.data_ptr(), out.stride(0), k_pool.data_ptr(), v_pool.data_ptr(),
@@ -1120,8 +1120,8 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
                                        context_lens, num_seqs, max_q_len, heads, kv_heads, head_dim, scale, window,
                                        keep_first, softcap, sink)
     common = (q, q_row_stride, out, k_pool, v_pool, block_table, query_start_loc, context_lens)
-    # Kept first keys and capped scores are options of the tcgen05 kernel (prompts) and of the mma.sync kernel
-    # (prompts it takes instead, and single tokens); the streaming decode kernel knows neither.
+    # Kept first keys are an option of the tcgen05 kernel (prompts) and of the mma.sync kernel (prompts it takes instead,
+    # and single tokens); the streaming decode kernel does not know them.  Capped scores every one of them takes.
     options = dict(keep_first=keep_first, softcap=softcap) if masked else {}
     if sink is not None:
         options["sink"] = sink
@@ -1137,7 +1137,7 @@ def paged_attention(q: torch.Tensor, q_row_stride: int, out: torch.Tensor, k_poo
                                 kv_heads, head_dim, scale, window, **options)
     if plan.num_decode:
         bound = min(plan.max_decode_context_len, reach) if reach else plan.max_decode_context_len
-        streaming = not masked and stream_attention_supports(q.dtype, heads, kv_heads, head_dim, page_size)
+        streaming = not (keep_first > 0 and window > 0) and stream_attention_supports(q.dtype, heads, kv_heads, head_dim, page_size)
         splits = decode_splits or decode_splits_for(plan.num_decode, kv_heads * parts, bound, head_dim, streaming)
         paged_attention_mma(*common, plan.decode_seqs, plan.num_decode, 1, heads, kv_heads, head_dim, scale,
                             window, splits, newest, streaming, **options)
