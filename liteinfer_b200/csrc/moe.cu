@@ -640,7 +640,8 @@ LI_EXPORT int li_moe_router(int dtype, const void* x, size_t x_stride, const flo
   const RouteRule rule{experts, top, groups, keep, renormalise, sigmoid, pair_rank, top + extra, floor, correction,
                        experts - identity_experts, identity};
   if (K < 1 || extra < 0 || (extra > 0 && !gated) || bad_rule(rule)) return LI_ERR_UNSUPPORTED;
-  if (identity_experts < 0 || (identity_experts > 0) != (identity != nullptr) || (identity_experts > 0 && gated)) return LI_ERR_UNSUPPORTED;
+  if (identity_experts < 0 || (identity_experts > 0) != (identity != nullptr) || (identity_experts > 0 && gated))
+    return LI_ERR_UNSUPPORTED;
   const bool wide = tokens > 128;
   const size_t smem = (size_t)(wide ? 8 : 1) * (route_floats(experts, groups) + 1) * sizeof(float);
   if (smem > 48 * 1024) return LI_ERR_UNSUPPORTED;

@@ -148,8 +148,8 @@ _SIGNATURES = {
                                              c_void_p, c_size_t, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
                                              c_float, c_void_p, c_void_p, c_int, c_void_p]),
     "li_gemm_skinny_plan": ("gemm_skinny", [c_int, c_int, c_void_p, c_void_p]),
-    "li_gemm_stream": ("gemm_stream", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p,
-                                       c_int, c_void_p, c_void_p]),
+    "li_gemm_stream": ("gemm_stream", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
+                                       c_void_p, c_int, c_void_p, c_void_p]),
     "li_gemm_stream_supports": ("gemm_stream", [c_int, c_int, c_int]),
     "li_gemm_tcgen05": ("gemm_tcgen05", [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float,
                                          c_void_p, c_void_p]),
@@ -2067,8 +2067,8 @@ def moe_grouped(mode: str, a: torch.Tensor, weight: torch.Tensor, out: torch.Ten
     _check(_fn("li_moe_grouped")(_code(a), {"gate_up": 0, "down": 1, "up": 2}[mode], a.data_ptr(), a.stride(0), weight.data_ptr(),
                                  out.data_ptr(), out.stride(0), plan.order.data_ptr(), plan.offsets.data_ptr(),
                                  plan.tile_expert.data_ptr(), plan.tile_row0.data_ptr(), _ptr(pair_weights), top, N, K,
-                                 EXPERT_ACTIVATIONS[activation] if mode == "gate_up" else 0, float(limit), float(alpha), plan.max_tiles,
-                                 plan.tile_rows, int(eights), _stream()), "moe_grouped")
+                                 EXPERT_ACTIVATIONS[activation] if mode == "gate_up" else 0, float(limit), float(alpha),
+                                 plan.max_tiles, plan.tile_rows, int(eights), _stream()), "moe_grouped")
     return out
 
 
